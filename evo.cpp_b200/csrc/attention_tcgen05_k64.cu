@@ -27,9 +27,16 @@
 // so the row maximum and the row sum are its own (no exchange between warps),
 // with the scale-and-shift and the sums as packed F32 pairs.  Every wait is
 // time-bounded and raises the sticky error word of the projection kernels.
+//
+// The same walk with kWindow is the window attention of decoder blocks (window_attention, decoder_ops.hpp):
+// head sizes 64 .. 128 in steps of 8 (the tensor maps are [rows, heads, dim], so a box that reaches past a
+// head's end reads zeros), grouped key/value heads, only the key tiles that the window and the kept first
+// tokens touch, scores capped by tanh and lowered by a distance table, a sink in the row sum and a sigmoid
+// gate per row and head on the output.
 #include <cuda.h>
 
 #include "common.cuh"
+#include "decoder_types.cuh"
 #include "ops_internal.hpp"
 #include "projection_featurizer.cuh"  // round_pair_bf16
 #include "tcgen05.cuh"
@@ -156,10 +163,27 @@ __device__ __forceinline__ void tmem_store_16(const std::uint32_t taddr, const s
 }
 __device__ __forceinline__ void tmem_store_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
+struct WindowParams {
+  int kv_heads, dim, value_dim, window, keep_first;
+  float scale, softcap;
+  const float *distance_bias;  // [heads, bias_stride] or null
+  std::size_t bias_stride;
+  const bf16 *gate;            // [rows, gate_stride] or null
+  std::size_t gate_stride;
+  int sink;
+};
+
+__device__ __forceinline__ float fast_reciprocal(const float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <bool kWindow>
 __global__ void __launch_bounds__(kThreads, 2)
 flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, bf16 *const output, const int rows,
-                         const int total_keys, const int heads, int *const error_word) {
+                         const int total_keys, const int heads, const WindowParams w, int *const error_word) {
   extern __shared__ __align__(1024) unsigned char smem[];
   const std::uint32_t smem_base = smem_u32(smem);
   auto bar = [&](const int index) { return smem_base + kBarrierOffset + 8U * index; };
@@ -174,7 +198,18 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int prefix = total_keys - rows;
   // keys this block may see: 0 .. prefix + q0 + 127, inside the cache
   const int visible = min(total_keys, prefix + q0 + kRows);
-  const int tiles = (visible + kKeys - 1) / kKeys;
+  int tiles = (visible + kKeys - 1) / kKeys;
+  // window form: tiles with kept first tokens, then the tiles from the first row's window on
+  int kept_tiles = 0, low_tile = 0;
+  if constexpr (kWindow) {
+    low_tile = w.window > 0 ? max(0, prefix + q0 - w.window + 1) / kKeys : 0;
+    kept_tiles = min((w.keep_first + kKeys - 1) / kKeys, low_tile);
+    tiles += kept_tiles - low_tile;
+  }
+  const auto first_key = [&](const int j) {
+    if constexpr (kWindow) return (j < kept_tiles ? j : low_tile + (j - kept_tiles)) * kKeys;
+    else return j * kKeys;
+  };
 
   if (threadIdx.x == 0) {
     mbar_init(bar(kQFull), 1);
@@ -210,22 +245,31 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   } else if (warp == 0) {
     if (lane == 0) {
       const int column = head * kRows;
+      int kv_head = 0;
+      if constexpr (kWindow) kv_head = head / (heads / w.kv_heads);
+      const auto load_tile = [&](const std::uint32_t dst, const CUtensorMap *const map, const std::uint32_t full,
+                                 const int half_bytes, const int map_head, const int row) {
+        if constexpr (kWindow) {
+          tma_load_3d(dst, map, full, 0, map_head, row);
+          tma_load_3d(dst + half_bytes, map, full, 64, map_head, row);
+        } else {
+          tma_load_2d(dst, map, full, column, row);
+          tma_load_2d(dst + half_bytes, map, full, column + 64, row);
+        }
+      };
       mbar_expect_tx(bar(kQFull), kQBytes);
-      tma_load_2d(smem_base + kQOffset, &map_q, bar(kQFull), column, q0);
-      tma_load_2d(smem_base + kQOffset + kQHalfBytes, &map_q, bar(kQFull), column + 64, q0);
+      load_tile(smem_base + kQOffset, &map_q, bar(kQFull), kQHalfBytes, head, q0);
       for (int j = 0; j < tiles; ++j) {
         const int s = j & 1;
         const std::uint32_t phase = (j >> 1) & 1U;
         if (!mbar_wait(bar(kKEmpty + s), phase ^ 1U, abort_flag)) break;
         const std::uint32_t k_dst = smem_base + kKOffset + s * kKvBytes;
         mbar_expect_tx(bar(kKFull + s), kKvBytes);
-        tma_load_2d(k_dst, &map_k, bar(kKFull + s), column, j * kKeys);
-        tma_load_2d(k_dst + kKvHalfBytes, &map_k, bar(kKFull + s), column + 64, j * kKeys);
+        load_tile(k_dst, &map_k, bar(kKFull + s), kKvHalfBytes, kv_head, first_key(j));
         if (!mbar_wait(bar(kVEmpty + s), phase ^ 1U, abort_flag)) break;
         const std::uint32_t v_dst = smem_base + kVOffset + s * kKvBytes;
         mbar_expect_tx(bar(kVFull + s), kKvBytes);
-        tma_load_2d(v_dst, &map_v, bar(kVFull + s), column, j * kKeys);
-        tma_load_2d(v_dst + kKvHalfBytes, &map_v, bar(kVFull + s), column + 64, j * kKeys);
+        load_tile(v_dst, &map_v, bar(kVFull + s), kKvHalfBytes, kv_head, first_key(j));
       }
     }
   } else if (warp == 1) {
@@ -275,10 +319,27 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int row = quarter * 32 + lane;  // query row inside the block = TMEM lane
     const std::uint32_t lane_base = static_cast<std::uint32_t>(quarter * 32) << 16U;
     const int position = prefix + q0 + row;  // last key this row may see
-    const float scale_log2 = 1.4426950408889634F * rsqrtf(static_cast<float>(kRows));
+    constexpr float kLog2e = 1.4426950408889634F;
+    // window form: the scores are final and in base-2 units before the maximum is taken
+    const float scale_log2 = kWindow ? 1.0F : kLog2e * rsqrtf(static_cast<float>(kRows));
     const float slack = kLazyDoublings / scale_log2;  // in score units
     const unsigned long long scale_pair = pack_f32x2(scale_log2, scale_log2);
     float reference = -INFINITY, running_sum = 0.0F;
+    float cap_log2 = 0.0F, score_scale = 0.0F;
+    const float *bias_row = nullptr;
+    if constexpr (kWindow) {
+      if (w.sink != 0) {  // the sink is a score of 0 without a value
+        reference = 0.0F;
+        running_sum = 1.0F;
+      } else {
+        reference = -3.0e38F;  // finite: a tile may hide every key from a row
+      }
+      cap_log2 = w.softcap * kLog2e;
+      // with a cap: exponent of e^(2 s / cap) in base 2; without: the score in base 2
+      score_scale = w.softcap > 0.0F ? w.scale * 2.0F * kLog2e / w.softcap : w.scale * kLog2e;
+      // (rows past the last query compute on table entries inside the table and are not stored)
+      if (w.distance_bias != nullptr) bias_row = w.distance_bias + head * w.bias_stride + min(position, total_keys - 1);
+    }
     bool ok = true;
 
     for (int j = 0; j < tiles; ++j) {
@@ -297,7 +358,42 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) v[i] = chunk[i / 32][i % 32];
       }
-      if (j * kKeys + kKeys - 1 > prefix + q0) {     // some key hidden from some row
+      if constexpr (kWindow) {
+        const int key0 = first_key(j);
+        const bool partial = key0 + kKeys - 1 > prefix + q0 ||
+                             (w.window > 0 && prefix + q0 + kRows - 1 - key0 >= w.window && key0 + kKeys > w.keep_first);
+        if (w.softcap > 0.0F) {
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) {
+            const float e = fast_exp2(__uint_as_float(v[i]) * score_scale);
+            v[i] = __float_as_uint(fmaf(-2.0F * cap_log2, fast_reciprocal(e + 1.0F), cap_log2));  // cap tanh(s / cap)
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * score_scale);
+        }
+        if (bias_row != nullptr) {
+          const int distance0 = min(position, total_keys - 1) - key0;
+          const float *const bias = bias_row - key0;
+          if (partial) {
+#pragma unroll
+            for (int i = 0; i < kKeys; ++i)
+              v[i] = __float_as_uint(fmaf(-kLog2e, __ldg(bias - min(i, distance0)), __uint_as_float(v[i])));
+          } else {
+#pragma unroll
+            for (int i = 0; i < kKeys; ++i)
+              v[i] = __float_as_uint(fmaf(-kLog2e, __ldg(bias - i), __uint_as_float(v[i])));
+          }
+        }
+        if (partial) {
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) {
+            const int key = key0 + i;
+            const bool seen = key <= position && (w.window == 0 || position - key < w.window || key < w.keep_first);
+            if (!seen) v[i] = 0xff800000U;  // -inf
+          }
+        }
+      } else if (j * kKeys + kKeys - 1 > prefix + q0) {     // some key hidden from some row
 #pragma unroll
         for (int i = 0; i < kKeys; ++i)
           if (j * kKeys + i > position) v[i] = 0xff800000U;  // -inf
@@ -366,7 +462,31 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       __syncwarp();
       if (lane == 0) mbar_arrive(bar(kPFull));
     }
-    if (ok && tiles > 0 && mbar_wait(bar(kOFull), (tiles - 1) & 1U, abort_flag)) {
+    if (kWindow && ok && tiles > 0 && mbar_wait(bar(kOFull), (tiles - 1) & 1U, abort_flag)) {
+      tc_fence_after();
+      float factor = 1.0F / running_sum;
+      if (w.gate != nullptr && q0 + row < rows)
+        factor *= sigmoid_f32(bf2f(w.gate[static_cast<std::size_t>(q0 + row) * w.gate_stride + head]));
+      bf16 *const out = output + (static_cast<std::size_t>(q0 + row) * heads + head) * w.value_dim;
+#pragma unroll
+      for (int c = 0; c < kRows / 32; ++c) {
+        std::uint32_t o[32];
+        tmem_load_32(tmem_o + lane_base + c * 32, o);  // warp-wide: before the row test
+        tmem_load_wait();
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          if (q0 + row < rows && c * 32 + 8 * q < w.value_dim) {
+            uint4 word;
+            word.x = round_pair_bf16(__uint_as_float(o[8 * q]) * factor, __uint_as_float(o[8 * q + 1]) * factor);
+            word.y = round_pair_bf16(__uint_as_float(o[8 * q + 2]) * factor, __uint_as_float(o[8 * q + 3]) * factor);
+            word.z = round_pair_bf16(__uint_as_float(o[8 * q + 4]) * factor, __uint_as_float(o[8 * q + 5]) * factor);
+            word.w = round_pair_bf16(__uint_as_float(o[8 * q + 6]) * factor, __uint_as_float(o[8 * q + 7]) * factor);
+            *reinterpret_cast<uint4 *>(out + c * 32 + 8 * q) = word;
+          }
+        }
+      }
+    }
+    if (!kWindow && ok && tiles > 0 && mbar_wait(bar(kOFull), (tiles - 1) & 1U, abort_flag)) {
       tc_fence_after();
       const float inverse = 1.0F / running_sum;
       bf16 *const out = output + static_cast<std::size_t>(q0 + row) * (static_cast<std::size_t>(heads) * kRows) +
@@ -422,16 +542,58 @@ int flash_tcgen05_attention_k64(const void *query, const void *key_cache, const 
       (status = tc::make_bf16_tile_map(&map_k, key_cache, total_keys, width, kKeys)) != kOk ||
       (status = tc::make_bf16_tile_map(&map_v, value_cache, total_keys, width, kKeys)) != kOk)
     return status;
-  if (cudaFuncSetAttribute(flash_tcgen05_k64_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
-          cudaSuccess ||
-      cudaFuncSetAttribute(flash_tcgen05_k64_kernel, cudaFuncAttributePreferredSharedMemoryCarveout,
+  if (cudaFuncSetAttribute(flash_tcgen05_k64_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                           kSmemBytes) != cudaSuccess ||
+      cudaFuncSetAttribute(flash_tcgen05_k64_kernel<false>, cudaFuncAttributePreferredSharedMemoryCarveout,
                            cudaSharedmemCarveoutMaxShared) != cudaSuccess)
     return fail(kCuda, "cannot raise the attention shared-memory limit");
   const dim3 grid(ceil_div_u(rows, kRows), static_cast<unsigned int>(heads));
-  flash_tcgen05_k64_kernel<<<grid, kThreads, kSmemBytes, stream>>>(map_q, map_k, map_v, static_cast<bf16 *>(output),
-                                                                  static_cast<int>(rows), static_cast<int>(total_keys),
-                                                                  static_cast<int>(heads), error);
+  flash_tcgen05_k64_kernel<false><<<grid, kThreads, kSmemBytes, stream>>>(
+      map_q, map_k, map_v, static_cast<bf16 *>(output), static_cast<int>(rows), static_cast<int>(total_keys),
+      static_cast<int>(heads), WindowParams{}, error);
   return check_launch("tcgen05 attention kernel (64-key tiles)");
+}
+
+bool window_attention_tcgen05_applicable(const WindowAttentionArgs &a) {
+  const auto takes = [](const std::size_t dim) { return dim >= 64 && dim <= static_cast<std::size_t>(kRows) && dim % 8 == 0; };
+  return a.type == Activation::kBf16 && a.dynamic_position == nullptr && takes(a.dim) && takes(a.value_dim) &&
+         a.rows > 0 && a.position + a.rows < 0x7fff0000U && aligned16(a.query) && aligned16(a.key_cache) &&
+         aligned16(a.value_cache) && aligned16(a.output);
+}
+
+int window_attention_tcgen05(const WindowAttentionArgs &a, cudaStream_t stream) {
+  int status = kOk;
+  int *const error = tc::error_word(&status, nullptr);
+  if (error == nullptr) return status;
+  const std::size_t total_keys = a.position + a.rows;
+  CUtensorMap map_q, map_k, map_v;
+  if ((status = tc::make_bf16_head_map(&map_q, a.query, a.rows, a.heads, a.dim, kRows)) != kOk ||
+      (status = tc::make_bf16_head_map(&map_k, a.key_cache, total_keys, a.kv_heads, a.dim, kKeys)) != kOk ||
+      (status = tc::make_bf16_head_map(&map_v, a.value_cache, total_keys, a.kv_heads, a.value_dim, kKeys)) != kOk)
+    return status;
+  if (cudaFuncSetAttribute(flash_tcgen05_k64_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
+          cudaSuccess ||
+      cudaFuncSetAttribute(flash_tcgen05_k64_kernel<true>, cudaFuncAttributePreferredSharedMemoryCarveout,
+                           cudaSharedmemCarveoutMaxShared) != cudaSuccess)
+    return fail(kCuda, "cannot raise the attention shared-memory limit");
+  WindowParams w{};
+  w.kv_heads = static_cast<int>(a.kv_heads);
+  w.dim = static_cast<int>(a.dim);
+  w.value_dim = static_cast<int>(a.value_dim);
+  w.window = static_cast<int>(a.window >= total_keys ? 0 : a.window);  // nothing is hidden: no limit
+  w.keep_first = static_cast<int>(a.keep_first > total_keys ? total_keys : a.keep_first);
+  w.scale = a.scale;
+  w.softcap = a.softcap;
+  w.distance_bias = a.distance_bias;
+  w.bias_stride = a.bias_stride;
+  w.gate = static_cast<const bf16 *>(a.gate);
+  w.gate_stride = a.gate_stride;
+  w.sink = a.sink ? 1 : 0;
+  const dim3 grid(ceil_div_u(a.rows, kRows), static_cast<unsigned int>(a.heads));
+  flash_tcgen05_k64_kernel<true><<<grid, kThreads, kSmemBytes, stream>>>(
+      map_q, map_k, map_v, static_cast<bf16 *>(a.output), static_cast<int>(a.rows), static_cast<int>(total_keys),
+      static_cast<int>(a.heads), w, error);
+  return check_launch("tcgen05 window attention kernel");
 }
 
 }  // namespace evob

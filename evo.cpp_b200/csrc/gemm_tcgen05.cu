@@ -134,6 +134,25 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
       if (row < M && col < n_limit) {
         float *const out_row = ep.out_f32 + static_cast<std::size_t>(split) * ep.partial_stride +
                                static_cast<std::size_t>(row) * ep.ld_out;
+        if (col + 32 <= n_limit && (ep.ld_out % 4) == 0 && (ep.partial_stride % 4) == 0 &&
+            (reinterpret_cast<std::uintptr_t>(ep.out_f32) & 15U) == 0) {
+#pragma unroll
+          for (int q = 0; q < 8; ++q) {
+            float4 *const slot = reinterpret_cast<float4 *>(out_row + col + 4 * q);
+            float4 value = make_float4(__uint_as_float(v[4 * q]) * scale, __uint_as_float(v[4 * q + 1]) * scale,
+                                       __uint_as_float(v[4 * q + 2]) * scale, __uint_as_float(v[4 * q + 3]) * scale);
+            if (ep.bias_f32 != nullptr) {
+              const float *const b = ep.bias_f32 + col + 4 * q;
+              value.x += b[0], value.y += b[1], value.z += b[2], value.w += b[3];
+            }
+            if (ep.accumulate_f32 != 0) {
+              const float4 old = *slot;
+              value.x += old.x, value.y += old.y, value.z += old.z, value.w += old.w;
+            }
+            *slot = value;
+          }
+          continue;
+        }
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           if (col + j < n_limit) {
@@ -838,6 +857,12 @@ gemm_simt_kernel(const void *__restrict__ a_raw, const void *__restrict__ b_raw,
       const int col = n0 + tx * 4 + j;
       if (col >= N) continue;
       float value = acc[i][j] * (ep.row_scale != nullptr ? ep.alpha * ep.row_scale[row] : ep.alpha);
+      if (ep.out_f32 != nullptr) {
+        float *const slot = ep.out_f32 + static_cast<std::size_t>(row) * ep.ld_out + col;
+        if (ep.bias_f32 != nullptr) value += ep.bias_f32[col];
+        *slot = ep.accumulate_f32 != 0 ? *slot + value : value;
+        continue;
+      }
       if (ep.bias_mode == 1) value += bf2f(ep.bias[col]);
       value = rbf(value);
       if (ep.bias_mode == 2) value = rbf(value + bf2f(ep.bias[col]));
@@ -873,6 +898,12 @@ splitk_finish_kernel(const float *__restrict__ partials, const int splits, const
       const float first = ep.gate_mode == 2 ? bf2f(gelu_round(value)) : rbf(value);
       const float second = rbf(sum(first_column + 128));
       result = rbf(first * second);
+    } else if (ep.out_f32 != nullptr) {
+      float *const slot = ep.out_f32 + static_cast<std::size_t>(row) * ep.ld_out + col;
+      float value = sum(col);
+      if (ep.bias_f32 != nullptr) value += ep.bias_f32[col];
+      *slot = ep.accumulate_f32 != 0 ? *slot + value : value;
+      continue;
     } else {
       float value = sum(col);
       if (ep.bias_mode == 1) value += bf2f(ep.bias[col]);
@@ -1062,6 +1093,21 @@ int make_bf16_tile_map(CUtensorMap *map, const void *base, const std::size_t row
                        const std::size_t columns, const int box_rows) {
   return make_map(map, base, false, rows, columns, box_rows);
 }
+int make_bf16_head_map(CUtensorMap *map, const void *base, const std::size_t rows, const std::size_t heads,
+                       const std::size_t dim, const int box_rows) {
+  const EncodeTiled encode = encode_tiled();
+  if (encode == nullptr) return fail(kCuda, "cuTensorMapEncodeTiled is unavailable");
+  const cuuint64_t dims[3] = {dim, heads, rows};
+  const cuuint64_t strides[2] = {dim * 2, heads * dim * 2};
+  const cuuint32_t box[3] = {64, 1, static_cast<cuuint32_t>(box_rows)};
+  const cuuint32_t element_strides[3] = {1, 1, 1};
+  const CUresult result = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void *>(base), dims, strides,
+                                 box, element_strides, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+                                 CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (result != CUDA_SUCCESS)
+    return fail(kCuda, "cuTensorMapEncodeTiled failed with code " + std::to_string(static_cast<int>(result)));
+  return kOk;
+}
 int *error_word(int *status, int *sm_count) {
   DeviceState *const state = device_state(status);
   if (state == nullptr) return nullptr;
@@ -1116,7 +1162,9 @@ int linear(const LinearArgs &args, cudaStream_t stream) {
   if (args.output_f32 != nullptr &&
       (fp8 || args.gate_mode != 0 || args.bias_mode != 0 || args.residual != nullptr))
     return fail(kInvalidArgument, "the F32-result mode takes BF16 operands and no BF16 epilogue");
-  if (args.output_f32 == nullptr && args.row_scale == nullptr && small_batch_linear_applicable(args))
+  // (an F32 result keeps the tile kernel unless the caller gave a split workspace, i.e. wants the weight-stream forms)
+  if ((args.output_f32 == nullptr || args.split_workspace != nullptr) && args.weight_wrap_features == 0 &&
+      args.row_scale == nullptr && small_batch_linear_applicable(args))
     return small_batch_linear(args, stream);
   const std::size_t out_columns =
       args.gate_mode != 0 ? args.out_features / 2 : args.out_features;
@@ -1146,7 +1194,7 @@ int linear(const LinearArgs &args, cudaStream_t stream) {
   // (measured at 128 rows: 27.6 / 31.8 us against 34.8 / 71.7 us for 4096x4096 / 4096x11264 weights, but
   // 48 / 75 us against 37 / 61 us for 12288 / 22528 weight rows, where the tile kernel has enough tiles
   // and the partial sums cost more than the swap saves; at 16 rows 17 / 28 / 28 / 44 us against 33 / 72 / 37 / 59 us)
-  if (tma_ok && args.split_workspace != nullptr && args.output_f32 == nullptr &&
+  if (tma_ok && args.split_workspace != nullptr &&
       (args.rows <= 64 || (args.rows <= 128 && args.out_features <= 8192)) &&
       pitch % kBlockKBytes == 0 && args.weight_wrap_features == 0 &&
       (args.gate_mode == 0 || args.out_features % 256 == 0)) {

@@ -22,6 +22,9 @@ struct GemvParams {
   const void *w;       // [N, K] same type
   const bf16 *bias, *residual;
   bf16 *out;
+  float *out_f32;           // F32 result instead of out: [out_f32 +] alpha * sum [+ bias_f32]
+  const float *bias_f32;
+  int accumulate_f32;
   int rows, K, N;      // N = weight rows
   float alpha;
   int bias_mode, gate_mode;
@@ -161,6 +164,13 @@ gemv_kernel(const GemvParams p) {
     for (int w = 0; w < kWarps; ++w) sum += partial[w][c][r];
     return sum;
   };
+  if (p.out_f32 != nullptr) {
+    float *const slot = p.out_f32 + static_cast<std::size_t>(r) * out_columns + column;
+    float value = total(local) * p.alpha;
+    if (p.bias_f32 != nullptr) value += p.bias_f32[column];
+    *slot = p.accumulate_f32 != 0 ? *slot + value : value;
+    return;
+  }
   bf16 *const out_row = p.out + static_cast<std::size_t>(r) * out_columns;
   if (gated) {
     const float first = total(2 * local) * p.alpha, second = rbf(total(2 * local + 1) * p.alpha);
@@ -232,6 +242,9 @@ int small_batch_linear(const LinearArgs &a, cudaStream_t stream) {
   p.bias = static_cast<const bf16 *>(a.bias);
   p.residual = static_cast<const bf16 *>(a.residual);
   p.out = static_cast<bf16 *>(a.output);
+  p.out_f32 = a.output_f32;
+  p.bias_f32 = a.bias_f32;
+  p.accumulate_f32 = a.accumulate_f32 ? 1 : 0;
   p.rows = static_cast<int>(a.rows);
   p.K = static_cast<int>(a.in_features);
   p.N = static_cast<int>(a.out_features);

@@ -7,6 +7,7 @@
 #include "../../../include/evo/evo_b200.h"
 
 #include <algorithm>
+#include <cstddef>
 #include <cstring>
 #include <exception>
 #include <functional>
@@ -239,14 +240,18 @@ evo_status evo_context_create(const evo_model *model, const evo_context_params *
     const bool q8_kv = (p.flags & EVO_CONTEXT_FLAG_FAST_Q8_KV) != 0;
     const bool fp8_ffn = (p.flags & EVO_CONTEXT_FLAG_B200_FP8_FFN) != 0;
     const bool tensor_core = fp8_ffn || (p.flags & EVO_CONTEXT_FLAG_B200_TENSORCORE_FP8) != 0;
+    const bool float32 = (p.flags & EVO_CONTEXT_FLAG_B200_FLOAT32) != 0;
+    if (float32 && (tensor_core || q8_kv))
+      return fail(evob::kInvalidArgument, "the float32 profile does not combine with another one");
     auto context = std::make_unique<evo_context>();
-    context->profile = fp8_ffn ? "b200-fp8" : tensor_core ? "b200-tc" : "exact";
+    context->profile = float32 ? "float32" : fp8_ffn ? "b200-fp8" : tensor_core ? "b200-tc" : "exact";
     // upstream's name for the quantised-cache profile; the projection profile is appended when
     // it is not the default
     if (q8_kv) context->profile = context->profile == "exact" ? "fast-q8-kv" : "fast-q8-kv+" + context->profile;
     const int status = evob::Context::create(
         model->weights, p.context_size,
-        fp8_ffn       ? evob::ExecutionProfile::kTensorCoreFfn
+        float32       ? evob::ExecutionProfile::kFloat32
+        : fp8_ffn     ? evob::ExecutionProfile::kTensorCoreFfn
         : tensor_core ? evob::ExecutionProfile::kTensorCore
                       : evob::ExecutionProfile::kExact,
         (p.flags & EVO_CONTEXT_FLAG_B200_FULL_ARENA) != 0, &context->context, q8_kv);
@@ -731,7 +736,8 @@ evo_status evo_b200_scheduler_create(const evo_model *model, const evo_b200_sche
     auto handle = std::make_unique<evo_b200_scheduler>();
     const int status = evob::Scheduler::create(
         model->weights, params->workers, params->maximum_queue, params->context_size,
-        fp8_ffn       ? evob::ExecutionProfile::kTensorCoreFfn
+        (params->context_flags & EVO_CONTEXT_FLAG_B200_FLOAT32) != 0 ? evob::ExecutionProfile::kFloat32
+        : fp8_ffn     ? evob::ExecutionProfile::kTensorCoreFfn
         : tensor_core ? evob::ExecutionProfile::kTensorCore
                       : evob::ExecutionProfile::kExact,
         (params->context_flags & EVO_CONTEXT_FLAG_B200_FULL_ARENA) != 0, q8_kv, &handle->scheduler);
@@ -748,14 +754,19 @@ evo_status evo_b200_scheduler_submit(evo_b200_scheduler *scheduler, const evo_b2
   return protect([&]() -> int {
     if (ticket != nullptr) *ticket = 0;
     if (scheduler == nullptr || request == nullptr || ticket == nullptr ||
-        request->struct_size < sizeof(evo_b200_request) || (request->sequence == nullptr && request->length != 0))
+        request->struct_size < offsetof(evo_b200_request, tokens))
       return fail(evob::kInvalidArgument, "scheduler, request and ticket output are required");
+    const bool ids = request->struct_size >= sizeof(evo_b200_request) && request->tokens != nullptr;
+    if (!ids && request->sequence == nullptr && request->length != 0)
+      return fail(evob::kInvalidArgument, "a request needs its sequence");
     if (request->kind != EVO_B200_REQUEST_SCORE && request->kind != EVO_B200_REQUEST_GENERATE)
       return fail(evob::kInvalidArgument, "request kind must be score or generate");
     evob::SchedulerRequest copy;
     copy.kind = request->kind == EVO_B200_REQUEST_SCORE ? evob::SchedulerRequest::Kind::kScore
                                                         : evob::SchedulerRequest::Kind::kGenerate;
-    copy.sequence.assign(request->sequence, request->sequence + request->length);
+    if (ids) copy.tokens.assign(request->tokens, request->tokens + request->token_count);
+    else copy.tokens.assign(request->sequence, request->sequence + request->length);  // identity byte tokenizer
+    copy.byte_output = !ids;
     copy.new_tokens = request->new_tokens;
     if (copy.kind == evob::SchedulerRequest::Kind::kGenerate) {
       copy.sampling.temperature = request->sampler.temperature;
@@ -776,6 +787,8 @@ evo_status evo_b200_scheduler_submit(evo_b200_scheduler *scheduler, const evo_b2
           view.token_log_likelihoods = result.token_log_likelihoods.data();
           view.generated = result.generated.data();
           view.generated_length = result.generated.size();
+          view.generated_tokens = result.generated_tokens.data();
+          view.generated_token_count = result.generated_tokens.size();
           view.queue_seconds = result.queue_seconds;
           view.run_seconds = result.run_seconds;
           done(id, &view, user_data);

@@ -7,17 +7,22 @@
 // stdout and one `evo_metrics {...}` line on stderr; `embed` writes one NPY v1
 // F32 matrix per record plus an embeddings.jsonl manifest into an empty or new
 // directory (src/cuda/inference_cli.cpp:278-337, 972-1108).  Exit code = evo_status.
+// Models whose vocabulary is not bytes are driven with token ids: `run --prompt-tokens`, the `tokens` /
+// `prompt_tokens` members of serve requests, and `replay`, which feeds a recorded trace of token ids through
+// the model step by step and writes the logits that the trace asks for.
 #include <algorithm>
 #include <chrono>
 #include <cmath>
 #include <cstdint>
 #include <cstdio>
 #include <cstring>
+#include <deque>
 #include <filesystem>
 #include <fstream>
 #include <iomanip>
 #include <iostream>
 #include <limits>
+#include <map>
 #include <memory>
 #include <mutex>
 #include <sstream>
@@ -26,6 +31,7 @@
 
 #include "../../../include/evo/evo.h"
 #include "../../../include/evo/evo_b200.h"
+#include "json.hpp"
 
 namespace {
 
@@ -41,6 +47,9 @@ struct Options {
   // variant-score: inline (--sequence --position --ref --alt) or file form (--vcf --reference)
   std::string sequence, reference_allele, alternate_allele, strand = "both", normalization = "sum";
   std::string vcf_path, reference_path;
+  // token ids as prompt (run); replay
+  std::vector<uint32_t> prompt_tokens;
+  size_t max_tokens = 0;
   // serve
   size_t workers = 4, max_queue = 64;
   // generation / scoring diagnostics (upstream src/cli.cpp:166-172): how many prompt tokens the cached
@@ -174,6 +183,22 @@ bool json_field(const std::string &line, const std::string &key, std::string *va
   return false;
 }
 
+// Token ids of a JSON array (serve, replay) or of a comma-separated list (--prompt-tokens).
+bool json_ids(const evob::Json *array, std::vector<uint32_t> *ids) {
+  if (array == nullptr || array->kind != evob::Json::kArray) return false;
+  for (const evob::Json &item : array->items) {
+    if (item.kind != evob::Json::kNumber || !(item.number >= 0.0) || item.number > 4294967295.0 ||
+        item.number != std::floor(item.number))
+      return false;
+    ids->push_back(static_cast<uint32_t>(item.number));
+  }
+  return true;
+}
+
+void print_ids(std::ostream &out, const uint32_t *ids, const size_t count) {
+  for (size_t i = 0; i < count; ++i) out << (i ? "," : "") << ids[i];
+}
+
 struct Collected {
   std::vector<float> logits;
   size_t rows = 0, columns = 0;
@@ -264,7 +289,12 @@ Options parse(int argc, char **argv) {
     else if (a == "--repetitions") o.repetitions = std::stoull(value(i));
     else if (a == "--output-format") o.output_format = value(i);
     else if (a == "--name") o.name = value(i);
-    else if (a == "--output") o.output = value(i);
+    else if (a == "--output" || a == "--out") o.output = value(i);
+    else if (a == "--dtype") {
+      const std::string dtype = value(i);
+      if (dtype != "bfloat16" && dtype != "float32") die(EVO_STATUS_INVALID_ARGUMENT, "--dtype must be bfloat16 or float32");
+      o.profile = dtype == "float32" ? "float32" : "exact";
+    }
     else if (a == "--layer") o.layer = std::stoull(value(i));
     else if (a == "--pooling") o.pooling = value(i);
     else if (a == "--allow-test-fixture") o.allow_fixture = true;
@@ -290,6 +320,12 @@ Options parse(int argc, char **argv) {
       o.dump_layer = static_cast<size_t>(layer);
       o.dump_layer_path = spec.substr(colon + 1);
     }
+    else if (a == "--prompt-tokens") {
+      const std::string text = "[" + value(i) + "]";
+      evob::Json list;
+      if (!evob::JsonParser(text.data(), text.data() + text.size()).parse(&list) || !json_ids(&list, &o.prompt_tokens))
+        die(EVO_STATUS_INVALID_ARGUMENT, "--prompt-tokens must be token ids separated by commas");
+    } else if (a == "--max-tokens") o.max_tokens = std::stoull(value(i));
     else if (a == "--sequence") o.sequence = value(i);
     else if (a == "--vcf") o.vcf_path = value(i);
     else if (a == "--workers" || a == "--max-batch") o.workers = std::stoull(value(i));
@@ -307,7 +343,8 @@ Options parse(int argc, char **argv) {
       for (std::string item; std::getline(list, item, ',');) o.gpus.push_back(std::stoi(item));
     } else if (a == "--version") { std::cout << evo_version_string() << '\n'; std::exit(0); }
     else if (a == "--help" || a == "-h") {
-      std::cout << "usage:\n  evo run -m MODEL -p DNA -n TOKENS [--ctx N --gpu 0,1 --profile exact|b200-tc|b200-fp8|fast-q8-kv]\n"
+      std::cout << "usage:\n  evo run -m MODEL -p DNA -n TOKENS [--ctx N --gpu 0,1 --profile exact|b200-tc|b200-fp8|fast-q8-kv|float32]\n"
+                   "  evo run -m MODEL --prompt-tokens 1,2,3 -n TOKENS [...]   (prints token ids)\n"
                    "          [--force-prompt-threshold N --dump-tokens --dump-logits PATH --dump-layer INDEX:PATH]\n"
                    "  evo score -m MODEL --input FASTA_FASTQ_OR_TEXT [--dump-tokens --dump-logits PATH --dump-layer INDEX:PATH]\n"
                    "  evo bench -m MODEL --input FASTA_FASTQ_OR_TEXT [--warmup N --repetitions N]\n"
@@ -316,6 +353,7 @@ Options parse(int argc, char **argv) {
                    "  evo variant-score -m MODEL --sequence DNA --position POS --ref REF --alt ALT "
                    "[--window N --strand forward|reverse|both --normalization sum|mean]\n"
                    "  evo serve -m MODEL [--workers N --max-queue M --ctx N --profile ...] < requests.jsonl\n"
+                   "  evo replay -m MODEL --dtype bfloat16|float32 --out DIR --max-tokens N < steps.jsonl\n"
                    "  evo variant-score -m MODEL --vcf VARIANTS.vcf[.gz] --reference GENOME.fa "
                    "[--window N --strand ... --normalization ...]\n";
       std::exit(0);
@@ -327,8 +365,9 @@ Options parse(int argc, char **argv) {
     die(EVO_STATUS_INVALID_ARGUMENT, "--force-prompt-threshold is only valid for generation");
   if ((!o.dump_logits_path.empty() || !o.dump_layer_path.empty()) && !generation && o.command != "score")
     die(EVO_STATUS_INVALID_ARGUMENT, "--dump-logits and --dump-layer are valid for generation and scoring only");
-  if (o.profile != "exact" && o.profile != "b200-tc" && o.profile != "b200-fp8" && o.profile != "fast-q8-kv")
-    die(EVO_STATUS_UNSUPPORTED, "profile must be exact, b200-tc, b200-fp8 or fast-q8-kv");
+  if (o.profile != "exact" && o.profile != "b200-tc" && o.profile != "b200-fp8" && o.profile != "fast-q8-kv" &&
+      o.profile != "float32")
+    die(EVO_STATUS_UNSUPPORTED, "profile must be exact, b200-tc, b200-fp8, fast-q8-kv or float32");
   return o;
 }
 
@@ -377,15 +416,116 @@ Collected prefill_with_layer_dump(evo_context *context, const std::string &bytes
   return sink.logits;
 }
 
-evo_context *new_context(const evo_model *model, const Options &o) {
+evo_status create_context(const evo_model *model, const Options &o, evo_context **context) {
   evo_context_params params = evo_context_default_params();
   params.context_size = o.context;
+  if (o.profile == "float32") params.flags |= EVO_CONTEXT_FLAG_B200_FLOAT32;
   if (o.profile == "b200-tc") params.flags |= EVO_CONTEXT_FLAG_B200_TENSORCORE_FP8;
   if (o.profile == "b200-fp8") params.flags |= EVO_CONTEXT_FLAG_B200_FP8_FFN;
   if (o.profile == "fast-q8-kv") params.flags |= EVO_CONTEXT_FLAG_FAST_Q8_KV;
+  return evo_context_create(model, &params, context);
+}
+
+evo_context *new_context(const evo_model *model, const Options &o) {
   evo_context *context = nullptr;
-  check(evo_context_create(model, &params, &context), "context");
+  check(create_context(model, o, &context), "context");
   return context;
+}
+
+// `evo replay`: one JSON step per input line,
+//   {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["a"]}
+// Every request owns one context while it lives (generation's own: its first tokens start the sequence, a
+// single later token is a decode step, several are the next chunk of the prompt); contexts of ended requests
+// serve later ones.  The logits at the wanted places go to DIR/<step>.f32 in entry order, and a line
+// "done <step>" follows every step.
+constexpr int kNoFloat32Exit = 3;
+
+int replay(const evo_model *model, Options o) {
+  if (o.output.empty()) die(EVO_STATUS_INVALID_ARGUMENT, "replay needs --out");
+  const size_t vocab = evo_model_vocab_size(model), limit = evo_model_max_context(model);
+  o.context = o.max_tokens == 0 ? std::min<size_t>(o.context, limit) : std::min(o.max_tokens, limit);
+  std::deque<evo_context *> idle;
+  std::map<std::string, evo_context *> live;
+  evo_context *first = nullptr;
+  const evo_status created = create_context(model, o, &first);
+  if (created == EVO_STATUS_UNSUPPORTED && o.profile == "float32") die(kNoFloat32Exit, evo_last_error());
+  check(created, "context");
+  idle.push_back(first);
+  struct Sink {
+    const std::vector<size_t> *want;  // places in the entry, ascending or not
+    std::vector<float> *rows;
+    size_t begin;                     // slot of the entry's first wanted row in *rows
+    size_t position;                  // sequence position of the entry's first token
+    static evo_status take(const float *logits, size_t rows, size_t columns, size_t offset, void *user) {
+      const Sink &sink = *static_cast<Sink *>(user);
+      const size_t place0 = offset - sink.position;
+      for (size_t k = 0; k < sink.want->size(); ++k) {
+        const size_t place = (*sink.want)[k];
+        if (place >= place0 && place < place0 + rows)
+          std::copy_n(logits + (place - place0) * columns, columns, sink.rows->begin() + (sink.begin + k) * columns);
+      }
+      return EVO_STATUS_OK;
+    }
+  };
+  for (std::string line; std::getline(std::cin, line);) {
+    if (line.find_first_not_of(" \t\r") == std::string::npos) continue;
+    evob::Json step;
+    const evob::Json *number = nullptr, *entries = nullptr;
+    if (!evob::JsonParser(line.data(), line.data() + line.size()).parse(&step) ||
+        (number = step.get("step")) == nullptr || number->kind != evob::Json::kNumber ||
+        (entries = step.get("entries")) == nullptr || entries->kind != evob::Json::kArray)
+      die(EVO_STATUS_INVALID_ARGUMENT, "replay: a line is not a step");
+    const std::string name = std::to_string(static_cast<unsigned long long>(number->number));
+    std::vector<float> rows;
+    for (const evob::Json &entry : entries->items) {
+      const evob::Json *id = entry.get("id"), *places = entry.get("want");
+      std::vector<uint32_t> tokens, wanted;
+      if (id == nullptr || id->kind != evob::Json::kString || !json_ids(entry.get("tokens"), &tokens) || tokens.empty() ||
+          (places != nullptr && !json_ids(places, &wanted)))
+        die(EVO_STATUS_INVALID_ARGUMENT, "replay: step " + name + " has a malformed entry");
+      const std::vector<size_t> want(wanted.begin(), wanted.end());
+      for (const size_t place : want)
+        if (place >= tokens.size()) die(EVO_STATUS_INVALID_ARGUMENT, "replay: step " + name + " wants a place outside its tokens");
+      Sink sink{&want, &rows, rows.size() / vocab, 0};
+      rows.resize(rows.size() + want.size() * vocab);
+      auto found = live.find(id->text);
+      if (found == live.end()) {
+        if (idle.empty()) idle.push_back(new_context(model, o));
+        found = live.emplace(id->text, idle.front()).first;
+        idle.pop_front();
+        check(evo_b200_context_prefill_tokens(found->second, tokens.data(), tokens.size(), EVO_B200_PREFILL_FRESH,
+                                              Sink::take, &sink), "replay prompt");
+        continue;
+      }
+      evo_context *const context = found->second;
+      sink.position = evo_context_position(context);
+      if (tokens.size() == 1) {
+        check(evo_context_decode(context, tokens[0], Sink::take, &sink), "replay decode");
+        continue;
+      }
+      const size_t capacity = evo_b200_context_activation_capacity(context);
+      for (size_t begin = 0; begin < tokens.size(); begin += capacity)
+        check(evo_b200_context_prefill_tokens(context, tokens.data() + begin, std::min(capacity, tokens.size() - begin),
+                                              EVO_B200_PREFILL_CHUNK, Sink::take, &sink), "replay chunk");
+    }
+    if (!rows.empty()) {
+      std::ofstream out(std::filesystem::path(o.output) / (name + ".f32"), std::ios::binary | std::ios::trunc);
+      out.write(reinterpret_cast<const char *>(rows.data()), static_cast<std::streamsize>(rows.size() * sizeof(float)));
+      out.close();
+      if (!out) die(EVO_STATUS_IO, "cannot write the logits of step " + name);
+    }
+    if (const evob::Json *ended = step.get("end"))
+      for (const evob::Json &id : ended->items) {
+        const auto found = live.find(id.text);
+        if (found == live.end()) continue;
+        idle.push_back(found->second);
+        live.erase(found);
+      }
+    std::cout << "done " << name << std::endl;
+  }
+  for (const auto &entry : live) evo_context_free(entry.second);
+  for (evo_context *context : idle) evo_context_free(context);
+  return 0;
 }
 
 Collected prefill(evo_context *context, const std::string &bytes) {
@@ -473,6 +613,11 @@ int main(int argc, char **argv) {
   const size_t vocab = evo_model_vocab_size(model);
   evo_context *last_context = nullptr;
 
+  if (o.command == "replay") {
+    const int code = replay(model, o);
+    evo_model_free(model);
+    return code;
+  }
   if (o.command == "score") {
     if (o.input.empty()) die(EVO_STATUS_INVALID_ARGUMENT, "score needs --input");
     const bool dumping = !o.dump_logits_path.empty() || !o.dump_layer_path.empty();
@@ -756,6 +901,7 @@ int main(int argc, char **argv) {
     // order), on a pool of contexts that share the model's weights.
     //   {"id":"a","op":"score","sequence":"ACGT..."}
     //   {"id":"b","op":"generate","prompt":"ACGT","tokens":16,"temperature":1,"top_k":1,"top_p":1,"seed":0}
+    //   {"id":"c","op":"score","tokens":[5,17,3]}   {"id":"d","op":"generate","prompt_tokens":[5,17],"tokens":16}
     evo_b200_scheduler_params sp{};
     sp.struct_size = sizeof(sp);
     sp.workers = o.workers;
@@ -764,11 +910,13 @@ int main(int argc, char **argv) {
     if (o.profile == "b200-tc") sp.context_flags |= EVO_CONTEXT_FLAG_B200_TENSORCORE_FP8;
     if (o.profile == "b200-fp8") sp.context_flags |= EVO_CONTEXT_FLAG_B200_FP8_FFN;
     if (o.profile == "fast-q8-kv") sp.context_flags |= EVO_CONTEXT_FLAG_FAST_Q8_KV;
+    if (o.profile == "float32") sp.context_flags |= EVO_CONTEXT_FLAG_B200_FLOAT32;
     evo_b200_scheduler *scheduler = nullptr;
     check(evo_b200_scheduler_create(model, &sp, &scheduler), "scheduler");
     struct Pending {
       std::string id, op;
       std::mutex *output;
+      bool token_ids = false;
     };
     std::mutex output;
     const auto respond = [](uint64_t, const evo_b200_request_result *r, void *user) {
@@ -788,6 +936,10 @@ int main(int argc, char **argv) {
         line << std::setprecision(17) << ",\"tokens\":" << r->scored_tokens + 1 << ",\"scored_tokens\":"
              << r->scored_tokens << ",\"log_likelihood\":" << r->log_likelihood << ",\"mean_log_likelihood\":"
              << r->log_likelihood / static_cast<double>(r->scored_tokens);
+      } else if (pending->token_ids) {
+        line << ",\"generated_tokens\":[";
+        print_ids(line, r->generated_tokens, r->generated_token_count);
+        line << ']';
       } else {
         line << ",\"generated\":";
         json_string(line, std::string(reinterpret_cast<const char *>(r->generated), r->generated_length));
@@ -819,9 +971,16 @@ int main(int argc, char **argv) {
         std::cout << "}}\n";
         std::cout.flush();
       };
-      if (has_op && pending->op == "score" && json_field(line, "sequence", &payload)) {
+      // token ids instead of bytes: "tokens" of a score request, "prompt_tokens" of a generation
+      std::vector<uint32_t> ids;
+      {
+        evob::Json parsed;
+        if (evob::JsonParser(line.data(), line.data() + line.size()).parse(&parsed))
+          pending->token_ids = json_ids(parsed.get(pending->op == "score" ? "tokens" : "prompt_tokens"), &ids) && !ids.empty();
+      }
+      if (has_op && pending->op == "score" && (pending->token_ids || json_field(line, "sequence", &payload))) {
         request.kind = EVO_B200_REQUEST_SCORE;
-      } else if (has_op && pending->op == "generate" && json_field(line, "prompt", &payload)) {
+      } else if (has_op && pending->op == "generate" && (pending->token_ids || json_field(line, "prompt", &payload))) {
         request.kind = EVO_B200_REQUEST_GENERATE;
         try {
           if (json_field(line, "tokens", &number)) request.new_tokens = std::stoull(number);
@@ -839,6 +998,10 @@ int main(int argc, char **argv) {
       }
       request.sequence = reinterpret_cast<const uint8_t *>(payload.data());
       request.length = payload.size();
+      if (pending->token_ids) {
+        request.tokens = ids.data();
+        request.token_count = ids.size();
+      }
       uint64_t ticket = 0;
       Pending *const raw = pending.get();
       const evo_status submitted = evo_b200_scheduler_submit(scheduler, &request, respond, raw, &ticket);
@@ -856,8 +1019,12 @@ int main(int argc, char **argv) {
               << totals.active_peak << ",\"workers\":" << o.workers << "}}\n";
     evo_b200_scheduler_free(scheduler);
   } else if (o.command == "run") {
-    if (o.prompt.empty()) die(EVO_STATUS_INVALID_ARGUMENT, "run needs a prompt (-p)");
-    if (o.prompt.size() + o.tokens > o.context)
+    const bool token_ids = !o.prompt_tokens.empty();
+    std::vector<uint32_t> prompt_ids = o.prompt_tokens;
+    if (!token_ids)
+      for (const char c : o.prompt) prompt_ids.push_back(static_cast<unsigned char>(c));
+    if (prompt_ids.empty()) die(EVO_STATUS_INVALID_ARGUMENT, "run needs a prompt (-p)");
+    if (prompt_ids.size() + o.tokens > o.context)
       die(EVO_STATUS_INVALID_ARGUMENT, "prompt plus generated tokens exceed --ctx");
     evo_sampler_params sp = evo_sampler_default_params();
     sp.temperature = o.temperature;
@@ -867,13 +1034,14 @@ int main(int argc, char **argv) {
     evo_sampler *sampler = nullptr;
     check(evo_sampler_create(&sp, &sampler), "sampler");
     last_context = new_context(model, o);
-    if (o.dump_tokens) print_tokens("prompt", o.prompt);
+    if (o.dump_tokens && !token_ids) print_tokens("prompt", o.prompt);
+    if (token_ids && !o.dump_layer_path.empty()) die(EVO_STATUS_INVALID_ARGUMENT, "--dump-layer takes a byte prompt (-p)");
     // Upstream's generation pass (src/cuda/inference_cli.cpp:436-470): the first tokens of the prompt - all of
     // it up to min(3000, activation capacity) unless --force-prompt-threshold says otherwise - run as one
     // exact cached prefill, the rest of the prompt is teacher-forced through decode.
     const size_t capacity = evo_b200_context_activation_capacity(last_context);
     const size_t threshold = o.force_prompt_threshold != 0 ? o.force_prompt_threshold : std::min<size_t>(3000, capacity);
-    const size_t prefilled = std::min(o.prompt.size(), threshold);
+    const size_t prefilled = std::min(prompt_ids.size(), threshold);
     if (prefilled > capacity)
       die(EVO_STATUS_INVALID_ARGUMENT, "prompt prefill: exact cached prefill must fit one activation chunk; lower "
                                        "--force-prompt-threshold to at most " + std::to_string(capacity));
@@ -882,18 +1050,16 @@ int main(int argc, char **argv) {
     if (!o.dump_layer_path.empty()) {
       out = prefill_with_layer_dump(last_context, o.prompt.substr(0, prefilled), o, true);
     } else {
-      std::vector<uint32_t> ids(prefilled);
-      for (size_t i = 0; i < prefilled; ++i) ids[i] = static_cast<unsigned char>(o.prompt[i]);
-      check(evo_b200_context_prefill_tokens(last_context, ids.data(), ids.size(), EVO_B200_PREFILL_CACHED, collect, &out),
-            "prompt prefill");
+      check(evo_b200_context_prefill_tokens(last_context, prompt_ids.data(), prefilled, EVO_B200_PREFILL_CACHED, collect,
+                                            &out), "prompt prefill");
     }
     metrics.prefill_seconds = seconds_since(start);
     metrics.prefill_tokens = prefilled;
     std::vector<float> logits(out.logits.end() - static_cast<std::ptrdiff_t>(vocab), out.logits.end());
     start = std::chrono::steady_clock::now();
-    for (size_t i = prefilled; i < o.prompt.size(); ++i) {
+    for (size_t i = prefilled; i < prompt_ids.size(); ++i) {
       Collected step;
-      check(evo_context_decode(last_context, static_cast<unsigned char>(o.prompt[i]), collect, &step),
+      check(evo_context_decode(last_context, prompt_ids[i], collect, &step),
             "teacher-forced prompt token");
       logits = step.logits;
       ++metrics.teacher_force_tokens;
@@ -902,6 +1068,7 @@ int main(int argc, char **argv) {
     Matrix dumped;  // --dump-logits: the logits every sampling step saw, [generated tokens, vocabulary]
     dumped.columns = vocab;
     std::string generated;
+    std::vector<uint32_t> generated_ids;
     start = std::chrono::steady_clock::now();
     for (size_t i = 0; i < o.tokens; ++i) {
       if (!o.dump_logits_path.empty()) {
@@ -910,9 +1077,13 @@ int main(int argc, char **argv) {
       }
       uint32_t token = 0;
       check(evo_sampler_sample(sampler, logits.data(), vocab, &token), "sample");
-      uint8_t byte = 0;
-      check(evo_model_decode_token(model, token, &byte), "decode token");
-      generated.push_back(static_cast<char>(byte));
+      if (token_ids) {
+        generated_ids.push_back(token);
+      } else {
+        uint8_t byte = 0;
+        check(evo_model_decode_token(model, token, &byte), "decode token");
+        generated.push_back(static_cast<char>(byte));
+      }
       if (i + 1 == o.tokens) break;
       Collected step;
       check(evo_context_decode(last_context, token, collect, &step), "decode");
@@ -924,12 +1095,15 @@ int main(int argc, char **argv) {
       write_npy(o.dump_logits_path, dumped);
       metrics.retained_logits_peak_bytes = dumped.values.size() * sizeof(float);
     }
-    if (o.output_format == "fasta") std::cout << '>' << o.name << '\n' << generated << '\n';
+    if (token_ids) {
+      print_ids(std::cout, generated_ids.data(), generated_ids.size());
+      std::cout << '\n';
+    } else if (o.output_format == "fasta") std::cout << '>' << o.name << '\n' << generated << '\n';
     else std::cout << generated;
     std::cout.flush();
     evo_sampler_free(sampler);
   } else {
-    die(EVO_STATUS_UNSUPPORTED, "unknown command " + o.command + " (run, score, bench, embed, variant-score, serve)");
+    die(EVO_STATUS_UNSUPPORTED, "unknown command " + o.command + " (run, score, bench, embed, variant-score, serve, replay)");
   }
   print_metrics(metrics, o, last_context);
   if (last_context != nullptr) evo_context_free(last_context);

@@ -8,185 +8,14 @@
 #include <cstdlib>
 #include <cstring>
 
-#include "../common.cuh"
-#include "../ops_internal.hpp"
-#include "model.hpp"
+#include "stage.hpp"
 
 namespace evob {
 
 namespace {
 constexpr std::size_t kArenaRows = 8192;       // upstream src/cuda/model.cu:31
 constexpr std::size_t kFixtureArenaRows = 8;   // upstream src/cuda/model.cu:32
-
-#define EVOB_TRY(expr)                    \
-  do {                                    \
-    const int status__ = (expr);          \
-    if (status__ != kOk) return status__; \
-  } while (0)
-
-// Runs one operator launch; when the stage is profiling, brackets it with CUDA
-// events on the stage stream and files the elapsed time under `category`.
-#define EVOB_OP(category, expr)           \
-  do {                                    \
-    s.begin_op(category);                 \
-    const int status__ = (expr);          \
-    s.end_op();                           \
-    if (status__ != kOk) return status__; \
-  } while (0)
-
-struct DeviceGuard {
-  int previous = 0;
-  explicit DeviceGuard(const int device) {
-    cudaGetDevice(&previous);
-    cudaSetDevice(device);
-  }
-  ~DeviceGuard() { cudaSetDevice(previous); }
-};
 }  // namespace
-
-// Rows of history kept in front of a continuation chunk inside the activation
-// buffers (>= the longest filter's reach of 127 + 2 featurizer rows, and a
-// multiple of 16 so the tensor-core FIR tiles keep their alignment).
-constexpr std::size_t kHistoryPad = 144;
-constexpr std::size_t kSplitWorkspaceBytes = std::size_t{64} << 20;
-constexpr std::size_t kQ8PageTokens = 16384;  // upstream src/cuda/model.cu:33
-
-struct LayerState {
-  float *short_cache = nullptr;  // [3D, short_taps-1]
-  float *inner_cache = nullptr;  // [D, taps-1]
-  float *modal_state = nullptr;  // [D, S]
-  void *key_cache = nullptr, *value_cache = nullptr;  // [context, D] BF16
-  // Pipelines only: the last projection rows of the previous wavefront chunk
-  // ([history_rows, 3D] BF16).  The projection arena is shared by all blocks of
-  // a stage, so a block's own history is parked here between chunks.
-  void *history = nullptr;
-  std::size_t history_rows = 0;
-  // fast-q8-kv: page p holds positions [p * kQ8PageTokens, ...); pointers are mirrored in four
-  // device arrays (key codes, value codes, key scales, value scales) that the kernels index
-  std::vector<void *> q8_pages[4];
-  void **q8_tables = nullptr;  // [4][page_count] device
-  std::size_t q8_page_count = 0;
-  Q8PageTable q8_table() const {
-    Q8PageTable t;
-    t.key = reinterpret_cast<std::int8_t *const *>(q8_tables);
-    t.value = reinterpret_cast<std::int8_t *const *>(q8_tables + q8_page_count);
-    t.key_scale = reinterpret_cast<float *const *>(q8_tables + 2 * q8_page_count);
-    t.value_scale = reinterpret_cast<float *const *>(q8_tables + 3 * q8_page_count);
-    t.page_tokens = kQ8PageTokens;
-    return t;
-  }
-};
-
-struct Context::Stage {
-  std::shared_ptr<StageWeights> weights;
-  int device = 0;
-  cudaStream_t stream = nullptr;
-  cudaEvent_t done = nullptr;
-  std::vector<void *> allocations;
-  std::size_t arena_bytes = 0, cache_bytes = 0;
-  // activations
-  void *hidden = nullptr, *residual = nullptr, *normalized = nullptr, *mixer_out = nullptr;
-  void *codes = nullptr, *projection = nullptr, *query = nullptr, *gated = nullptr;
-  void *codes_wide = nullptr;   // [T, I] E4M3 codes of the gated MLP activations (FP8 FFN profile)
-  float *row_scale = nullptr;   // [T] dequantisation factor of the row-quantised operand in flight
-  void *mlp_first = nullptr, *mlp_second = nullptr;
-  void *short_filtered = nullptr, *x2 = nullptr, *x1 = nullptr, *value = nullptr, *pregate = nullptr;
-  float *modal_scratch = nullptr;
-  void *split_workspace = nullptr;  // F32 partial sums of split-K projections (<= 128 rows)
-  // fast-q8-kv: BF16 images [context, D] of the keys and values one attention block at a time
-  void *kv_image_key = nullptr, *kv_image_value = nullptr;
-  std::uint32_t *tokens = nullptr;
-  void *logits = nullptr;
-  std::vector<LayerState> layers;
-
-  // ---- optional per-operator timing
-  bool profiling = false;
-  std::vector<cudaEvent_t> events;    // pairs: start, stop
-  std::vector<int> event_category;    // one per pair in use
-  double category_ms[kProfileCategories] = {};
-  std::uint64_t category_launches[kProfileCategories] = {};
-
-  void begin_op(const int category) {
-    if (!profiling) return;
-    const std::size_t pair = event_category.size();
-    while (events.size() < 2 * (pair + 1)) {
-      cudaEvent_t event = nullptr;
-      cudaEventCreate(&event);
-      events.push_back(event);
-    }
-    event_category.push_back(category);
-    cudaEventRecord(events[2 * pair], stream);
-  }
-  void end_op() {
-    if (!profiling || event_category.empty()) return;
-    cudaEventRecord(events[2 * (event_category.size() - 1) + 1], stream);
-  }
-  // Call after the stream has been synchronised.
-  void collect_profile() {
-    for (std::size_t pair = 0; pair < event_category.size(); ++pair) {
-      float ms = 0.0F;
-      if (cudaEventElapsedTime(&ms, events[2 * pair], events[2 * pair + 1]) == cudaSuccess) {
-        category_ms[event_category[pair]] += ms;
-        ++category_launches[event_category[pair]];
-      }
-    }
-    event_category.clear();
-  }
-
-  // Advances (or rewinds) every row-indexed activation pointer by `rows`.
-  void shift_rows(const long rows, const std::size_t D, const std::size_t I) {
-    const auto move = [rows](void *&pointer, const std::size_t row_bytes) {
-      if (pointer != nullptr)
-        pointer = static_cast<unsigned char *>(pointer) + rows * static_cast<long>(row_bytes);
-    };
-    for (void **p : {&hidden, &residual, &normalized, &mixer_out, &query, &x2, &x1, &value, &pregate})
-      move(*p, D * 2);
-    move(codes, D);
-    move(codes_wide, I);
-    if (row_scale != nullptr) row_scale += rows;
-    move(projection, D * 6);
-    move(short_filtered, D * 6);
-    for (void **p : {&gated, &mlp_first, &mlp_second}) move(*p, I * 2);
-  }
-
-  // Pages of one attention block up to position `tokens_end` (exclusive); new pointers are
-  // written into the device tables in stream order.
-  int ensure_q8_pages(LayerState &state, const std::size_t tokens_end, const std::size_t heads,
-                      const std::size_t head_dim) {
-    const std::size_t needed = (tokens_end + kQ8PageTokens - 1) / kQ8PageTokens;
-    if (needed > state.q8_page_count) return fail(kInvalidArgument, "quantised KV cache capacity exceeded");
-    for (std::size_t page = state.q8_pages[0].size(); page < needed; ++page) {
-      for (int which = 0; which < 4; ++which) {
-        void *memory = nullptr;
-        const std::size_t bytes = which < 2 ? kQ8PageTokens * heads * head_dim : kQ8PageTokens * heads * sizeof(float);
-        const int status = allocate(&memory, bytes, &cache_bytes);
-        if (status != kOk) return status;
-        state.q8_pages[which].push_back(memory);
-        if (cudaMemcpyAsync(state.q8_tables + which * state.q8_page_count + page, &state.q8_pages[which][page],
-                            sizeof(void *), cudaMemcpyHostToDevice, stream) != cudaSuccess)
-          return fail(kCuda, "cannot publish a quantised KV page");
-      }
-    }
-    return kOk;
-  }
-
-  int allocate(void **out, const std::size_t bytes, std::size_t *counter) {
-    if (cudaMalloc(out, bytes == 0 ? 16 : bytes) != cudaSuccess)
-      return fail(kCuda, "cannot allocate " + std::to_string(bytes >> 20) + " MiB on device " +
-                             std::to_string(device));
-    allocations.push_back(*out);
-    *counter += bytes;
-    return kOk;
-  }
-  ~Stage() {
-    DeviceGuard guard(device);
-    if (stream != nullptr) cudaStreamSynchronize(stream);
-    for (void *p : allocations) cudaFree(p);
-    for (cudaEvent_t event : events) cudaEventDestroy(event);
-    if (done != nullptr) cudaEventDestroy(done);
-    if (stream != nullptr) cudaStreamDestroy(stream);
-  }
-};
 
 // ---- activation taps (upstream dump_matching & friends, src/cuda/model.cu:1583-1742)
 namespace {
@@ -215,6 +44,8 @@ int deliver(const DumpPlan &plan, const std::size_t layer, const DumpPoint point
   }
   return kOk;
 }
+
+}  // namespace
 
 // BF16 [rows, columns] on the device -> F32 on the host -> sink.
 int emit_bf16(cudaStream_t stream, const DumpPlan &plan, const std::size_t layer, const DumpPoint point,
@@ -249,8 +80,6 @@ int emit_f32(cudaStream_t stream, const DumpPlan &plan, const std::size_t layer,
                 values.begin() + static_cast<std::ptrdiff_t>(row * active));
   return deliver(plan, layer, point, values, rows, active);
 }
-
-}  // namespace
 
 const char *dump_point_name(const int point) {
   static const char *const names[static_cast<int>(DumpPoint::kDumpPoints)] = {
@@ -400,12 +229,17 @@ int Context::decode_step_graph(const std::uint32_t *host_token, bool *launched) 
       return kOk;
     }
     dynamic_position_ = device_position_;
-    int status = embedding(first.tokens, first.weights->embedding, 1, c.width, c.vocab, first.hidden, stream);
-    if (status == kOk) status = run_stage(first, 1, Mode::kDecode, -1, nullptr);
+    int status = c.decoder() ? decoder_embed(first, first.tokens, 1, position_)
+                             : embedding(first.tokens, first.weights->embedding, 1, c.width, c.vocab, first.hidden, stream);
     if (status == kOk)
+      status = c.decoder() ? run_decoder_stage(first, 1, Mode::kDecode, position_, -1, nullptr, nullptr)
+                           : run_stage(first, 1, Mode::kDecode, -1, nullptr);
+    if (status == kOk && c.decoder()) {
+      status = decoder_head(first, 1);
+    } else if (status == kOk)
       status = rms_norm(first.hidden, first.weights->final_norm, 1, c.width, c.epsilon, first.normalized,
                         nullptr, 1.0F, stream);
-    if (status == kOk) {
+    if (status == kOk && !c.decoder()) {
       LinearArgs a;
       a.split_workspace = first.split_workspace;
       a.split_workspace_bytes = kSplitWorkspaceBytes;
@@ -452,6 +286,9 @@ int Context::create(std::shared_ptr<ModelWeights> weights, const std::size_t con
   context->weights_ = weights;
   context->profile_ = profile;
   context->q8_kv_ = q8_kv;
+  if (c.decoder() ? q8_kv || profile == ExecutionProfile::kTensorCoreFfn : profile == ExecutionProfile::kFloat32)
+    return fail(kUnsupported, c.decoder() ? "decoder graphs run in the exact, b200-tc and float32 profiles"
+                                          : "StripedHyena2 models have no float32 profile");
   if (const char *const parts = std::getenv("EVO_B200_FP8_FFN_PARTS"))
     context->fp8_ffn_parts_ = static_cast<unsigned>(std::strtoul(parts, nullptr, 0)) & 7U;
   context->context_size_ = context_size;
@@ -468,6 +305,11 @@ int Context::create(std::shared_ptr<ModelWeights> weights, const std::size_t con
     if (cudaStreamCreateWithFlags(&stage->stream, cudaStreamNonBlocking) != cudaSuccess ||
         cudaEventCreateWithFlags(&stage->done, cudaEventDisableTiming) != cudaSuccess)
       return fail(kCuda, "cannot create the context stream");
+    if (c.decoder()) {
+      EVOB_TRY(context->allocate_decoder_stage(*stage));
+      context->stages_.push_back(std::move(stage));
+      continue;
+    }
     std::size_t *arena = &stage->arena_bytes;
     EVOB_TRY(stage->allocate(&stage->hidden, T * D * 2, arena));
     EVOB_TRY(stage->allocate(&stage->residual, T * D * 2, arena));
@@ -614,7 +456,7 @@ const char *profile_category_name(const int category) {
   static const char *const names[kProfileCategories] = {
       "rms_norm", "gemm_bf16_tcgen05", "gemm_e4m3_tcgen05", "gemm_e4m3_emulated", "hcs_fused_fir",
       "hcm_fused_fir", "hcl_modal_scan", "attention", "state_step", "elementwise", "row_quantize",
-      "gemm_e4m3_ffn_tcgen05"};
+      "gemm_e4m3_ffn_tcgen05", "recurrent_mixer", "poly_norm"};
   return category >= 0 && category < kProfileCategories ? names[category] : "";
 }
 
@@ -1087,7 +929,7 @@ int Context::forward(const std::uint32_t *host_tokens, const std::uint32_t *devi
   // in front of them.  (Short chunks and the exact cached-attention profile
   // keep the step kernels.)
   const bool continuation_window = mode == Mode::kContinue && rows >= 16 && !cached_attention_ &&
-                                   capture_layer < 0 && history_current_ && dumps == nullptr;
+                                   capture_layer < 0 && history_current_ && dumps == nullptr && !c.decoder();
   struct ShiftBack {
     Context *context;
     bool active;
@@ -1102,8 +944,8 @@ int Context::forward(const std::uint32_t *host_tokens, const std::uint32_t *devi
     for (auto &stage : stages_) stage->shift_rows(static_cast<long>(kHistoryPad), c.width, c.inner_width);
   bool graph_step = false;
   if (decode_graph_allowed_ && mode == Mode::kDecode && stages_.size() == 1 && host_tokens != nullptr &&
-      !first.profiling && !cached_attention_ && c.head_dim() == 128 && capture_layer < 0 &&
-      dumps == nullptr && position_ >= std::max({c.short_taps, c.hcs_taps, c.hcm_taps}))
+      !first.profiling && !cached_attention_ && capture_layer < 0 && dumps == nullptr &&
+      (c.decoder() || (c.head_dim() == 128 && position_ >= std::max({c.short_taps, c.hcs_taps, c.hcm_taps}))))
     status = decode_step_graph(host_tokens, &graph_step);
   if (!graph_step && status == kOk) {
     DeviceGuard guard(first.device);
@@ -1114,11 +956,12 @@ int Context::forward(const std::uint32_t *host_tokens, const std::uint32_t *devi
       device_tokens = first.tokens;
     }
     if (status == kOk)
-      status = embedding(device_tokens, first.weights->embedding, rows, c.width, c.vocab, first.hidden,
-                         first.stream);
+      status = c.decoder() ? decoder_embed(first, device_tokens, rows, initial ? 0 : position_)
+                           : embedding(device_tokens, first.weights->embedding, rows, c.width, c.vocab, first.hidden,
+                                       first.stream);
   }
   const bool wavefront = stages_.size() > 1 && (mode == Mode::kPrefill || mode == Mode::kStateless) &&
-                         rows >= 512 && capture_layer < 0 && dumps == nullptr;
+                         rows >= 512 && capture_layer < 0 && dumps == nullptr && !c.decoder();
   if (wavefront && status == kOk) status = run_wavefront(rows, mode, capture_layer, captured);
   for (std::size_t index = 0; index < stages_.size() && status == kOk && !wavefront && !graph_step; ++index) {
     Stage &stage = *stages_[index];
@@ -1127,10 +970,12 @@ int Context::forward(const std::uint32_t *host_tokens, const std::uint32_t *devi
       Stage &previous = *stages_[index - 1];
       if (cudaStreamWaitEvent(stage.stream, previous.done, 0) != cudaSuccess ||
           cudaMemcpyPeerAsync(stage.hidden, stage.device, previous.hidden, previous.device,
-                              rows * c.width * 2, stage.stream) != cudaSuccess)
+                              rows * c.width * c.hidden_bytes(), stage.stream) != cudaSuccess)
         status = fail(kCuda, "stage hand-off failed");
     }
-    if (status == kOk)
+    if (status == kOk && c.decoder())
+      status = run_decoder_stage(stage, rows, mode, initial ? 0 : position_, capture_layer, captured, dumps);
+    else if (status == kOk)
       status = continuation_window
                    ? run_stage(stage, rows, Mode::kWindow, -1, nullptr, kHistoryPad, position_)
                    : run_stage(stage, rows, mode, capture_layer, captured, 0, 0, dumps);
@@ -1143,13 +988,15 @@ int Context::forward(const std::uint32_t *host_tokens, const std::uint32_t *devi
       Stage &last = *stages_.back();
       if (cudaStreamWaitEvent(first.stream, last.done, 0) != cudaSuccess ||
           cudaMemcpyPeerAsync(first.hidden, first.device, last.hidden, last.device,
-                              rows * c.width * 2, first.stream) != cudaSuccess)
+                              rows * c.width * c.hidden_bytes(), first.stream) != cudaSuccess)
         status = fail(kCuda, "stage hand-off failed");
     }
-    if (status == kOk && !graph_step)
+    if (status == kOk && !graph_step && c.decoder())
+      status = decoder_head(first, rows);
+    else if (status == kOk && !graph_step)
       status = rms_norm(first.hidden, first.weights->final_norm, rows, c.width, c.epsilon,
                         first.normalized, nullptr, 1.0F, first.stream);
-    if (status == kOk && !graph_step) {
+    if (status == kOk && !graph_step && !c.decoder()) {
       LinearArgs a;
       a.split_workspace = first.split_workspace;
       a.split_workspace_bytes = kSplitWorkspaceBytes;
@@ -1163,14 +1010,16 @@ int Context::forward(const std::uint32_t *host_tokens, const std::uint32_t *devi
       status = linear(a, first.stream);
     }
     if (status == kOk && logits != nullptr) {
-      std::vector<std::uint16_t> raw(rows * c.vocab);
-      if (cudaMemcpyAsync(raw.data(), first.logits, raw.size() * 2, cudaMemcpyDeviceToHost,
+      // BF16 logits are widened here; decoders' heads leave F32
+      std::vector<std::uint16_t> raw(c.decoder() ? 0 : rows * c.vocab);
+      logits->resize(rows * c.vocab);
+      void *const host = c.decoder() ? static_cast<void *>(logits->data()) : static_cast<void *>(raw.data());
+      if (cudaMemcpyAsync(host, first.logits, logits->size() * (c.decoder() ? 4 : 2), cudaMemcpyDeviceToHost,
                           first.stream) != cudaSuccess ||
           cudaStreamSynchronize(first.stream) != cudaSuccess) {
         status = fail(kCuda, std::string("logits read-back failed: ") +
                                  cudaGetErrorString(cudaGetLastError()));
       } else {
-        logits->resize(raw.size());
         for (std::size_t j = 0; j < raw.size(); ++j) {
           const std::uint32_t bits = static_cast<std::uint32_t>(raw[j]) << 16U;
           std::memcpy(&(*logits)[j], &bits, 4);
@@ -1194,7 +1043,8 @@ int Context::forward(const std::uint32_t *host_tokens, const std::uint32_t *devi
   history_current_ = (initial && !stateless) || continuation_window;
   position_ = stateless ? 0 : (initial ? rows : position_ + rows);
   state_valid_ = !stateless;
-  if (initial) cached_attention_ = mode == Mode::kCachedPrefill;
+  // (a decoder has one attention arithmetic: its cached prefill is an ordinary one)
+  if (initial) cached_attention_ = mode == Mode::kCachedPrefill && !c.decoder();
   return kOk;
 }
 

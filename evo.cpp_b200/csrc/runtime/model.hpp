@@ -1,5 +1,5 @@
-// StripedHyena2 runtime: configuration, device-resident weights, per-context
-// state and the layer pipeline.  Mirrors the public surface of upstream's
+// Model runtime: configuration, device-resident weights, per-context state and the layer pipeline of
+// StripedHyena2 models and of decoders described by a config.json.  Mirrors the public surface of upstream's
 // evo::cuda::PipelineModel (include/evo/cuda/model.hpp:107-229): load,
 // shared-weight contexts, prefill / stateless / cached prefill, chunk
 // continuation, decode, layer capture, stage reporting.
@@ -18,7 +18,13 @@
 
 namespace evob {
 
-enum class MixerType { kHcs, kHcm, kHcl, kAttention };
+// The last three are mixers of decoder blocks (BlockGraph::kDecoder).
+enum class MixerType { kHcs, kHcm, kHcl, kAttention, kWindowAttention, kGatedLinear, kGatedDelta };
+
+// Which block graph a model runs through: StripedHyena2 (BF16 residual, RoPE / Hyena mixers, gated MLP,
+// tied head) or the decoder graph (F32 residual, a mixer and an optional feed-forward per block, each
+// with its own sizes, learned positions, own head).
+enum class BlockGraph { kStripedHyena2, kDecoder };
 
 // Operator classes reported by the optional per-operator timing.
 enum ProfileCategory : int {
@@ -34,6 +40,8 @@ enum ProfileCategory : int {
   kCatElementwise,     // embedding, gates, splits
   kCatRowQuantize,     // per-row E4M3 quantisation in front of the FP8 FFN / output projections
   kCatGemmFp8Ffn,      // tcgen05 E4M3 output and MLP projections (profile b200-fp8)
+  kCatRecurrence,      // gated linear attention and gated delta rule: preparation, recurrence, output norm and gate
+  kCatPolyNorm,        // normalised polynomial activation of a decoder's feed-forward
   kProfileCategories
 };
 const char *profile_category_name(int category);
@@ -75,7 +83,43 @@ struct DumpPlan {
 // F32 accumulation (its own execution profile, tolerance parity).
 // kTensorCoreFfn additionally runs the output and MLP projections of prefill
 // chunks in E4M3 with dynamic per-row activation scales (profile "b200-fp8").
-enum class ExecutionProfile { kExact, kTensorCore, kTensorCoreFfn };
+// kFloat32 (decoder graphs only) keeps every activation and cache in F32 and multiplies in F32.
+enum class ExecutionProfile { kExact, kTensorCore, kTensorCoreFfn, kFloat32 };
+
+// One block of a decoder graph.  Sizes are per head; what a mixer does not have stays 0.
+struct DecoderBlock {
+  MixerType mixer = MixerType::kWindowAttention;
+  std::size_t heads = 0, kv_heads = 0, dim = 0, value_dim = 0;
+  // kWindowAttention: row i sees key j <= i with i - j < window or j < keep_first
+  std::size_t window = 0, keep_first = 0;
+  float scale = 1.0F, softcap = 0.0F;
+  std::size_t conv_taps = 0;             // kGatedDelta
+  std::size_t decay_rank = 0;            // kGatedLinear: width of the bottleneck in front of the decays
+  float tau = 1.0F;                      // kGatedLinear
+  std::size_t inner_width = 0;           // feed-forward, 0: none
+
+  // Columns of the fused input projection [queries | keys | values | output gate | beta or decay
+  // bottleneck | decay]; every segment starts at a multiple of eight columns (zero weight rows between).
+  std::size_t query_width() const { return mixer == MixerType::kGatedDelta ? kv_heads * dim : heads * dim; }
+  std::size_t key_width() const { return kv_heads * dim; }
+  std::size_t value_width() const {
+    return mixer == MixerType::kWindowAttention ? kv_heads * value_dim : heads * value_dim;
+  }
+  std::size_t gate_width() const { return mixer == MixerType::kWindowAttention ? heads : heads * value_dim; }
+  static std::size_t padded(const std::size_t columns) { return (columns + 7) / 8 * 8; }
+  std::size_t key_column() const { return padded(query_width()); }
+  std::size_t value_column() const { return key_column() + padded(key_width()); }
+  std::size_t gate_column() const { return value_column() + padded(value_width()); }
+  std::size_t beta_column() const { return gate_column() + padded(gate_width()); }
+  std::size_t beta_width() const {
+    return mixer == MixerType::kGatedDelta ? heads : mixer == MixerType::kGatedLinear ? decay_rank : 0;
+  }
+  std::size_t decay_column() const { return beta_column() + padded(beta_width()); }
+  std::size_t projection_width() const {
+    return decay_column() + (mixer == MixerType::kGatedDelta ? padded(heads) : 0);
+  }
+  std::size_t output_width() const { return heads * value_dim; }
+};
 
 struct ModelConfig {
   std::string architecture, model_id, model_name, artifact_profile;
@@ -86,10 +130,18 @@ struct ModelConfig {
   float epsilon = 1e-6F, rope_scale = 1.0F, rope_base = 10000.0F;
   bool fp8_projection = false, hcm_filter_f32 = false, qkv_source_head_major = false;
   std::vector<MixerType> mixers;  // one per block
+  BlockGraph graph = BlockGraph::kStripedHyena2;
+  std::vector<DecoderBlock> blocks;  // decoder graphs: one per block
+  bool decoder() const { return graph == BlockGraph::kDecoder; }
+  // bytes of one residual element
+  std::size_t hidden_bytes() const { return decoder() ? sizeof(float) : 2; }
   std::size_t head_dim() const { return width / heads; }
 };
 
+// Picks the design by the architecture that the file names (config.json, else the typed metadata).
 int read_model_config(const ModelFile &file, bool allow_test_fixture, ModelConfig *config);
+// gigusun.cpp: the reader of a Gigusun config.json (sizes of the decay bottlenecks come from the tensors).
+int read_gigusun_config(const ModelFile &file, ModelConfig *config);
 // Every tensor the configuration calls for is there with its type and shape, and nothing else is
 // (host only; load_weights makes the same checks while it gathers the views).
 int check_tensor_set(const ModelFile &file, const ModelConfig &config);
@@ -108,6 +160,15 @@ struct LayerWeights {
   const void *l1 = nullptr, *l2 = nullptr, *l3 = nullptr;
   const void *l12 = nullptr;  // row-interleaved [2I, D] for the fused gate GEMM
   std::size_t payload_bytes = 0;
+  // ---- decoder blocks.  pre_norm / post_norm hold the whole gain (one plus the stored weight),
+  // projection the fused input projection (DecoderBlock), l1 / l3 the feed-forward's up and down weights.
+  const float *query_norm = nullptr, *key_norm = nullptr;  // [dim]
+  const float *distance_bias = nullptr;                    // [heads, max_seqlen]
+  const float *conv = nullptr;                             // [gate_column, conv_taps], by projection column
+  const float *decay_rate = nullptr, *decay_shift = nullptr;  // delta: -exp(A_log), dt_bias [heads]
+  const float *decay_weight = nullptr, *decay_bias = nullptr; // linear: [decay_rank, heads * dim], [heads * dim]
+  const float *output_norm = nullptr;                      // [value_dim]
+  const float *activation = nullptr;                       // [4] coefficients of the polynomial activation
   // E4M3 copies for the FP8 FFN profile (StageWeights::ensure_fp8_ffn): codes in the
   // layout of the BF16 tensor, and 1 / (448 / max|w|) for the epilogue.
   const void *out_codes = nullptr, *l12_codes = nullptr, *l3_codes = nullptr;
@@ -121,6 +182,9 @@ struct StageWeights {
   std::vector<LayerWeights> layers;
   const void *embedding = nullptr;    // stage 0 (and the last slice of a per-process pipeline)
   const float *final_norm = nullptr;  // same
+  const void *head = nullptr;         // same; the embedding where the head is tied
+  const void *positions = nullptr;    // decoders: [max_seqlen, width] BF16
+  const float *embedding_norm = nullptr;  // decoders: gain of the norm behind the embedding
   void *slab = nullptr;
   std::size_t slab_bytes = 0, weight_bytes = 0;
   // Quantises the output / MLP projection weights of every block once (first
@@ -239,6 +303,15 @@ class Context {
   int run_stage(Stage &stage, std::size_t rows, Mode mode, long capture_layer,
                 std::vector<float> *captured, std::size_t window_begin = 0,
                 std::size_t window_position = 0, const DumpPlan *dumps = nullptr);
+  // decoder.cu: the decoder graph's counterparts - activation and cache memory of a stage, the
+  // embedding, the blocks (position = sequence position of the first row), the final norm and head.
+  int allocate_decoder_stage(Stage &stage);
+  int decoder_embed(Stage &stage, const std::uint32_t *device_tokens, std::size_t rows, std::size_t position);
+  int run_decoder_stage(Stage &stage, std::size_t rows, Mode mode, std::size_t position, long capture_layer,
+                        std::vector<float> *captured, const DumpPlan *dumps);
+  int decoder_head(Stage &stage, std::size_t rows);
+  int decoder_linear(Stage &stage, const void *input, const void *weight, std::size_t rows, std::size_t in_features,
+                     std::size_t out_features, void *output, float *output_f32, bool accumulate);
   // Taps of block `layer` of `stage` (dumps.cu-style helpers in model.cu).
   int dump_mixer_taps(Stage &stage, std::size_t local_layer, std::size_t rows, Mode mode,
                       const DumpPlan &dumps);

@@ -1,6 +1,7 @@
-// Model configuration, stage planning and weight upload.
+// Model configuration and stage planning.  read_model_config picks the design by the architecture the
+// file names; each design has its own reader.
 //
-// read_model_config follows upstream's metadata contract
+// read_striped_hyena_config follows upstream's metadata contract
 // (src/cuda/model.cu:517-870): typed config.* keys, semantic flags that must
 // equal the supported Evo 2 profile, projection / medium-filter dtype keys,
 // fixture permission.  One deliberate difference: a registered model id may
@@ -13,6 +14,7 @@
 
 #include "../common.cuh"
 #include "../ops_internal.hpp"
+#include "json.hpp"
 #include "model.hpp"
 
 namespace evob {
@@ -42,9 +44,40 @@ const KnownModel kKnownModels[] = {
 
 }  // namespace
 
-int read_model_config(const ModelFile &file, const bool allow_test_fixture,
-                      ModelConfig *config) {
+namespace {
+
+int read_striped_hyena_config(const ModelFile &file, bool allow_test_fixture, ModelConfig *config);
+
+// Designs that a config.json describes, by the architecture it names.  (StripedHyena2 artifacts carry
+// typed metadata inside the Safetensors file instead.)
+struct ConfiguredDesign {
+  const char *architecture;
+  int (*read)(const ModelFile &file, ModelConfig *config);
+};
+const ConfiguredDesign kConfiguredDesigns[] = {
+    {"Gigusun", read_gigusun_config},
+};
+
+}  // namespace
+
+int read_model_config(const ModelFile &file, const bool allow_test_fixture, ModelConfig *config) {
   if (config == nullptr) return fail(kInvalidArgument, "model config output is null");
+  if (const Json *root = file.configuration()) {
+    const Json *architecture = root->get("architecture");
+    if (architecture != nullptr && architecture->kind == Json::kString) {
+      for (const ConfiguredDesign &design : kConfiguredDesigns)
+        if (architecture->text == design.architecture) return design.read(file, config);
+      if (file.metadata("evo2.profile") == nullptr)
+        return fail(kUnsupported, "config.json names an unknown architecture: " + architecture->text);
+    }
+  }
+  return read_striped_hyena_config(file, allow_test_fixture, config);
+}
+
+namespace {
+
+int read_striped_hyena_config(const ModelFile &file, const bool allow_test_fixture,
+                              ModelConfig *config) {
   ModelConfig c;
   std::string abi;
   EVOB_TRY(file.get_string("evo2.profile", &c.artifact_profile));
@@ -196,6 +229,8 @@ int read_model_config(const ModelFile &file, const bool allow_test_fixture,
   *config = std::move(c);
   return kOk;
 }
+
+}  // namespace
 
 std::vector<std::pair<std::size_t, std::size_t>> plan_stages(
     const std::vector<std::size_t> &layer_bytes, const std::size_t stage_count,

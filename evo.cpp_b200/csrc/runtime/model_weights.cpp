@@ -15,23 +15,16 @@
 #include "../common.cuh"
 #include "../ops_internal.hpp"
 #include "model.hpp"
+#include "weights.hpp"
 
 namespace evob {
 namespace {
 
-constexpr std::size_t kAlign = 256;
-std::size_t aligned(const std::size_t bytes) { return (bytes + kAlign - 1) / kAlign * kAlign; }
-
-struct Expected {
-  std::string name;
-  TensorType type;
-  std::vector<std::size_t> shape;
-};
-
-std::vector<Expected> expected_block_tensors(const ModelConfig &c, const std::size_t layer) {
+std::vector<ExpectedTensor> expected_block_tensors(const ModelConfig &c, const std::size_t layer) {
+  if (c.decoder()) return gigusun_block_tensors(c, layer);
   const std::string p = "blocks." + std::to_string(layer) + ".";
   const std::size_t D = c.width, I = c.inner_width;
-  std::vector<Expected> list;
+  std::vector<ExpectedTensor> list;
   list.push_back({p + "pre_norm.scale", TensorType::kF32, {D}});
   const MixerType type = c.mixers[layer];
   if (type == MixerType::kAttention) {
@@ -68,50 +61,35 @@ std::vector<Expected> expected_block_tensors(const ModelConfig &c, const std::si
   return list;
 }
 
-int lookup(const ModelFile &file, const Expected &e, const TensorView **out) {
-  const TensorView *tensor = file.find(e.name);
-  if (tensor == nullptr) return fail(kModelFormat, "required tensor is missing: " + e.name);
-  if (tensor->type != e.type || tensor->shape != e.shape)
-    return fail(kModelFormat, "tensor has an unexpected dtype or shape: " + e.name);
-  *out = tensor;
-  return kOk;
-}
-
 bool gate_fusable(const ModelConfig &c) {
   return c.inner_width % 128 == 0 && c.width % 8 == 0 && c.width >= 64;
 }
 
-// Cursor over a stage slab.
-struct Uploader {
-  unsigned char *base = nullptr;
-  std::size_t offset = 0;
-  cudaStream_t stream = nullptr;
-  bool dry_run = true;
+// Tensors outside the blocks.
+std::vector<ExpectedTensor> expected_model_tensors(const ModelConfig &c) {
+  if (c.decoder()) return gigusun_model_tensors(c);
+  return {{"embedding_layer.weight", TensorType::kBF16, {c.vocab, c.width}},
+          {"unembed.weight", TensorType::kBF16, {c.vocab, c.width}},
+          {"norm.scale", TensorType::kF32, {c.width}}};
+}
 
-  void *place(const std::size_t bytes) {
-    void *p = dry_run ? nullptr : base + offset;
-    offset += aligned(bytes);
-    return p;
-  }
-  int copy(void *dst, const void *src, const std::size_t bytes) {
-    if (dry_run || bytes == 0) return kOk;
-    if (cudaMemcpyAsync(dst, src, bytes, cudaMemcpyHostToDevice, stream) != cudaSuccess)
-      return fail(kCuda, "weight upload failed");
-    return kOk;
-  }
-  int tensor(const TensorView &t, const void **out) {
-    void *dst = place(t.bytes);
-    *out = dst;
-    return copy(dst, t.data, t.bytes);
-  }
-};
+int upload_model_tensors(const ModelFile &file, const ModelConfig &c, WeightUploader *up, StageWeights *stage) {
+  if (c.decoder()) return upload_gigusun_model(file, c, up, stage);
+  const void *p = nullptr;
+  int status = up->tensor(*file.find("embedding_layer.weight"), &stage->embedding);
+  if (status == kOk) status = up->tensor(*file.find("norm.scale"), &p);
+  stage->final_norm = static_cast<const float *>(p);
+  stage->head = stage->embedding;  // tied
+  return status;
+}
 
 int upload_layer(const ModelFile &file, const ModelConfig &c, const std::size_t layer,
-                 Uploader *up, LayerWeights *w, std::vector<unsigned char> *host_scratch) {
-  const std::vector<Expected> expected = expected_block_tensors(c, layer);
+                 WeightUploader *up, LayerWeights *w, std::vector<unsigned char> *host_scratch) {
+  if (c.decoder()) return upload_gigusun_block(file, c, layer, up, w);
+  const std::vector<ExpectedTensor> expected = expected_block_tensors(c, layer);
   std::vector<const TensorView *> t(expected.size());
   for (std::size_t i = 0; i < expected.size(); ++i) {
-    const int status = lookup(file, expected[i], &t[i]);
+    const int status = lookup_tensor(file, expected[i], &t[i]);
     if (status != kOk) return status;
     w->payload_bytes += t[i]->bytes;
   }
@@ -231,7 +209,7 @@ int StageWeights::ensure_fp8_ffn(const ModelConfig &c) {
     ~Restore() { cudaSetDevice(device); }
   } restore{previous};
   if (cudaSetDevice(device) != cudaSuccess) return fail(kCuda, "cannot select the stage's device");
-  const std::size_t per_layer = aligned(D * D) + aligned(2 * I * D) + aligned(D * I);
+  const std::size_t per_layer = weight_aligned(D * D) + weight_aligned(2 * I * D) + weight_aligned(D * I);
   void *slab_memory = nullptr;
   if (cudaMalloc(&slab_memory, per_layer * layers.size() + 256) != cudaSuccess)
     return fail(kCuda, "cannot allocate " + std::to_string((per_layer * layers.size()) >> 20) +
@@ -258,7 +236,7 @@ int StageWeights::ensure_fp8_ffn(const ModelConfig &c) {
     status = quantize_bf16(source, elements, quant, cursor, nullptr, stream);
     *codes = cursor;
     *dequant = 1.0F / quant;
-    cursor += aligned(elements);
+    cursor += weight_aligned(elements);
   };
   for (LayerWeights &w : layers) {
     convert(w.out_weight, D * D, &w.out_codes, &w.out_dequant);
@@ -279,24 +257,31 @@ int StageWeights::ensure_fp8_ffn(const ModelConfig &c) {
   return kOk;
 }
 
-int check_tensor_set(const ModelFile &file, const ModelConfig &c) {
-  std::set<std::string> expected_names = {"embedding_layer.weight", "unembed.weight", "norm.scale"};
+// Every tensor the configuration calls for with its type and shape; artifacts of the runtime profile hold
+// nothing else (a design with a config.json may carry tensors of its own beside them: they are not read).
+// layer_bytes (optional) receives the payload of every block.
+static int check_tensors(const ModelFile &file, const ModelConfig &c, std::vector<std::size_t> *layer_bytes) {
+  std::set<std::string> expected_names;
   const TensorView *view = nullptr;
   int status;
-  if ((status = lookup(file, {"embedding_layer.weight", TensorType::kBF16, {c.vocab, c.width}}, &view)) != kOk ||
-      (status = lookup(file, {"unembed.weight", TensorType::kBF16, {c.vocab, c.width}}, &view)) != kOk ||
-      (status = lookup(file, {"norm.scale", TensorType::kF32, {c.width}}, &view)) != kOk)
-    return status;
+  for (const ExpectedTensor &e : expected_model_tensors(c)) {
+    if ((status = lookup_tensor(file, e, &view)) != kOk) return status;
+    expected_names.insert(e.name);
+  }
   for (std::size_t layer = 0; layer < c.layers; ++layer)
-    for (const Expected &e : expected_block_tensors(c, layer)) {
-      if ((status = lookup(file, e, &view)) != kOk) return status;
+    for (const ExpectedTensor &e : expected_block_tensors(c, layer)) {
+      if ((status = lookup_tensor(file, e, &view)) != kOk) return status;
       expected_names.insert(e.name);
+      if (layer_bytes != nullptr && layer < layer_bytes->size()) (*layer_bytes)[layer] += view->bytes;
     }
+  if (c.decoder()) return kOk;
   for (const TensorView &tensor : file.tensors())
     if (expected_names.count(tensor.name) == 0)
       return fail(kModelFormat, "unknown tensor for model profile '" + c.model_id + "': " + tensor.name);
   return kOk;
 }
+
+int check_tensor_set(const ModelFile &file, const ModelConfig &c) { return check_tensors(file, c, nullptr); }
 
 int load_weights(const ModelFile &file, const std::vector<int> &devices,
                  const bool allow_test_fixture, const std::size_t layer_limit,
@@ -328,24 +313,10 @@ int load_weights(const ModelFile &file, const std::vector<int> &devices,
   if (layers > c.layers || layers < stage_count)
     return fail(kInvalidArgument, "CUDA layer limit must cover at least one layer per device");
 
-  // exact tensor set
-  std::set<std::string> expected_names = {"embedding_layer.weight", "unembed.weight", "norm.scale"};
-  const TensorView *embedding = nullptr, *unembed = nullptr, *norm = nullptr;
-  if ((status = lookup(file, {"embedding_layer.weight", TensorType::kBF16, {c.vocab, c.width}}, &embedding)) != kOk ||
-      (status = lookup(file, {"unembed.weight", TensorType::kBF16, {c.vocab, c.width}}, &unembed)) != kOk ||
-      (status = lookup(file, {"norm.scale", TensorType::kF32, {c.width}}, &norm)) != kOk)
-    return status;
+  if (c.decoder() && sliced)
+    return fail(kUnsupported, "decoder graphs run whole in one process: pipeline slices are not available");
   std::vector<std::size_t> layer_bytes(layers, 0);
-  for (std::size_t layer = 0; layer < c.layers; ++layer)
-    for (const Expected &e : expected_block_tensors(c, layer)) {
-      const TensorView *view = nullptr;
-      if ((status = lookup(file, e, &view)) != kOk) return status;
-      expected_names.insert(e.name);
-      if (layer < layers) layer_bytes[layer] += view->bytes;
-    }
-  for (const TensorView &view : file.tensors())
-    if (expected_names.count(view.name) == 0)
-      return fail(kModelFormat, "unknown tensor for model profile '" + c.model_id + "': " + view.name);
+  if ((status = check_tensors(file, c, &layer_bytes)) != kOk) return status;
 
   // Upstream's byte-balanced split serves its limit of four devices.  Beyond it a stage holds
   // only a few blocks, and a greedy byte target then leaves one stage a block more than its
@@ -368,7 +339,7 @@ int load_weights(const ModelFile &file, const std::vector<int> &devices,
     stage->layer_end = plan[s].second;
     stage->layers.resize(stage->layer_end - stage->layer_begin);
     for (int pass = 0; pass < 2 && status == kOk; ++pass) {
-      Uploader up;
+      WeightUploader up;
       up.dry_run = pass == 0;
       if (pass == 1) {
         if (cudaSetDevice(stage->device) != cudaSuccess ||
@@ -385,10 +356,8 @@ int load_weights(const ModelFile &file, const std::vector<int> &devices,
         }
       }
       if (holds_embedding) {
-        const void *p = nullptr;
-        status = up.tensor(*embedding, &stage->embedding);
-        if (status == kOk) status = up.tensor(*norm, &p);
-        stage->final_norm = static_cast<const float *>(p);
+        StageWeights scratch_stage;
+        status = upload_model_tensors(file, c, &up, pass == 1 ? stage.get() : &scratch_stage);
       }
       for (std::size_t layer = stage->layer_begin; layer < stage->layer_end && status == kOk; ++layer) {
         LayerWeights scratch_weights;
@@ -403,7 +372,8 @@ int load_weights(const ModelFile &file, const std::vector<int> &devices,
         cudaStreamDestroy(up.stream);
       }
     }
-    stage->weight_bytes = (holds_embedding ? embedding->bytes + unembed->bytes + norm->bytes : 0);
+    if (holds_embedding)
+      for (const ExpectedTensor &e : expected_model_tensors(c)) stage->weight_bytes += file.find(e.name)->bytes;
     for (const LayerWeights &w : stage->layers) stage->weight_bytes += w.payload_bytes;
     weights->stages.push_back(std::move(stage));
   }

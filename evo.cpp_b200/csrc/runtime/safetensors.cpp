@@ -11,151 +11,10 @@
 #include <sstream>
 
 #include "../common.cuh"
+#include "json.hpp"
 
 namespace evob {
 namespace {
-
-// ---- a small JSON reader (objects, arrays, strings, integers, literals)
-struct Json {
-  enum Kind { kNull, kBool, kNumber, kString, kArray, kObject } kind = kNull;
-  bool boolean = false;
-  double number = 0;
-  std::string text;
-  std::vector<Json> items;
-  std::vector<std::pair<std::string, Json>> members;  // insertion order
-  const Json *get(const std::string &key) const {
-    for (const auto &m : members)
-      if (m.first == key) return &m.second;
-    return nullptr;
-  }
-};
-
-class JsonParser {
- public:
-  JsonParser(const char *begin, const char *end) : p_(begin), end_(end) {}
-  bool parse(Json *out) {
-    skip();
-    if (!value(out, 0)) return false;
-    skip();
-    return p_ == end_;
-  }
-
- private:
-  const char *p_, *end_;
-  void skip() {
-    while (p_ < end_ && (*p_ == ' ' || *p_ == '\n' || *p_ == '\t' || *p_ == '\r')) ++p_;
-  }
-  bool literal(const char *word) {
-    const std::size_t n = std::strlen(word);
-    if (static_cast<std::size_t>(end_ - p_) < n || std::memcmp(p_, word, n) != 0) return false;
-    p_ += n;
-    return true;
-  }
-  bool string(std::string *out) {
-    if (p_ >= end_ || *p_ != '"') return false;
-    ++p_;
-    out->clear();
-    while (p_ < end_ && *p_ != '"') {
-      if (*p_ == '\\') {
-        if (++p_ >= end_) return false;
-        switch (*p_) {
-          case '"': out->push_back('"'); break;
-          case '\\': out->push_back('\\'); break;
-          case '/': out->push_back('/'); break;
-          case 'b': out->push_back('\b'); break;
-          case 'f': out->push_back('\f'); break;
-          case 'n': out->push_back('\n'); break;
-          case 'r': out->push_back('\r'); break;
-          case 't': out->push_back('\t'); break;
-          case 'u': {
-            if (end_ - p_ < 5) return false;
-            unsigned code = 0;
-            for (int i = 1; i <= 4; ++i) {
-              const char c = p_[i];
-              code <<= 4;
-              if (c >= '0' && c <= '9') code |= c - '0';
-              else if (c >= 'a' && c <= 'f') code |= c - 'a' + 10;
-              else if (c >= 'A' && c <= 'F') code |= c - 'A' + 10;
-              else return false;
-            }
-            p_ += 4;
-            if (code < 0x80) out->push_back(static_cast<char>(code));
-            else if (code < 0x800) {
-              out->push_back(static_cast<char>(0xc0 | (code >> 6)));
-              out->push_back(static_cast<char>(0x80 | (code & 0x3f)));
-            } else {
-              out->push_back(static_cast<char>(0xe0 | (code >> 12)));
-              out->push_back(static_cast<char>(0x80 | ((code >> 6) & 0x3f)));
-              out->push_back(static_cast<char>(0x80 | (code & 0x3f)));
-            }
-            break;
-          }
-          default: return false;
-        }
-        ++p_;
-      } else {
-        out->push_back(*p_++);
-      }
-    }
-    if (p_ >= end_) return false;
-    ++p_;
-    return true;
-  }
-  bool value(Json *out, const int depth) {
-    if (depth > 16 || p_ >= end_) return false;
-    if (*p_ == '{') {
-      out->kind = Json::kObject;
-      ++p_;
-      skip();
-      if (p_ < end_ && *p_ == '}') { ++p_; return true; }
-      for (;;) {
-        std::string key;
-        skip();
-        if (!string(&key)) return false;
-        skip();
-        if (p_ >= end_ || *p_ != ':') return false;
-        ++p_;
-        skip();
-        Json member;
-        if (!value(&member, depth + 1)) return false;
-        out->members.emplace_back(std::move(key), std::move(member));
-        skip();
-        if (p_ < end_ && *p_ == ',') { ++p_; continue; }
-        if (p_ < end_ && *p_ == '}') { ++p_; return true; }
-        return false;
-      }
-    }
-    if (*p_ == '[') {
-      out->kind = Json::kArray;
-      ++p_;
-      skip();
-      if (p_ < end_ && *p_ == ']') { ++p_; return true; }
-      for (;;) {
-        Json item;
-        skip();
-        if (!value(&item, depth + 1)) return false;
-        out->items.push_back(std::move(item));
-        skip();
-        if (p_ < end_ && *p_ == ',') { ++p_; continue; }
-        if (p_ < end_ && *p_ == ']') { ++p_; return true; }
-        return false;
-      }
-    }
-    if (*p_ == '"') {
-      out->kind = Json::kString;
-      return string(&out->text);
-    }
-    if (literal("true")) { out->kind = Json::kBool; out->boolean = true; return true; }
-    if (literal("false")) { out->kind = Json::kBool; return true; }
-    if (literal("null")) { out->kind = Json::kNull; return true; }
-    const char *start = p_;
-    while (p_ < end_ && (std::strchr("+-0123456789.eE", *p_) != nullptr)) ++p_;
-    if (p_ == start) return false;
-    out->kind = Json::kNumber;
-    out->number = std::strtod(std::string(start, p_).c_str(), nullptr);
-    return true;
-  }
-};
 
 bool ends_with(const std::string &s, const std::string &suffix) {
   return s.size() >= suffix.size() &&
@@ -195,7 +54,8 @@ int ModelFile::open_shard(const std::string &path, const bool first) {
   const auto *bytes = static_cast<const unsigned char *>(address);
   std::uint64_t header_length = 0;
   for (int i = 0; i < 8; ++i) header_length |= static_cast<std::uint64_t>(bytes[i]) << (8 * i);
-  if (header_length == 0 || header_length > length - 8 || header_length % 8 != 0 ||
+  // (designs with a config.json take any Safetensors writer's header; artifacts of the runtime profile are padded)
+  if (header_length == 0 || header_length > length - 8 || (header_length % 8 != 0 && configuration_ == nullptr) ||
       header_length > (1ULL << 28))
     return fail(kModelFormat, "Safetensors header length is invalid: " + path);
   Json header;
@@ -232,6 +92,7 @@ int ModelFile::open_shard(const std::string &path, const bool first) {
     if (dtype->text == "F32") { entry.view.type = TensorType::kF32; element = 4; }
     else if (dtype->text == "BF16") { entry.view.type = TensorType::kBF16; element = 2; }
     else if (dtype->text == "F8_E4M3") { entry.view.type = TensorType::kE4M3; element = 1; }
+    else if (dtype->text == "I32") { entry.view.type = TensorType::kI32; element = 4; }
     else return fail(kModelFormat, "unsupported tensor dtype " + dtype->text + ": " + name);
     if (shape->items.empty() || shape->items.size() > 8)
       return fail(kModelFormat, "tensor rank is unsupported: " + name);
@@ -281,6 +142,17 @@ int ModelFile::open(const std::string &path, std::shared_ptr<ModelFile> *out) {
   std::string index_path;
   if (is_directory(path)) {
     struct stat st;
+    if (stat((path + "/config.json").c_str(), &st) == 0) {
+      std::ifstream stream(path + "/config.json");
+      std::stringstream buffer;
+      buffer << stream.rdbuf();
+      const std::string text = buffer.str();
+      auto configuration = std::make_shared<Json>();
+      if (!stream || !JsonParser(text.data(), text.data() + text.size()).parse(configuration.get()) ||
+          configuration->kind != Json::kObject)
+        return fail(kModelFormat, "config.json is not a JSON object: " + path);
+      file->configuration_ = std::move(configuration);
+    }
     if (stat((path + "/model.safetensors.index.json").c_str(), &st) == 0)
       index_path = path + "/model.safetensors.index.json";
     else {

@@ -3,7 +3,9 @@
 // Follows upstream's container contract (docs/model-format.md:31-127,
 // src/model_format.cpp): 8-byte little-endian header length, JSON header,
 // dense payload with contiguous non-overlapping tensors, dtypes F32 / BF16 /
-// F8_E4M3, typed string metadata with s:/u:/f:/b:/l:/x: prefixes.
+// F8_E4M3 / I32, typed string metadata with s:/u:/f:/b:/l:/x: prefixes.  A
+// directory may hold a config.json beside its tensors: designs that are
+// described by one (architecture, layers) are read from there.
 #pragma once
 
 #include <cstddef>
@@ -15,7 +17,9 @@
 
 namespace evob {
 
-enum class TensorType { kF32, kBF16, kE4M3 };
+struct Json;
+
+enum class TensorType { kF32, kBF16, kE4M3, kI32 };
 
 struct TensorView {
   std::string name;
@@ -43,6 +47,8 @@ class ModelFile {
   const std::vector<TensorView> &tensors() const { return tensors_; }
   const std::string *metadata(const std::string &key) const;
   std::size_t payload_bytes() const { return payload_bytes_; }
+  // The parsed config.json of a model directory (designs that are configured by one); null without it.
+  const Json *configuration() const { return configuration_.get(); }
 
   // Typed metadata accessors; missing key or wrong prefix -> kModelFormat.
   int get_string(const std::string &key, std::string *out) const;
@@ -62,6 +68,7 @@ class ModelFile {
   std::vector<TensorView> tensors_;
   std::map<std::string, std::size_t> index_;
   std::map<std::string, std::string> metadata_;
+  std::shared_ptr<const Json> configuration_;
   std::size_t payload_bytes_ = 0;
 };
 

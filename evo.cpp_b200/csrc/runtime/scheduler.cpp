@@ -55,14 +55,14 @@ struct Scheduler::Impl {
     const SchedulerRequest &request = work.request;
     const std::size_t vocab = context.config().vocab;
     const std::size_t chunk = context.activation_capacity();
-    const std::vector<std::uint8_t> &bytes = request.sequence;
+    const std::vector<std::uint32_t> &prompt = request.tokens;
     const bool score = request.kind == SchedulerRequest::Kind::kScore;
-    if (bytes.empty() || (score && bytes.size() < 2)) {
+    if (prompt.empty() || (score && prompt.size() < 2)) {
       result->status = kInvalidArgument;
       result->error = score ? "scoring needs at least two tokens" : "generation needs a prompt";
       return;
     }
-    if (bytes.size() + (score ? 0 : request.new_tokens) > context.context_capacity()) {
+    if (prompt.size() + (score ? 0 : request.new_tokens) > context.context_capacity()) {
       result->status = kInvalidArgument;
       result->error = "request exceeds the context capacity of " + std::to_string(context.context_capacity());
       return;
@@ -74,14 +74,14 @@ struct Scheduler::Impl {
     }
     std::vector<float> logits;
     std::vector<std::uint32_t> tokens;
-    for (std::size_t offset = 0; offset < bytes.size(); offset += chunk) {
+    for (std::size_t offset = 0; offset < prompt.size(); offset += chunk) {
       if (work.cancelled.load(std::memory_order_relaxed)) {
         result->cancelled = true;
         return;
       }
-      const std::size_t rows = std::min(chunk, bytes.size() - offset);
-      tokens.assign(bytes.begin() + static_cast<std::ptrdiff_t>(offset),
-                    bytes.begin() + static_cast<std::ptrdiff_t>(offset + rows));
+      const std::size_t rows = std::min(chunk, prompt.size() - offset);
+      tokens.assign(prompt.begin() + static_cast<std::ptrdiff_t>(offset),
+                    prompt.begin() + static_cast<std::ptrdiff_t>(offset + rows));
       const int status = offset == 0 ? context.prefill(tokens, &logits) : context.prefill_chunk(tokens, &logits);
       if (status != kOk) {
         result->status = status;
@@ -89,16 +89,16 @@ struct Scheduler::Impl {
         return;
       }
       if (score) {
-        // row r of this chunk predicts byte offset + r + 1
-        for (std::size_t r = 0; r < rows && offset + r + 1 < bytes.size(); ++r) {
-          const double value = log_probability(logits.data() + r * vocab, vocab, bytes[offset + r + 1]);
+        // row r of this chunk predicts token offset + r + 1
+        for (std::size_t r = 0; r < rows && offset + r + 1 < prompt.size(); ++r) {
+          const double value = log_probability(logits.data() + r * vocab, vocab, prompt[offset + r + 1]);
           result->token_log_likelihoods.push_back(value);
           result->log_likelihood += value;
         }
       }
     }
     if (score) {
-      result->scored_tokens = bytes.size() - 1;
+      result->scored_tokens = prompt.size() - 1;
       return;
     }
     Sampler sampler(request.sampling);
@@ -111,9 +111,10 @@ struct Scheduler::Impl {
       }
       std::uint32_t token = 0;
       int status = sampler.sample(last_row, vocab, &token);
-      if (status == kOk && token > 255) break;  // not a byte: generation ends (upstream token_to_byte)
+      if (status == kOk && request.byte_output && token > 255) break;  // not a byte: generation ends (upstream token_to_byte)
       if (status == kOk) {
-        result->generated.push_back(static_cast<std::uint8_t>(token));
+        result->generated_tokens.push_back(token);
+        if (request.byte_output) result->generated.push_back(static_cast<std::uint8_t>(token));
         if (produced + 1 == request.new_tokens) break;
         status = context.decode(token, &step);
       }

@@ -31,7 +31,8 @@ namespace evob {
 struct SchedulerRequest {
   enum class Kind { kScore, kGenerate };
   Kind kind = Kind::kScore;
-  std::vector<std::uint8_t> sequence;  // bytes to score, or the prompt
+  std::vector<std::uint32_t> tokens;   // ids to score, or the prompt
+  bool byte_output = true;             // generate: stop at the first id that is not a byte
   std::size_t new_tokens = 0;          // generate: tokens to sample after the prompt
   SamplingConfig sampling;
 };
@@ -43,7 +44,8 @@ struct SchedulerResult {
   double log_likelihood = 0.0;      // score: sum of next-token log-likelihoods
   std::size_t scored_tokens = 0;
   std::vector<double> token_log_likelihoods;
-  std::vector<std::uint8_t> generated;  // generate: sampled bytes (stops early at a token above 255)
+  std::vector<std::uint8_t> generated;  // generate: sampled bytes (byte_output; stops early at a token above 255)
+  std::vector<std::uint32_t> generated_tokens;  // generate: every sampled id
   double queue_seconds = 0.0, run_seconds = 0.0;
 };
 

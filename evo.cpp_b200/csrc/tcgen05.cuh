@@ -74,6 +74,16 @@ __device__ __forceinline__ void tma_load_2d(const std::uint32_t dst,
       "l"(map), "r"(bar), "r"(x), "r"(y)
       : "memory");
 }
+__device__ __forceinline__ void tma_load_3d(const std::uint32_t dst,
+                                            const CUtensorMap *const map,
+                                            const std::uint32_t bar,
+                                            const int x, const int y, const int z) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::"
+      "bytes [%0], [%1, {%3, %4, %5}], [%2];" ::"r"(dst),
+      "l"(map), "r"(bar), "r"(x), "r"(y), "r"(z)
+      : "memory");
+}
 __device__ __forceinline__ void tc_fence_before() {
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
 }
@@ -147,6 +157,10 @@ __device__ __forceinline__ std::uint64_t smem_descriptor(
 // 2-D BF16 tensor map over a row-major [rows, columns] matrix with boxes of
 // 64 columns (one 128-byte swizzle atom) x box_rows rows, SWIZZLE_128B.
 int make_bf16_tile_map(CUtensorMap *map, const void *base, std::size_t rows, std::size_t columns,
+                       int box_rows);
+// 3-D BF16 tensor map over [rows, heads, dim] with boxes of 64 dimensions x one head x box_rows rows,
+// SWIZZLE_128B: dimensions past the head's end read as zeros, not as the next head.
+int make_bf16_head_map(CUtensorMap *map, const void *base, std::size_t rows, std::size_t heads, std::size_t dim,
                        int box_rows);
 // Per-device sticky error word raised by a timed-out wait in any tcgen05
 // kernel (reported by gemm_error_state); also the device's SM count.

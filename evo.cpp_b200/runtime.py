@@ -17,6 +17,7 @@ CONTEXT_FLAG_FAST_Q8_KV = 1 << 0
 CONTEXT_FLAG_TENSORCORE_FP8 = 1 << 8
 CONTEXT_FLAG_FULL_ARENA = 1 << 9
 CONTEXT_FLAG_FP8_FFN = 1 << 10
+CONTEXT_FLAG_FLOAT32 = 1 << 11
 
 DUMP_POINTS = ("block_output", "pre_norm", "mixer_input_projection", "mixer_short_filter", "mixer_short_state",
                "mixer_inner_state", "mixer_x2", "mixer_x1", "mixer_value", "mixer_pregate", "mixer_state",
@@ -76,7 +77,8 @@ class SchedulerParams(ctypes.Structure):
 
 class Request(ctypes.Structure):
     _fields_ = [("struct_size", ctypes.c_size_t), ("kind", ctypes.c_int32), ("sequence", ctypes.c_char_p),
-                ("length", ctypes.c_size_t), ("new_tokens", ctypes.c_size_t), ("sampler", SamplerParams)]
+                ("length", ctypes.c_size_t), ("new_tokens", ctypes.c_size_t), ("sampler", SamplerParams),
+                ("tokens", ctypes.POINTER(ctypes.c_uint32)), ("token_count", ctypes.c_size_t)]
 
 
 class RequestResult(ctypes.Structure):
@@ -84,7 +86,8 @@ class RequestResult(ctypes.Structure):
                 ("cancelled", ctypes.c_int32), ("log_likelihood", ctypes.c_double), ("scored_tokens", ctypes.c_size_t),
                 ("token_log_likelihoods", ctypes.POINTER(ctypes.c_double)),
                 ("generated", ctypes.POINTER(ctypes.c_uint8)), ("generated_length", ctypes.c_size_t),
-                ("queue_seconds", ctypes.c_double), ("run_seconds", ctypes.c_double)]
+                ("queue_seconds", ctypes.c_double), ("run_seconds", ctypes.c_double),
+                ("generated_tokens", ctypes.POINTER(ctypes.c_uint32)), ("generated_token_count", ctypes.c_size_t)]
 
 
 class SchedulerMetrics(ctypes.Structure):
@@ -279,16 +282,23 @@ class Scheduler:
                      "log_likelihood": r.log_likelihood, "scored_tokens": r.scored_tokens,
                      "token_log_likelihoods": [r.token_log_likelihoods[i] for i in range(r.scored_tokens)],
                      "generated": bytes(r.generated[i] for i in range(r.generated_length)),
+                     "generated_tokens": [r.generated_tokens[i] for i in range(r.generated_token_count)],
                      "queue_seconds": r.queue_seconds, "run_seconds": r.run_seconds}
             with self._lock:
                 self.results[ticket] = entry
 
         self._callback = on_done
 
-    def _submit(self, kind: int, payload: bytes, new_tokens: int = 0, **sampler) -> int:
+    def _submit(self, kind: int, payload, new_tokens: int = 0, **sampler) -> int:
+        """payload: bytes, or a sequence of token ids."""
         request = Request()
         request.struct_size = ctypes.sizeof(Request)
-        request.kind, request.sequence, request.length, request.new_tokens = kind, payload, len(payload), new_tokens
+        request.kind, request.new_tokens = kind, new_tokens
+        if isinstance(payload, bytes):
+            request.sequence, request.length = payload, len(payload)
+        else:
+            ids = (ctypes.c_uint32 * max(1, len(payload)))(*payload)
+            request.tokens, request.token_count = ids, len(payload)
         request.sampler = self.library.lib.evo_sampler_default_params()
         for name, value in sampler.items():
             setattr(request.sampler, name, value)
@@ -303,6 +313,12 @@ class Scheduler:
 
     def generate(self, prompt: bytes, tokens: int, **sampler) -> int:
         return self._submit(1, bytes(prompt), tokens, **sampler)
+
+    def score_tokens(self, tokens) -> int:
+        return self._submit(0, list(tokens))
+
+    def generate_tokens(self, prompt, tokens: int, **sampler) -> int:
+        return self._submit(1, list(prompt), tokens, **sampler)
 
     def cancel(self, ticket: int) -> bool:
         return bool(self.library.lib.evo_b200_scheduler_cancel(self.handle, ticket))

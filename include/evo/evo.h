@@ -74,7 +74,10 @@ enum {
    * this is new arithmetic under its own name, with tolerance parity against
    * "exact" (upstream's rule for approximate profiles:
    * docs/execution-profiles.md:77-82).  Implies the tensor-core projections. */
-  EVO_CONTEXT_FLAG_B200_FP8_FFN = 1u << 10u
+  EVO_CONTEXT_FLAG_B200_FP8_FFN = 1u << 10u,
+  /* Profile "float32": every activation, cache and product in F32 (weights keep their stored values).
+   * Decoder models (config.json) only; other models refuse it with EVO_STATUS_UNSUPPORTED. */
+  EVO_CONTEXT_FLAG_B200_FLOAT32 = 1u << 11u
 };
 
 typedef struct evo_model evo_model;

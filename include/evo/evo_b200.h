@@ -25,7 +25,7 @@ typedef struct evo_b200_stage_info {
 
 /* Enqueues one prefill of `rows` token ids that already live on the device of
  * pipeline stage 0 (uint32, rows <= activation capacity) on the context's
- * stream and returns without waiting.  BF16 logits [rows, vocab] stay on the
+ * stream and returns without waiting.  BF16 logits [rows, vocab] (F32 for decoder models) stay on the
  * device; *device_logits_out (optional) receives their address.  stateless != 0
  * keeps no caches (position stays 0); otherwise the context is left ready for
  * decode.  Call evo_b200_context_synchronize before reading results. */
@@ -72,7 +72,9 @@ EVO_API size_t evo_b200_context_activation_capacity(const evo_context *context);
  * the same refusals (a synthetic fixture needs allow_test_fixture; precision metadata that disagrees
  * with the configuration, an unsupported projection dtype and tensors outside the profile's exact set
  * are rejected here, before any device work).  mixer_types (optional) receives one code per block -
- * 0 HCS, 1 HCM, 2 HCL, 3 attention - up to mixer_capacity.  The three names are NUL-terminated and cut
+ * 0 HCS, 1 HCM, 2 HCL, 3 attention; decoder blocks 4 window attention, 5 gated linear attention,
+ * 6 gated delta rule - up to mixer_capacity.  Models described by a config.json (a directory path) report
+ * the largest head count, state size and inner width of their blocks.  The three names are NUL-terminated and cut
  * at 63 bytes. */
 typedef struct evo_b200_model_config {
   size_t struct_size;
@@ -269,6 +271,11 @@ typedef struct evo_b200_request {
   size_t length;
   size_t new_tokens;          /* generate only */
   evo_sampler_params sampler; /* generate only */
+  /* Token ids instead of bytes (used when not null; `sequence` is then ignored).  Generation from token
+   * ids may produce any id of the vocabulary; from bytes it stops at the first id above 255.  Callers
+   * with the struct_size of an earlier header keep the byte form. */
+  const uint32_t *tokens;
+  size_t token_count;
 } evo_b200_request;
 typedef struct evo_b200_request_result {
   size_t struct_size;
@@ -282,6 +289,8 @@ typedef struct evo_b200_request_result {
   size_t generated_length;
   double queue_seconds;
   double run_seconds;
+  const uint32_t *generated_tokens; /* every sampled id, also those of `generated` */
+  size_t generated_token_count;
 } evo_b200_request_result;
 typedef void (*evo_b200_request_callback)(uint64_t ticket, const evo_b200_request_result *result,
                                           void *user_data);
