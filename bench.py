@@ -874,13 +874,24 @@ def main() -> None:
                         help="do not also time the opt-in b200-fp8 profile")
     parser.add_argument("--decode-tokens", type=int, default=64,
                         help="cached-decode steps timed after a 1,024-token prompt (0 disables)")
+    parser.add_argument("--design", default=None, choices=["gigusun"],
+                        help="instead of the headline workload: a decoder of this design beside a StripedHyena2 stack "
+                             "of equal width, block count and weights (prefill, decode, operator classes)")
+    parser.add_argument("--design-widths", default="2048,4096", help="model widths of --design")
     args = parser.parse_args()
     select_model(args.model)
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
-    if args.impl == "reference":
+    if args.design is not None:
+        import importlib
+
+        package = load_package()
+        bench = importlib.import_module("evo_cpp_b200.decoder_bench")
+        print(json.dumps(bench.run(package, ClockSampler, args.steps, max(args.warmup, 3), [1024, 8192],
+                                   [int(w) for w in args.design_widths.split(",")], args.decode_tokens)))
+    elif args.impl == "reference":
         run_reference(args, rank, world)
     elif world > 1 and args.multi_gpu == "pipeline":
         run_pipeline(args, rank, world, local_rank)

@@ -65,8 +65,51 @@ OPS_SIGNATURES: dict[str, list] = {
     "evo_b200_q8_kv_expand": [_P, _P, _P, _P, _Z, _Z, _Z, _Z, _P, _P, _P],
     "evo_b200_q8_attention_decode": [_P, _P, _P, _P, _P, _Z, _Z, _Z, _Z, _Z, _P, _P],
 }
+# operators of decoder graphs
+OPS_SIGNATURES.update({
+    "evo_b200_embed_positions": [_P, _P, _P, _P, _Z, _Z, _Z, _Z, _F, _P, _P],
+    "evo_b200_rms_norm_residual": [_P, _P, _Z, _Z, _F, _I, _P, _P],
+    "evo_b200_poly_norm": [_P, _P, _Z, _Z, _F, _I, _P, _P],
+    "evo_b200_distance_bias_table": [_P, _P, _Z, _Z, _P, _P],
+    "evo_b200_f32_linear": [_P, _P, _Z, _Z, _Z, _I, _P, _P],
+    "evo_b200_bf16_linear_f32_result": [_P, _P, _Z, _Z, _Z, _I, _P, _Z, _P, _P],
+    "evo_b200_head_norm_append": [_P, _P],
+    "evo_b200_window_attention": [_P, _P],
+    "evo_b200_recurrent_mixer": [_P, _P],
+})
+
+
+def _fields(text: str) -> list[tuple[str, type]]:
+    """"p a b|z c|f d|i e" -> ctypes fields (pointer, size_t, float, int32) in order."""
+    kinds = {"p": _P, "z": _Z, "f": _F, "i": ctypes.c_int32}
+    return [(name, kinds[group.split()[0]]) for group in text.split("|") for name in group.split()[1:]]
+
+
+class _Arguments(ctypes.Structure):
+    def __init__(self, **values):
+        super().__init__(struct_size=ctypes.sizeof(self), **values)
+
+
+class HeadNorm(_Arguments):
+    _fields_ = _fields("z struct_size|p projection|z stride key_column value_column|p query_gain key_gain query "
+                       "key_cache value_cache|z rows position capacity heads kv_heads dim value_dim|f epsilon|i float32")
+
+
+class WindowAttention(_Arguments):
+    _fields_ = _fields("z struct_size|p query key_cache value_cache gate|z gate_stride|p distance_bias|z bias_stride|"
+                       "p output|z rows position capacity heads kv_heads dim value_dim window keep_first|"
+                       "f scale softcap|i sink float32 kernel")
+
+
+class Recurrent(_Arguments):
+    _fields_ = _fields("z struct_size|i delta|p projection|z stride key_column value_column gate_column beta_column "
+                       "decay_column rows heads kv_heads dim value_dim|p conv|z conv_taps|p conv_history decay_rate "
+                       "decay_shift decay_weight decay_bias|z decay_rank|f tau|p output_norm|f epsilon|p state|i fresh|"
+                       "p workspace output|i float32")
+
+
 # entry points that do not return a status
-OPS_OTHER = ("evo_b200_last_error", "evo_b200_hcl_scratch_floats", "evo_b200_linear_executor_free",
+OPS_OTHER = ("evo_b200_last_error", "evo_b200_recurrent_workspace_bytes", "evo_b200_hcl_scratch_floats", "evo_b200_linear_executor_free",
              "evo_b200_linear_executor_name", "evo_b200_linear_executor_cached_bytes",
              "evo_b200_e4m3_encode", "evo_b200_e4m3_decode", "evo_b200_e4m3_scaled_roundtrip")
 
@@ -87,6 +130,8 @@ class Ops:
                 "(there is no CPU fallback)")
         self.lib = ctypes.CDLL(str(path))
         self.lib.evo_b200_last_error.restype = ctypes.c_char_p
+        self.lib.evo_b200_recurrent_workspace_bytes.restype = _Z
+        self.lib.evo_b200_recurrent_workspace_bytes.argtypes = [_I, _Z, _Z, _Z, _Z, _Z, _I]
         self.lib.evo_b200_hcl_scratch_floats.restype = _Z
         self.lib.evo_b200_hcl_scratch_floats.argtypes = [_Z, _Z, _Z]
         self.lib.evo_b200_linear_executor_free.restype = None

@@ -290,3 +290,107 @@ def write_model(path: Path, metadata: dict[str, str], tensors: Iterable[tuple[st
 def write_synthetic(path: Path, spec: dict, seed: int, **kwargs) -> list[Path]:
     shard = kwargs.pop("max_shard_bytes", 4 << 30)
     return write_model(path, spec["metadata"], synthetic_tensors(spec, seed, **kwargs), max_shard_bytes=shard)
+
+
+# ---- Gigusun decoders: a directory with config.json and model.safetensors
+def gigusun_config(layers: list[dict], *, vocab: int, width: int, max_positions: int, eps: float = 1e-6) -> dict:
+    return {"architecture": "Gigusun", "vocab": vocab, "width": width, "max_positions": max_positions,
+            "norm": {"eps": eps}, "layers": layers}
+
+
+def gigusun_manifest(config: dict, decay_rank: int = 16) -> list[tuple[str, tuple[int, ...]]]:
+    """(tensor name, shape) of a configuration, in file order."""
+    D = config["width"]
+    rows = [("embed", (config["vocab"], D)), ("pos", (config["max_positions"], D)), ("embed.norm", (D,))]
+    for i, layer in enumerate(config["layers"]):
+        m, p = layer["mixer"], f"l{i}.mix."
+        H, dim, vdim = m["heads"], m["dim"], m["vdim"]
+        G = m.get("kv_heads", H)
+        rows.append((f"l{i}.norm1", (D,)))
+        if layer["type"] == "attention":
+            rows += [(p + "q", (H * dim, D)), (p + "k", (G * dim, D)), (p + "v", (G * vdim, D)), (p + "q.norm", (dim,)),
+                     (p + "k.norm", (dim,)), (p + "r1", (H,)), (p + "r2", (H,)), (p + "g", (H, D))]
+        elif layer["type"] == "gla":
+            rows += [(p + "q", (H * dim, D)), (p + "k", (H * dim, D)), (p + "v", (H * vdim, D)), (p + "g", (H * vdim, D)),
+                     (p + "norm", (vdim,)), (p + "a1", (decay_rank, D)), (p + "a2", (H * dim, decay_rank)),
+                     (p + "a2.b", (H * dim,))]
+        else:
+            taps = m["conv"]
+            rows += [(p + "q", (G * dim, D)), (p + "q.conv", (G * dim, taps)), (p + "k", (G * dim, D)),
+                     (p + "k.conv", (G * dim, taps)), (p + "v", (H * vdim, D)), (p + "v.conv", (H * vdim, taps)),
+                     (p + "b", (H, D)), (p + "A_log", (H,)), (p + "norm", (vdim,)), (p + "a", (H, D)),
+                     (p + "dt_bias", (H,)), (p + "g", (H * vdim, D))]
+        rows.append((p + "o", (D, H * vdim)))
+        if layer["mlp"] is not None:
+            ff = layer["mlp"]["ff"]
+            rows += [(f"l{i}.norm2", (D,)), (f"l{i}.mlp.up", (ff, D)), (f"l{i}.mlp.down", (D, ff)), (f"l{i}.mlp.act", (4,))]
+    return rows + [("final.norm", (D,)), ("head", (config["vocab"], D))]
+
+
+def gigusun_values(name: str, shape: tuple[int, ...], rng: np.random.Generator) -> np.ndarray:
+    """Random F32 values of one tensor on a scale that keeps every mechanism alive."""
+    leaf = name.split(".mix.")[-1]
+    if leaf in ("q.norm", "k.norm", "norm"):
+        return rng.uniform(0.7, 1.4, shape)
+    if name.endswith(("norm", "norm1", "norm2")):
+        return rng.normal(0.0, 0.15, shape)
+    if leaf in ("r1", "r2"):
+        return rng.uniform(0.1, 0.9, shape)
+    if leaf == "A_log":
+        return rng.uniform(-2.0, 1.0, shape)
+    if leaf == "dt_bias":
+        return rng.uniform(-3.0, 0.5, shape)
+    if leaf == "a2.b":
+        return rng.uniform(-1.0, 4.0, shape)
+    if leaf.endswith("conv"):
+        return rng.normal(0.0, 0.6, shape)
+    if name.endswith("mlp.act"):
+        return rng.normal(0.0, 0.5, shape)
+    if name in ("embed", "pos"):
+        return rng.normal(0.0, 1.0 if name == "embed" else 0.5, shape)
+    return rng.normal(0.0, 1.0 / math.sqrt(shape[-1]), shape)
+
+
+def gigusun_weights(config: dict, seed: int, decay_rank: int = 16) -> dict[str, np.ndarray]:
+    """{name: F32 values that BF16 holds exactly}."""
+    rng = np.random.default_rng(seed)
+    weights = {}
+    for name, shape in gigusun_manifest(config, decay_rank):
+        bits = np.frombuffer(_bf16_bytes(gigusun_values(name, shape, rng)), np.uint16).astype(np.uint32) << 16
+        weights[name] = bits.view(np.float32).reshape(shape)
+    return weights
+
+
+def write_gigusun(directory: Path, config: dict, weights: dict[str, np.ndarray]) -> Path:
+    """Writes config.json and model.safetensors; returns the directory (what a loader is pointed at)."""
+    directory = Path(directory)
+    directory.mkdir(parents=True, exist_ok=True)
+    (directory / "config.json").write_text(json.dumps(config, indent=1))
+    write_model(directory / "model.safetensors", {},
+                ((name, "BF16", list(values.shape), _bf16_bytes(values)) for name, values in weights.items()))
+    return directory
+
+
+def write_gigusun_random(directory: Path, config: dict, seed: int, device: str, decay_rank: int = 16) -> Path:
+    """As write_gigusun with seeded weights; the large matrices are drawn by torch on `device`."""
+    import torch
+
+    directory = Path(directory)
+    directory.mkdir(parents=True, exist_ok=True)
+    (directory / "config.json").write_text(json.dumps(config, indent=1))
+    rng = np.random.default_rng(seed)
+    generator = torch.Generator(device=device)
+    generator.manual_seed(seed)
+
+    def tensors():
+        for name, shape in gigusun_manifest(config, decay_rank):
+            if len(shape) == 2 and math.prod(shape) >= 1 << 16:
+                std = 1.0 if name == "embed" else 0.5 if name == "pos" else 1.0 / math.sqrt(shape[-1])
+                drawn = (torch.randn(math.prod(shape), generator=generator, device=device) * std).bfloat16()
+                payload = drawn.view(torch.int16).cpu().numpy().tobytes()
+            else:
+                payload = _bf16_bytes(gigusun_values(name, shape, rng))
+            yield name, "BF16", list(shape), payload
+
+    write_model(directory / "model.safetensors", {}, tensors(), max_shard_bytes=1 << 40)
+    return directory

@@ -189,7 +189,8 @@ distance_bias_kernel(const float *__restrict__ r1, const float *__restrict__ r2,
     table[static_cast<std::size_t>(head) * distances + d] = r1[head] * logf(fmaf(r2[head], static_cast<float>(d), 1.0F));
 }
 
-// 64 x 64 output tile, 16 inputs per step, 4 x 4 products per thread; plain F32 multiply-adds.
+// 64 x 64 output tile, 16 inputs per step, 4 x 4 products per thread; plain F32 multiply-adds, every step's 16
+// products summed on their own before they join the running sum.
 __global__ void __launch_bounds__(256)
 linear_f32_kernel(const float *__restrict__ input, const bf16 *__restrict__ weight, float *__restrict__ output,
                   const int rows, const int out_features, const int in_features, const bool accumulate) {
@@ -207,6 +208,7 @@ linear_f32_kernel(const float *__restrict__ input, const bf16 *__restrict__ weig
           n0 + r < out_features && inside ? bf2f(weight[static_cast<std::size_t>(n0 + r) * in_features + k0 + k]) : 0.0F;
     }
     __syncthreads();
+    float step[4][4] = {};
 #pragma unroll
     for (int k = 0; k < 16; ++k) {
       const float4 x = *reinterpret_cast<const float4 *>(&x_tile[k][ty * 4]);
@@ -215,8 +217,12 @@ linear_f32_kernel(const float *__restrict__ input, const bf16 *__restrict__ weig
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xs[i], ws[j], acc[i][j]);
+        for (int j = 0; j < 4; ++j) step[i][j] = fmaf(xs[i], ws[j], step[i][j]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] += step[i][j];
     __syncthreads();
   }
   for (int i = 0; i < 4; ++i)

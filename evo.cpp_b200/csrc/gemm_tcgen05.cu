@@ -110,18 +110,38 @@ __device__ __forceinline__ void tile_coordinates(const int tile, const int tiles
   *tile_n = local / rows;
 }
 
+// Per-warp shared-memory block in which F32 results are turned from rows per lane to columns per lane.
+constexpr int kStagingStride = 36;  // floats: 16-byte accesses of both directions without bank conflicts
+constexpr int kStagingBytes = 32 * kStagingStride * 4;
+
 // One warp's share of a finished 128 x BN accumulator (TMEM lane quarter `quarter` of the tile that
 // starts at column address tmem_tile): scale, bias, gate, residual and the BF16 rounding points of the
 // upstream graph, or the F32 / split-K forms.  Rows m0 .., columns n0 .. of the output.
 template <int BN>
 __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const int M, const int N, const int m0,
                                               const int n0, const int split, const std::uint32_t tmem_tile,
-                                              const int quarter, const int lane) {
+                                              const int quarter, const int lane, float *const staging) {
   const int row = m0 + quarter * 32 + lane;
   const float scale = ep.row_scale != nullptr && row < M ? ep.alpha * ep.row_scale[row] : ep.alpha;
   const std::uint32_t taddr = tmem_tile + (static_cast<std::uint32_t>(quarter * 32) << 16U);
   const bool gated = ep.gate_mode != 0;
   const int chunks = gated ? BN / 64 : BN / 32;
+  float *const f32_base =
+      ep.out_f32 != nullptr ? ep.out_f32 + static_cast<std::size_t>(split) * ep.partial_stride : nullptr;
+  const bool f32_vectors = ep.out_f32 != nullptr && (ep.ld_out % 4) == 0 && (ep.partial_stride % 4) == 0 && (N % 4) == 0 &&
+                           (reinterpret_cast<std::uintptr_t>(ep.out_f32) & 15U) == 0;
+  float4 old[8];
+  const auto fetch_old = [&](const int c) {
+    const int at = n0 + c * 32 + (lane % 8) * 4;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int r = m0 + quarter * 32 + 4 * i + lane / 8;
+      old[i] = ep.accumulate_f32 != 0 && r < M && at < N
+                   ? *reinterpret_cast<const float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at)
+                   : make_float4(0.0F, 0.0F, 0.0F, 0.0F);
+    }
+  };
+  if (f32_vectors) fetch_old(0);
   for (int c = 0; c < chunks; ++c) {
     std::uint32_t v[32];
     std::uint32_t w[32];
@@ -131,28 +151,41 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
     const int col = gated ? n0 / 2 + c * 32 : n0 + c * 32;
     const int n_limit = gated ? N / 2 : N;
     if (ep.out_f32 != nullptr) {
-      if (row < M && col < n_limit) {
-        float *const out_row = ep.out_f32 + static_cast<std::size_t>(split) * ep.partial_stride +
-                               static_cast<std::size_t>(row) * ep.ld_out;
-        if (col + 32 <= n_limit && (ep.ld_out % 4) == 0 && (ep.partial_stride % 4) == 0 &&
-            (reinterpret_cast<std::uintptr_t>(ep.out_f32) & 15U) == 0) {
+      if (f32_vectors) {
+        // whole 16-byte words: the warp turns its 32 x 32 block around in shared memory, so that eight lanes
+        // cover 128 bytes of a row; the values an accumulating product adds to were fetched one block ahead
 #pragma unroll
-          for (int q = 0; q < 8; ++q) {
-            float4 *const slot = reinterpret_cast<float4 *>(out_row + col + 4 * q);
-            float4 value = make_float4(__uint_as_float(v[4 * q]) * scale, __uint_as_float(v[4 * q + 1]) * scale,
-                                       __uint_as_float(v[4 * q + 2]) * scale, __uint_as_float(v[4 * q + 3]) * scale);
-            if (ep.bias_f32 != nullptr) {
-              const float *const b = ep.bias_f32 + col + 4 * q;
-              value.x += b[0], value.y += b[1], value.z += b[2], value.w += b[3];
-            }
-            if (ep.accumulate_f32 != 0) {
-              const float4 old = *slot;
-              value.x += old.x, value.y += old.y, value.z += old.z, value.w += old.w;
-            }
-            *slot = value;
-          }
-          continue;
+        for (int q = 0; q < 8; ++q)
+          *reinterpret_cast<float4 *>(staging + lane * kStagingStride + 4 * q) =
+              make_float4(__uint_as_float(v[4 * q]) * scale, __uint_as_float(v[4 * q + 1]) * scale,
+                          __uint_as_float(v[4 * q + 2]) * scale, __uint_as_float(v[4 * q + 3]) * scale);
+        __syncwarp();
+        float4 sums[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float4 value =
+              *reinterpret_cast<const float4 *>(staging + (4 * i + lane / 8) * kStagingStride + (lane % 8) * 4);
+          sums[i] = make_float4(value.x + old[i].x, value.y + old[i].y, value.z + old[i].z, value.w + old[i].w);
         }
+        __syncwarp();
+        const int at = n0 + c * 32 + (lane % 8) * 4;
+        if (c + 1 < chunks) fetch_old(c + 1);
+        if (at < n_limit) {
+          float4 shift = make_float4(0.0F, 0.0F, 0.0F, 0.0F);
+          if (ep.bias_f32 != nullptr)
+            shift = make_float4(ep.bias_f32[at], ep.bias_f32[at + 1], ep.bias_f32[at + 2], ep.bias_f32[at + 3]);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const int r = m0 + quarter * 32 + 4 * i + lane / 8;
+            if (r < M)
+              *reinterpret_cast<float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at) =
+                  make_float4(sums[i].x + shift.x, sums[i].y + shift.y, sums[i].z + shift.z, sums[i].w + shift.w);
+          }
+        }
+        continue;
+      }
+      if (row < M && col < n_limit) {
+        float *const out_row = f32_base + static_cast<std::size_t>(row) * ep.ld_out;
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           if (col + j < n_limit) {
@@ -234,7 +267,8 @@ struct SharedLayout {
   static constexpr int kBarrierCount = 2 * kStages + 4;
   static constexpr int kTmemPtrOffset = kBarrierOffset + kBarrierCount * 8;
   static constexpr int kAbortOffset = kTmemPtrOffset + 8;
-  static constexpr int kTotal = kAbortOffset + 8 + 1024;  // + alignment slack
+  static constexpr int kStagingOffset = (kAbortOffset + 8 + 15) / 16 * 16;  // one block per epilogue warp
+  static constexpr int kTotal = kStagingOffset + 4 * kStagingBytes + 1024;  // + alignment slack
 };
 
 template <bool kFp8, int BN>
@@ -382,7 +416,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
       const std::uint32_t acc_phase = (local >> 1) & 1U;
       if (!mbar_wait(tmem_full_bar(acc), acc_phase, abort_flag)) break;
       tc_fence_after();
-      epilogue_tile<BN>(ep, M, N, m0, n0, split, tmem_base + acc * BN, quarter, lane);
+      epilogue_tile<BN>(ep, M, N, m0, n0, split, tmem_base + acc * BN, quarter, lane,
+                        reinterpret_cast<float *>(smem + L::kStagingOffset + quarter * kStagingBytes));
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(tmem_empty_bar(acc));
@@ -427,7 +462,8 @@ struct PairLayout {
   static constexpr int kBarrierCount = 2 * kPairStages + 4;
   static constexpr int kTmemPtrOffset = kBarrierOffset + kBarrierCount * 8;
   static constexpr int kAbortOffset = kTmemPtrOffset + 8;
-  static constexpr int kTotal = kAbortOffset + 8 + 1024;  // + alignment slack
+  static constexpr int kStagingOffset = (kAbortOffset + 8 + 15) / 16 * 16;  // one block per epilogue warp
+  static constexpr int kTotal = kStagingOffset + 4 * kStagingBytes + 1024;  // + alignment slack
 };
 
 __device__ __forceinline__ std::uint32_t cluster_rank() {
@@ -627,7 +663,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
       const std::uint32_t acc_phase = (local >> 1) & 1U;
       if (!mbar_wait(tmem_full_bar(acc), acc_phase, abort_flag)) break;
       tc_fence_after();
-      epilogue_tile<kPairN>(ep, M, N, m0, n0, split, tmem_base + acc * kPairN, quarter, lane);
+      epilogue_tile<kPairN>(ep, M, N, m0, n0, split, tmem_base + acc * kPairN, quarter, lane,
+                            reinterpret_cast<float *>(smem + PairLayout::kStagingOffset + quarter * kStagingBytes));
       tc_fence_before();
       __syncwarp();
       if (lane == 0) {

@@ -2,6 +2,7 @@
 #include "../../include/evo_b200_ops.h"
 
 #include "common.cuh"
+#include "decoder_ops.hpp"
 #include "ops_internal.hpp"
 
 namespace {
@@ -9,6 +10,7 @@ namespace {
 using namespace evob;
 
 cudaStream_t as_stream(void *stream) { return static_cast<cudaStream_t>(stream); }
+Activation activation_of(const int float32) { return float32 != 0 ? Activation::kF32 : Activation::kBf16; }
 
 // Row-interleave W1/W2 in blocks of 128 rows so that every 256-column GEMM
 // tile holds matching halves of both up-projections.
@@ -588,6 +590,138 @@ int evo_b200_e4m3_encode_array(const float *values, size_t count, float scale, u
   if (!fp8::valid_scale(scale)) return fail(kInvalidArgument, "E4M3 scale must be positive and finite");
   for (size_t i = 0; i < count; ++i) codes[i] = fp8::encode_e4m3fn(values[i] * scale);
   return kOk;
+}
+
+int evo_b200_embed_positions(const void *tokens, const void *table, const void *positions, const void *gain,
+                             size_t rows, size_t width, size_t vocabulary, size_t position, float epsilon,
+                             void *output, void *stream) {
+  return embed_positions(static_cast<const std::uint32_t *>(tokens), table, positions, static_cast<const float *>(gain),
+                         rows, width, vocabulary, position, epsilon, static_cast<float *>(output), as_stream(stream));
+}
+int evo_b200_rms_norm_residual(const void *input, const void *gain, size_t rows, size_t width, float epsilon,
+                               int float32, void *output, void *stream) {
+  return rms_norm_residual(static_cast<const float *>(input), static_cast<const float *>(gain), rows, width, epsilon,
+                           output, activation_of(float32), as_stream(stream));
+}
+int evo_b200_poly_norm(const void *input, const void *coefficients, size_t rows, size_t width, float epsilon,
+                       int float32, void *output, void *stream) {
+  return poly_norm(input, static_cast<const float *>(coefficients), rows, width, epsilon, output,
+                   activation_of(float32), as_stream(stream));
+}
+int evo_b200_distance_bias_table(const void *r1, const void *r2, size_t heads, size_t distances, void *table,
+                                 void *stream) {
+  return distance_bias_table(static_cast<const float *>(r1), static_cast<const float *>(r2), heads, distances,
+                             static_cast<float *>(table), as_stream(stream));
+}
+int evo_b200_f32_linear(const void *input, const void *weight, size_t rows, size_t in_features, size_t out_features,
+                        int accumulate, void *output, void *stream) {
+  return linear_f32(static_cast<const float *>(input), weight, rows, in_features, out_features,
+                    static_cast<float *>(output), accumulate != 0, as_stream(stream));
+}
+int evo_b200_bf16_linear_f32_result(const void *input, const void *weight, size_t rows, size_t in_features,
+                                    size_t out_features, int accumulate, void *split_workspace,
+                                    size_t split_workspace_bytes, void *output, void *stream) {
+  LinearArgs a;
+  a.input = input;
+  a.weight = weight;
+  a.rows = rows;
+  a.in_features = in_features;
+  a.out_features = out_features;
+  a.output_f32 = static_cast<float *>(output);
+  a.accumulate_f32 = accumulate != 0;
+  a.split_workspace = split_workspace;
+  a.split_workspace_bytes = split_workspace_bytes;
+  return linear(a, as_stream(stream));
+}
+int evo_b200_head_norm_append(const evo_b200_head_norm *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args)) return fail(kInvalidArgument, "head norm arguments are required");
+  HeadNormArgs a;
+  a.projection = args->projection;
+  a.stride = args->stride;
+  a.key_column = args->key_column;
+  a.value_column = args->value_column;
+  a.query_gain = static_cast<const float *>(args->query_gain);
+  a.key_gain = static_cast<const float *>(args->key_gain);
+  a.query = args->query;
+  a.key_cache = args->key_cache;
+  a.value_cache = args->value_cache;
+  a.rows = args->rows;
+  a.position = args->position;
+  a.capacity = args->capacity;
+  a.heads = args->heads;
+  a.kv_heads = args->kv_heads;
+  a.dim = args->dim;
+  a.value_dim = args->value_dim;
+  a.epsilon = args->epsilon;
+  a.type = activation_of(args->float32);
+  return head_norm_append(a, as_stream(stream));
+}
+int evo_b200_window_attention(const evo_b200_window_attention_args *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args))
+    return fail(kInvalidArgument, "window attention arguments are required");
+  WindowAttentionArgs a;
+  a.query = args->query;
+  a.key_cache = args->key_cache;
+  a.value_cache = args->value_cache;
+  a.gate = args->gate;
+  a.gate_stride = args->gate_stride;
+  a.distance_bias = static_cast<const float *>(args->distance_bias);
+  a.bias_stride = args->bias_stride;
+  a.output = args->output;
+  a.rows = args->rows;
+  a.position = args->position;
+  a.capacity = args->capacity;
+  a.heads = args->heads;
+  a.kv_heads = args->kv_heads;
+  a.dim = args->dim;
+  a.value_dim = args->value_dim;
+  a.window = args->window;
+  a.keep_first = args->keep_first;
+  a.scale = args->scale;
+  a.softcap = args->softcap;
+  a.sink = args->sink != 0;
+  a.type = activation_of(args->float32);
+  a.force = args->kernel;
+  return window_attention(a, as_stream(stream));
+}
+size_t evo_b200_recurrent_workspace_bytes(int delta, size_t rows, size_t heads, size_t kv_heads, size_t dim,
+                                          size_t value_dim, int float32) {
+  return recurrent_workspace_bytes(delta != 0, rows, heads, kv_heads, dim, value_dim, activation_of(float32));
+}
+int evo_b200_recurrent_mixer(const evo_b200_recurrent_args *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args))
+    return fail(kInvalidArgument, "recurrent mixer arguments are required");
+  RecurrentArgs a;
+  a.delta = args->delta != 0;
+  a.projection = args->projection;
+  a.stride = args->stride;
+  a.key_column = args->key_column;
+  a.value_column = args->value_column;
+  a.gate_column = args->gate_column;
+  a.beta_column = args->beta_column;
+  a.decay_column = args->decay_column;
+  a.rows = args->rows;
+  a.heads = args->heads;
+  a.kv_heads = args->kv_heads;
+  a.dim = args->dim;
+  a.value_dim = args->value_dim;
+  a.conv = static_cast<const float *>(args->conv);
+  a.conv_taps = args->conv_taps;
+  a.conv_history = args->conv_history;
+  a.decay_rate = static_cast<const float *>(args->decay_rate);
+  a.decay_shift = static_cast<const float *>(args->decay_shift);
+  a.decay_weight = static_cast<const float *>(args->decay_weight);
+  a.decay_bias = static_cast<const float *>(args->decay_bias);
+  a.decay_rank = args->decay_rank;
+  a.tau = args->tau;
+  a.output_norm = static_cast<const float *>(args->output_norm);
+  a.epsilon = args->epsilon;
+  a.state = static_cast<float *>(args->state);
+  a.fresh = args->fresh != 0;
+  a.workspace = args->workspace;
+  a.output = args->output;
+  a.type = activation_of(args->float32);
+  return recurrent_mixer(a, as_stream(stream));
 }
 
 }  // extern "C"

@@ -6,9 +6,11 @@
 //   1. preparation: per token the decays and the queries / keys the recurrence reads (F32), for the delta
 //      rule also the short convolutions, the unit vectors, the step sizes, and the scalars of the blocked
 //      form below;
-//   2. the recurrence: columns of the state (one per value channel) never mix, so a CTA owns 16 of them;
-//      eight lanes share a column, each with kElements key channels of it in registers, and the tokens
-//      stream through a double-buffered shared-memory tile;
+//   2. the recurrence: columns of the state (one per value channel) never mix, so a CTA owns 16 of them and
+//      a warp four; the warp's lanes divide the key channels between them (2, 4 or 8 each, so that one
+//      shared-memory read of a key serves four columns) and the state stays in registers as packed pairs.
+//      Tokens stream through a double-buffered shared-memory tile; sums over the channels are shuffle
+//      exchanges that leave every lane with one column and one token;
 //   3. the output norm and gate, row-wise.
 //
 // Blocked delta rule.  Four tokens at a time, with S the state in front of the block, G_t = g_0 .. g_t and
@@ -16,7 +18,7 @@
 //   u_t = beta_t (v_t - G_t S^T k_t - sum_{s<t} D_ts (k_s.k_t) u_s)
 //   o_t = G_t S^T q_t + sum_{s<=t} D_ts (k_s.q_t) u_s
 //   S'  = G_3 S + sum_s D_3s k_s u_s^T
-// so the eight products with S are taken at once and reduced over the lanes together; the scalars
+// so the eight products with S are taken at once and summed over the lanes together; the scalars
 // depend on the head only and come from the preparation.
 #include "decoder_types.cuh"
 #include "ops_internal.hpp"
@@ -263,15 +265,67 @@ __device__ __forceinline__ void copy16(float *const dst, const float *const src)
                : "memory");
 }
 
-// Sums four values over the eight lanes of a column; lane p is left with the sum of value
-// 2 * bit2(p) + bit1(p).
-__device__ __forceinline__ float reduce_scatter4(const float (&v)[4], const int part) {
-  const bool high = (part & 4) != 0, odd = (part & 2) != 0;
-  float a = high ? v[2] : v[0], b = high ? v[3] : v[1];
-  a += __shfl_xor_sync(0xffffffffU, high ? v[0] : v[2], 4);
-  b += __shfl_xor_sync(0xffffffffU, high ? v[1] : v[3], 4);
-  float c = odd ? b : a;
-  c += __shfl_xor_sync(0xffffffffU, odd ? a : b, 2);
+// Packed F32 pairs: one instruction for two multiply-adds.
+using Pair = unsigned long long;
+__device__ __forceinline__ Pair pair_of(const float low, const float high) {
+  Pair d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(low), "f"(high));
+  return d;
+}
+__device__ __forceinline__ float low_of(const Pair v) { return __uint_as_float(static_cast<unsigned int>(v)); }
+__device__ __forceinline__ float high_of(const Pair v) { return __uint_as_float(static_cast<unsigned int>(v >> 32)); }
+__device__ __forceinline__ Pair fma2(const Pair a, const Pair b, const Pair c) {
+  Pair d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ Pair mul2(const Pair a, const Pair b) {
+  Pair d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
+// A lane's key channels in a shared-memory row: kElements = 2 -> 2 lane + i, otherwise runs of four, run r at
+// 128 r + 4 lane.
+template <int kElements>
+__device__ __forceinline__ int channel_of(const int lane, const int e) {
+  if constexpr (kElements == 2) return 2 * lane + e;
+  else return 128 * (e / 4) + 4 * lane + e % 4;
+}
+template <int kElements>
+__device__ __forceinline__ void load_pairs(const float *const row, const int lane, Pair (&v)[kElements / 2]) {
+  if constexpr (kElements == 2) {
+    v[0] = *reinterpret_cast<const Pair *>(row + 2 * lane);
+  } else {
+#pragma unroll
+    for (int r = 0; r < kElements / 4; ++r) {
+      const ulonglong2 w = *reinterpret_cast<const ulonglong2 *>(row + 128 * r + 4 * lane);
+      v[2 * r] = w.x;
+      v[2 * r + 1] = w.y;
+    }
+  }
+}
+
+// Sums of a warp's 4 columns x 4 tokens over its 32 lanes.  The first two exchanges leave a lane with the
+// column of its upper two bits, partly summed (over 4 of the 32 lanes).
+__device__ __forceinline__ void scatter_columns(const float (&v)[4][kBlock], const int lane, float (&own)[kBlock]) {
+  const bool upper = (lane & 16) != 0, odd = (lane & 8) != 0;
+  float half[2][kBlock];
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int t = 0; t < kBlock; ++t)
+      half[c][t] = (upper ? v[c + 2][t] : v[c][t]) + __shfl_xor_sync(0xffffffffU, upper ? v[c][t] : v[c + 2][t], 16);
+#pragma unroll
+  for (int t = 0; t < kBlock; ++t)
+    own[t] = (odd ? half[1][t] : half[0][t]) + __shfl_xor_sync(0xffffffffU, odd ? half[0][t] : half[1][t], 8);
+}
+// ... and this leaves the sum of token 2 * bit 2 + bit 1 in the lane.
+__device__ __forceinline__ float scatter_tokens(const float (&own)[kBlock], const int lane) {
+  const bool upper = (lane & 4) != 0, odd = (lane & 2) != 0;
+  const float a = (upper ? own[2] : own[0]) + __shfl_xor_sync(0xffffffffU, upper ? own[0] : own[2], 4);
+  const float b = (upper ? own[3] : own[1]) + __shfl_xor_sync(0xffffffffU, upper ? own[1] : own[3], 4);
+  const float c = (odd ? b : a) + __shfl_xor_sync(0xffffffffU, odd ? a : b, 2);
   return c + __shfl_xor_sync(0xffffffffU, c, 1);
 }
 
@@ -280,7 +334,8 @@ __global__ void __launch_bounds__(kRecurrenceThreads)
 recurrence_kernel(const float *__restrict__ queries, const float *__restrict__ keys, const float *__restrict__ alpha,
                   const T *__restrict__ values, const float *__restrict__ scalars, float *__restrict__ state,
                   float *__restrict__ output, const RecurrenceParams p) {
-  constexpr int kWidth = kElements * 8;
+  constexpr int kWidth = kElements * 32;
+  constexpr int kPairs = kElements / 2;
   constexpr int kVectors = kDelta ? 2 : 3;  // keys, queries (, decays)
   constexpr int kScalarFloats = kDelta ? kTile / kBlock * kScalars : 0;
   constexpr int kBuffer = kVectors * kTile * kWidth + kScalarFloats + kTile * kColumns;
@@ -288,9 +343,10 @@ recurrence_kernel(const float *__restrict__ queries, const float *__restrict__ k
   const int head = blockIdx.y, column0 = blockIdx.x * kColumns;
   const int key_head = kDelta ? head / (p.heads / p.kv_heads) : head;
   const int key_heads = kDelta ? p.kv_heads : p.heads;
-  const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, part = lane % 8;
-  const int local = warp * 4 + lane / 8, column = column0 + local;  // this thread's state column
-  const bool live = column < p.value_dim;
+  const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+  const int own_column = column0 + warp * 4 + lane / 8;  // the column whose sums this lane ends up with
+  const bool own_live = own_column < p.value_dim;
+  const int own_token = 2 * ((lane >> 2) & 1) + ((lane >> 1) & 1);
   const int tiles = (p.rows + kTile - 1) / kTile;
 
   for (int i = threadIdx.x; i < 2 * kBuffer; i += kRecurrenceThreads) smem[i] = 0.0F;  // channels past dim stay zero
@@ -320,30 +376,37 @@ recurrence_kernel(const float *__restrict__ queries, const float *__restrict__ k
   };
   // values go through registers: kTile x kColumns of them, two per thread
   constexpr int kValuesPerThread = kTile * kColumns / kRecurrenceThreads;
-  float staged[kValuesPerThread];
+  T staged[kValuesPerThread];  // widened only when they are stored: the loads stay in flight until then
   const auto load_values = [&](const int tile) {
 #pragma unroll
     for (int i = 0; i < kValuesPerThread; ++i) {
       const int index = i * kRecurrenceThreads + threadIdx.x, row = tile * kTile + index / kColumns, c = column0 + index % kColumns;
       staged[i] = row < p.rows && c < p.value_dim
-                      ? to_float(values[static_cast<std::size_t>(row) * p.value_stride + head * p.value_dim + c])
-                      : 0.0F;
+                      ? values[static_cast<std::size_t>(row) * p.value_stride + head * p.value_dim + c]
+                      : from_float<T>(0.0F);
     }
   };
   const auto store_values = [&](const int tile) {
     float *const b = buffer(tile) + kVectors * kTile * kWidth + kScalarFloats;
 #pragma unroll
-    for (int i = 0; i < kValuesPerThread; ++i) b[i * kRecurrenceThreads + threadIdx.x] = staged[i];
+    for (int i = 0; i < kValuesPerThread; ++i) b[i * kRecurrenceThreads + threadIdx.x] = to_float(staged[i]);
   };
 
-  float S[kElements];
+  Pair S[4][kPairs];  // [column of the warp][channel pair]
 #pragma unroll
-  for (int e = 0; e < kElements; ++e) {
-    const int d = (e / 4 * 8 + part) * 4 + e % 4;
-    S[e] = p.fresh == 0 && live && d < p.dim
-               ? state[(static_cast<std::size_t>(head) * p.dim + d) * p.value_dim + column]
-               : 0.0F;
-  }
+  for (int c = 0; c < 4; ++c)
+#pragma unroll
+    for (int e = 0; e < kPairs; ++e) {
+      float v[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int d = channel_of<kElements>(lane, 2 * e + i), column = column0 + warp * 4 + c;
+        v[i] = p.fresh == 0 && d < p.dim && column < p.value_dim
+                   ? state[(static_cast<std::size_t>(head) * p.dim + d) * p.value_dim + column]
+                   : 0.0F;
+      }
+      S[c][e] = pair_of(v[0], v[1]);
+    }
   fetch(0);
   load_values(0);
   for (int tile = 0; tile < tiles; ++tile) {
@@ -355,93 +418,114 @@ recurrence_kernel(const float *__restrict__ queries, const float *__restrict__ k
       load_values(tile + 1);
     }
     const float *const b = buffer(tile);
-    const float *const value_tile = b + kVectors * kTile * kWidth + kScalarFloats + local;
-    const float *const lane_base = b + part * 4;
-    const int blocks = min(kTile, p.rows - tile * kTile + kBlock - 1) / kBlock;
-    for (int block = 0; block < blocks; ++block) {
-      const float *const base = lane_base + block * kBlock * kWidth;
-      float read[kBlock];  // S^T q_t
+    const float *const value_tile = b + kVectors * kTile * kWidth + kScalarFloats + warp * 4;
+    // (rows past the last token are neutral: no key, no step, no decay)
+#pragma unroll
+    for (int block = 0; block < kTile / kBlock; ++block) {
+      const float *const base = b + block * kBlock * kWidth;
+      float o;
       if constexpr (kDelta) {
         const float *const c = b + kVectors * kTile * kWidth + block * kScalars;
-        float k[kBlock][kElements], held[kBlock];  // S^T k_t
+        Pair k[kBlock][kPairs];
+        float held[4][kBlock], read[4][kBlock];  // this lane's share of S^T k_t and S^T q_t
 #pragma unroll
         for (int t = 0; t < kBlock; ++t) {
-          float dk[2] = {0.0F, 0.0F}, dq[2] = {0.0F, 0.0F};
+          Pair q[kPairs];
+          load_pairs<kElements>(base + t * kWidth, lane, k[t]);
+          load_pairs<kElements>(base + (kTile + t) * kWidth, lane, q);
 #pragma unroll
-          for (int e = 0; e < kElements; e += 4) {
-            const float4 kv = *reinterpret_cast<const float4 *>(base + t * kWidth + e * 8);
-            const float4 qv = *reinterpret_cast<const float4 *>(base + (kTile + t) * kWidth + e * 8);
-            k[t][e] = kv.x, k[t][e + 1] = kv.y, k[t][e + 2] = kv.z, k[t][e + 3] = kv.w;
-            dk[0] = fmaf(S[e], kv.x, dk[0]);
-            dk[1] = fmaf(S[e + 1], kv.y, dk[1]);
-            dk[0] = fmaf(S[e + 2], kv.z, dk[0]);
-            dk[1] = fmaf(S[e + 3], kv.w, dk[1]);
-            dq[0] = fmaf(S[e], qv.x, dq[0]);
-            dq[1] = fmaf(S[e + 1], qv.y, dq[1]);
-            dq[0] = fmaf(S[e + 2], qv.z, dq[0]);
-            dq[1] = fmaf(S[e + 3], qv.w, dq[1]);
+          for (int column = 0; column < 4; ++column) {
+            Pair dk = mul2(S[column][0], k[t][0]), dq = mul2(S[column][0], q[0]);
+#pragma unroll
+            for (int e = 1; e < kPairs; ++e) {
+              dk = fma2(S[column][e], k[t][e], dk);
+              dq = fma2(S[column][e], q[e], dq);
+            }
+            held[column][t] = low_of(dk) + high_of(dk);
+            read[column][t] = low_of(dq) + high_of(dq);
           }
-          held[t] = dk[0] + dk[1];
-          read[t] = dq[0] + dq[1];
         }
-        const float mine = reduce_scatter4(held, part);
-        const float read_sum = reduce_scatter4(read, part);
+        float h[kBlock], r[kBlock];
+        scatter_columns(held, lane, h);
+        scatter_columns(read, lane, r);
 #pragma unroll
-        for (int t = 0; t < kBlock; ++t) held[t] = __shfl_sync(0xffffffffU, mine, (lane & 24) + 2 * t);
+        for (int offset = 4; offset > 0; offset /= 2)
+#pragma unroll
+          for (int t = 0; t < kBlock; ++t) h[t] += __shfl_xor_sync(0xffffffffU, h[t], offset);
+        const float read_sum = scatter_tokens(r, lane);
         const float4 beta = *reinterpret_cast<const float4 *>(c + kBeta);
         const float4 beta_g = *reinterpret_cast<const float4 *>(c + kBetaG);
         const float4 pair_a = *reinterpret_cast<const float4 *>(c + kPair);
         const float4 pair_b = *reinterpret_cast<const float4 *>(c + kPair + 4);
         const float4 tail = *reinterpret_cast<const float4 *>(c + kTail);
-        const float *const v = value_tile + block * kBlock * kColumns;
-        const float u0 = fmaf(-beta_g.x, held[0], beta.x * v[0]);
-        const float u1 = fmaf(-pair_a.x, u0, fmaf(-beta_g.y, held[1], beta.y * v[kColumns]));
-        const float u2 = fmaf(-pair_a.z, u1, fmaf(-pair_a.y, u0, fmaf(-beta_g.z, held[2], beta.z * v[2 * kColumns])));
-        const float u3 = fmaf(-pair_b.y, u2, fmaf(-pair_b.x, u1, fmaf(-pair_a.w, u0, fmaf(-beta_g.w, held[3], beta.w * v[3 * kColumns]))));
-        const int t = 2 * ((part >> 2) & 1) + ((part >> 1) & 1);
-        const float4 r = *reinterpret_cast<const float4 *>(c + kRead + 4 * t);
-        const float o = fmaf(r.w, u3, fmaf(r.z, u2, fmaf(r.y, u1, fmaf(r.x, u0, c[kG + t] * read_sum))));
-        const int row = tile * kTile + block * kBlock + t;
-        if ((part & 1) == 0 && live && row < p.rows)
-          output[(static_cast<std::size_t>(row) * p.heads + head) * p.value_dim + column] = o;
+        const float *const v = value_tile + block * kBlock * kColumns + lane / 8;
+        const float u0 = fmaf(-beta_g.x, h[0], beta.x * v[0]);
+        const float u1 = fmaf(-pair_a.x, u0, fmaf(-beta_g.y, h[1], beta.y * v[kColumns]));
+        const float u2 = fmaf(-pair_a.z, u1, fmaf(-pair_a.y, u0, fmaf(-beta_g.z, h[2], beta.z * v[2 * kColumns])));
+        const float u3 = fmaf(-pair_b.y, u2, fmaf(-pair_b.x, u1, fmaf(-pair_a.w, u0, fmaf(-beta_g.w, h[3], beta.w * v[3 * kColumns]))));
+        const float4 w = *reinterpret_cast<const float4 *>(c + kRead + 4 * own_token);
+        o = fmaf(w.w, u3, fmaf(w.z, u2, fmaf(w.y, u1, fmaf(w.x, u0, c[kG + own_token] * read_sum))));
+        // what the block adds to the columns: every lane needs all four
+        const float added[kBlock] = {tail.x * u0, tail.y * u1, tail.z * u2, u3};
         const float g = c[kG + kBlock - 1];
-        const float w0 = tail.x * u0, w1 = tail.y * u1, w2 = tail.z * u2;
+        const Pair gg = pair_of(g, g);
 #pragma unroll
-        for (int e = 0; e < kElements; ++e)
-          S[e] = fmaf(k[3][e], u3, fmaf(k[2][e], w2, fmaf(k[1][e], w1, fmaf(k[0][e], w0, g * S[e]))));
+        for (int column = 0; column < 4; ++column) {
+          Pair a[kBlock];
+#pragma unroll
+          for (int t = 0; t < kBlock; ++t) {
+            const float x = __shfl_sync(0xffffffffU, added[t], 8 * column);
+            a[t] = pair_of(x, x);
+          }
+#pragma unroll
+          for (int e = 0; e < kPairs; ++e)
+            S[column][e] = fma2(k[3][e], a[3], fma2(k[2][e], a[2], fma2(k[1][e], a[1], fma2(k[0][e], a[0], mul2(gg, S[column][e])))));
+        }
       } else {
+        float read[4][kBlock];
+        // the block's operands are requested up front: one warp per scheduler has nothing else to hide them
+        Pair k[kBlock][kPairs], q[kBlock][kPairs], a[kBlock][kPairs];
+        float4 v[kBlock];
 #pragma unroll
         for (int t = 0; t < kBlock; ++t) {
-          const float v = value_tile[(block * kBlock + t) * kColumns];
-          float dq[2] = {0.0F, 0.0F};
-#pragma unroll
-          for (int e = 0; e < kElements; e += 4) {
-            const float4 kv = *reinterpret_cast<const float4 *>(base + t * kWidth + e * 8);
-            const float4 qv = *reinterpret_cast<const float4 *>(base + (kTile + t) * kWidth + e * 8);
-            const float4 av = *reinterpret_cast<const float4 *>(base + (2 * kTile + t) * kWidth + e * 8);
-            S[e] = fmaf(kv.x, v, av.x * S[e]);
-            S[e + 1] = fmaf(kv.y, v, av.y * S[e + 1]);
-            S[e + 2] = fmaf(kv.z, v, av.z * S[e + 2]);
-            S[e + 3] = fmaf(kv.w, v, av.w * S[e + 3]);
-            dq[0] = fmaf(S[e], qv.x, dq[0]);
-            dq[1] = fmaf(S[e + 1], qv.y, dq[1]);
-            dq[0] = fmaf(S[e + 2], qv.z, dq[0]);
-            dq[1] = fmaf(S[e + 3], qv.w, dq[1]);
-          }
-          read[t] = dq[0] + dq[1];
+          load_pairs<kElements>(base + t * kWidth, lane, k[t]);
+          load_pairs<kElements>(base + (2 * kTile + t) * kWidth, lane, a[t]);
+          v[t] = *reinterpret_cast<const float4 *>(value_tile + (block * kBlock + t) * kColumns);
+          load_pairs<kElements>(base + (kTile + t) * kWidth, lane, q[t]);
         }
-        const float o = reduce_scatter4(read, part);
-        const int row = tile * kTile + block * kBlock + 2 * ((part >> 2) & 1) + ((part >> 1) & 1);
-        if ((part & 1) == 0 && live && row < p.rows)
-          output[(static_cast<std::size_t>(row) * p.heads + head) * p.value_dim + column] = o;
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+          const float vs[4] = {v[t].x, v[t].y, v[t].z, v[t].w};
+#pragma unroll
+          for (int column = 0; column < 4; ++column) {
+            const Pair vv = pair_of(vs[column], vs[column]);
+            Pair dq = 0ULL;
+#pragma unroll
+            for (int e = 0; e < kPairs; ++e) {
+              S[column][e] = fma2(k[t][e], vv, mul2(a[t][e], S[column][e]));
+              dq = e == 0 ? mul2(S[column][e], q[t][e]) : fma2(S[column][e], q[t][e], dq);
+            }
+            read[column][t] = low_of(dq) + high_of(dq);
+          }
+        }
+        float r[kBlock];
+        scatter_columns(read, lane, r);
+        o = scatter_tokens(r, lane);
       }
+      const int row = tile * kTile + block * kBlock + own_token;
+      if ((lane & 1) == 0 && own_live && row < p.rows)
+        output[(static_cast<std::size_t>(row) * p.heads + head) * p.value_dim + own_column] = o;
     }
   }
 #pragma unroll
-  for (int e = 0; e < kElements; ++e) {
-    const int d = (e / 4 * 8 + part) * 4 + e % 4;
-    if (live && d < p.dim) state[(static_cast<std::size_t>(head) * p.dim + d) * p.value_dim + column] = S[e];
-  }
+  for (int c = 0; c < 4; ++c)
+#pragma unroll
+    for (int e = 0; e < kElements; ++e) {
+      const int d = channel_of<kElements>(lane, e), column = column0 + warp * 4 + c;
+      if (d < p.dim && column < p.value_dim)
+        state[(static_cast<std::size_t>(head) * p.dim + d) * p.value_dim + column] =
+            e % 2 == 0 ? low_of(S[c][e / 2]) : high_of(S[c][e / 2]);
+    }
 }
 
 // ---------------------------------------------------------------- output norm and gate
@@ -481,7 +565,7 @@ template <bool kDelta, int kElements, typename T>
 int launch_recurrence(const float *queries, const float *keys, const float *alpha, const T *values,
                       const float *scalars, float *state, float *output, const RecurrenceParams &p,
                       cudaStream_t stream) {
-  constexpr std::size_t kBuffer = (kDelta ? 2 : 3) * kTile * kElements * 8 + (kDelta ? kTile / kBlock * kScalars : 0) + kTile * kColumns;
+  constexpr std::size_t kBuffer = (kDelta ? 2 : 3) * kTile * kElements * 32 + (kDelta ? kTile / kBlock * kScalars : 0) + kTile * kColumns;
   constexpr std::size_t bytes = 2 * kBuffer * sizeof(float);
   if (cudaFuncSetAttribute(recurrence_kernel<kDelta, kElements, T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                            static_cast<int>(bytes)) != cudaSuccess)
@@ -496,10 +580,9 @@ template <bool kDelta, typename T>
 int dispatch_recurrence(const float *queries, const float *keys, const float *alpha, const T *values,
                         const float *scalars, float *state, float *output, const RecurrenceParams &p,
                         cudaStream_t stream) {
-  if (p.dim <= 32) return launch_recurrence<kDelta, 4, T>(queries, keys, alpha, values, scalars, state, output, p, stream);
-  if (p.dim <= 64) return launch_recurrence<kDelta, 8, T>(queries, keys, alpha, values, scalars, state, output, p, stream);
-  if (p.dim <= 128) return launch_recurrence<kDelta, 16, T>(queries, keys, alpha, values, scalars, state, output, p, stream);
-  return launch_recurrence<kDelta, 32, T>(queries, keys, alpha, values, scalars, state, output, p, stream);
+  if (p.dim <= 64) return launch_recurrence<kDelta, 2, T>(queries, keys, alpha, values, scalars, state, output, p, stream);
+  if (p.dim <= 128) return launch_recurrence<kDelta, 4, T>(queries, keys, alpha, values, scalars, state, output, p, stream);
+  return launch_recurrence<kDelta, 8, T>(queries, keys, alpha, values, scalars, state, output, p, stream);
 }
 
 template <typename T>

@@ -227,7 +227,7 @@ int Context::run_decoder_stage(Stage &s, const std::size_t rows, const Mode mode
       a.workspace = s.recurrent_workspace;
       a.output = s.mixer_out;
       a.type = type;
-      EVOB_OP(kCatRecurrence, recurrent_mixer(a, stream));
+      EVOB_OP(a.delta ? kCatGatedDelta : kCatGatedLinear, recurrent_mixer(a, stream));
     }
     if (tap != nullptr)
       EVOB_TRY(emit_activation(stream, *tap, layer, DumpPoint::kMixerOutput, s.mixer_out, rows, b.output_width(), type));

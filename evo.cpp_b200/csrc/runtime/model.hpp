@@ -40,7 +40,8 @@ enum ProfileCategory : int {
   kCatElementwise,     // embedding, gates, splits
   kCatRowQuantize,     // per-row E4M3 quantisation in front of the FP8 FFN / output projections
   kCatGemmFp8Ffn,      // tcgen05 E4M3 output and MLP projections (profile b200-fp8)
-  kCatRecurrence,      // gated linear attention and gated delta rule: preparation, recurrence, output norm and gate
+  kCatGatedLinear,     // gated linear attention: preparation, recurrence, output norm and gate
+  kCatGatedDelta,      // gated delta rule: the same, with the short convolutions
   kCatPolyNorm,        // normalised polynomial activation of a decoder's feed-forward
   kProfileCategories
 };

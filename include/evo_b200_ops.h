@@ -366,6 +366,88 @@ EVO_B200_API float evo_b200_e4m3_scaled_roundtrip(float value, float scale);
 EVO_B200_API int evo_b200_e4m3_encode_array(const float *values, size_t count, float scale,
                                             uint8_t *codes);
 
+/* ---- operators of decoder graphs (models described by a config.json).  Activations are BF16, or F32 where
+ * `float32` is not 0; gains, tables, decays, recurrent states and the residual stream are F32. */
+/* output[r] = rms_norm(table[token[r]] + positions[position + r]) * gain, F32 [rows, width]; table
+ * [vocabulary, width] and positions BF16.  Ids >= vocabulary: a row of zeros and an asynchronous error. */
+EVO_B200_API int evo_b200_embed_positions(const void *tokens, const void *table, const void *positions,
+                                          const void *gain, size_t rows, size_t width, size_t vocabulary,
+                                          size_t position, float epsilon, void *output, void *stream);
+/* F32 input [rows, width] / root mean square * gain. */
+EVO_B200_API int evo_b200_rms_norm_residual(const void *input, const void *gain, size_t rows, size_t width,
+                                            float epsilon, int float32, void *output, void *stream);
+/* a N(z) + b N(z^2) + c N(z^3) + e, coefficients = {a, b, c, e} F32 on the device; N divides a row by its
+ * root mean square. */
+EVO_B200_API int evo_b200_poly_norm(const void *input, const void *coefficients, size_t rows, size_t width,
+                                    float epsilon, int float32, void *output, void *stream);
+/* table[h, d] = r1[h] ln(1 + r2[h] d). */
+EVO_B200_API int evo_b200_distance_bias_table(const void *r1, const void *r2, size_t heads, size_t distances,
+                                              void *table, void *stream);
+/* F32 [rows, in] x BF16 [out, in]^T with F32 multiply-adds; output (+)= product. */
+EVO_B200_API int evo_b200_f32_linear(const void *input, const void *weight, size_t rows, size_t in_features,
+                                     size_t out_features, int accumulate, void *output, void *stream);
+/* BF16 [rows, in] x BF16 [out, in]^T, the F32 accumulator stored (or added) without rounding; the split
+ * workspace (optional) enables the weight-stream forms for few rows. */
+EVO_B200_API int evo_b200_bf16_linear_f32_result(const void *input, const void *weight, size_t rows,
+                                                 size_t in_features, size_t out_features, int accumulate,
+                                                 void *split_workspace, size_t split_workspace_bytes, void *output,
+                                                 void *stream);
+/* Per-head RMS norm of queries and keys of a fused projection row [queries | keys at key_column | values at
+ * value_column]; queries to query [rows, heads, dim], keys and values to cache rows position + r. */
+typedef struct evo_b200_head_norm {
+  size_t struct_size;
+  const void *projection;
+  size_t stride, key_column, value_column;
+  const void *query_gain, *key_gain;
+  void *query, *key_cache, *value_cache;
+  size_t rows, position, capacity, heads, kv_heads, dim, value_dim;
+  float epsilon;
+  int32_t float32;
+} evo_b200_head_norm;
+EVO_B200_API int evo_b200_head_norm_append(const evo_b200_head_norm *args, void *stream);
+/* Softmax attention with grouped key/value heads [capacity, kv_heads, dim]: the query at position i sees key
+ * j <= i if i - j < window (0: no limit) or j < keep_first; score = softcap tanh(q.k scale / softcap)
+ * (softcap 0: q.k scale) - distance_bias[head, i - j] (optional); sink != 0 adds exp(0) to the denominator;
+ * output [rows, heads, value_dim] times sigmoid(gate[r * gate_stride + head]) (optional).  kernel: 0 chosen by
+ * size, 1 row kernel, 2 tile kernel, 3 tcgen05 kernel (EVO_STATUS_UNSUPPORTED where it does not apply). */
+typedef struct evo_b200_window_attention_args {
+  size_t struct_size;
+  const void *query, *key_cache, *value_cache, *gate;
+  size_t gate_stride;
+  const void *distance_bias;
+  size_t bias_stride;
+  void *output;
+  size_t rows, position, capacity, heads, kv_heads, dim, value_dim, window, keep_first;
+  float scale, softcap;
+  int32_t sink, float32, kernel;
+} evo_b200_window_attention_args;
+EVO_B200_API int evo_b200_window_attention(const evo_b200_window_attention_args *args, void *stream);
+/* Gated linear attention (delta == 0) or the gated delta rule with its short convolutions, with the output
+ * norm and gate: see csrc/decoder_ops.hpp for the members. */
+typedef struct evo_b200_recurrent_args {
+  size_t struct_size;
+  int32_t delta;
+  const void *projection;
+  size_t stride, key_column, value_column, gate_column, beta_column, decay_column;
+  size_t rows, heads, kv_heads, dim, value_dim;
+  const void *conv;
+  size_t conv_taps;
+  void *conv_history;
+  const void *decay_rate, *decay_shift, *decay_weight, *decay_bias;
+  size_t decay_rank;
+  float tau;
+  const void *output_norm;
+  float epsilon;
+  void *state;
+  int32_t fresh;
+  void *workspace;
+  void *output;
+  int32_t float32;
+} evo_b200_recurrent_args;
+EVO_B200_API size_t evo_b200_recurrent_workspace_bytes(int delta, size_t rows, size_t heads, size_t kv_heads,
+                                                       size_t dim, size_t value_dim, int float32);
+EVO_B200_API int evo_b200_recurrent_mixer(const evo_b200_recurrent_args *args, void *stream);
+
 #ifdef __cplusplus
 }
 #endif
