@@ -179,11 +179,27 @@ __device__ __forceinline__ float fast_reciprocal(const float x) {
   return y;
 }
 
-template <bool kWindow>
+// kCausal: plain softmax over every earlier key.  kWindow: window attention with the running row maximum.
+// kCapped: window attention whose scores a soft cap keeps inside +-kMaxCap in base-2 units: F32 sums and BF16
+// probabilities hold 2^score as it is, so there is no row maximum, no reference and no rescaling of O.
+enum class Form { kCausal, kWindow, kCapped };
+constexpr float kMaxCap = 100.0F;
+
+// tanh for |x| <= 1/2 by its Taylor series up to x^11 (the next term is below 5e-7), two at a time; cap is
+// multiplied in.
+constexpr float kSeriesLimit = 0.5F;
+__device__ __forceinline__ unsigned long long mul_f32x2(const unsigned long long a, const unsigned long long b) {
+  unsigned long long d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
+template <Form kForm>
 __global__ void __launch_bounds__(kThreads, 2)
 flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, bf16 *const output, const int rows,
                          const int total_keys, const int heads, const WindowParams w, int *const error_word) {
+  constexpr bool kWindow = kForm != Form::kCausal;
   extern __shared__ __align__(1024) unsigned char smem[];
   const std::uint32_t smem_base = smem_u32(smem);
   auto bar = [&](const int index) { return smem_base + kBarrierOffset + 8U * index; };
@@ -326,6 +342,7 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const unsigned long long scale_pair = pack_f32x2(scale_log2, scale_log2);
     float reference = -INFINITY, running_sum = 0.0F;
     float cap_log2 = 0.0F, score_scale = 0.0F;
+    unsigned long long ratio_pair = 0ULL, minus_log2e_pair = 0ULL, series[6] = {};
     const float *bias_row = nullptr;
     if constexpr (kWindow) {
       if (w.sink != 0) {  // the sink is a score of 0 without a value
@@ -338,6 +355,15 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       // with a cap: exponent of e^(2 s / cap) in base 2; without: the score in base 2
       score_scale = w.softcap > 0.0F ? w.scale * 2.0F * kLog2e / w.softcap : w.scale * kLog2e;
       // (rows past the last query compute on table entries inside the table and are not stored)
+      if constexpr (kForm == Form::kCapped) {
+        running_sum = w.sink != 0 ? 1.0F : 0.0F;
+        const float ratio = w.scale / w.softcap;
+        ratio_pair = pack_f32x2(ratio, ratio);
+        minus_log2e_pair = pack_f32x2(-kLog2e, -kLog2e);
+        const float coefficients[6] = {1.0F, -1.0F / 3.0F, 2.0F / 15.0F, -17.0F / 315.0F, 62.0F / 2835.0F, -1382.0F / 155925.0F};
+#pragma unroll
+        for (int i = 0; i < 6; ++i) series[i] = pack_f32x2(cap_log2 * coefficients[i], cap_log2 * coefficients[i]);
+      }
       if (w.distance_bias != nullptr) bias_row = w.distance_bias + head * w.bias_stride + min(position, total_keys - 1);
     }
     bool ok = true;
@@ -358,78 +384,157 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) v[i] = chunk[i / 32][i % 32];
       }
-      if constexpr (kWindow) {
+      std::uint32_t packed[kKeys / 2];
+      bool moved = false;
+      float alpha = 1.0F;
+      if constexpr (kForm == Form::kCapped) {
         const int key0 = first_key(j);
         const bool partial = key0 + kKeys - 1 > prefix + q0 ||
                              (w.window > 0 && prefix + q0 + kRows - 1 - key0 >= w.window && key0 + kKeys > w.keep_first);
-        if (w.softcap > 0.0F) {
+        const int distance0 = min(position, total_keys - 1) - key0;
+        const float *const bias = bias_row - key0;
+        unsigned long long partial_sum[2] = {0ULL, 0ULL};
 #pragma unroll
-          for (int i = 0; i < kKeys; ++i) {
-            const float e = fast_exp2(__uint_as_float(v[i]) * score_scale);
-            v[i] = __float_as_uint(fmaf(-2.0F * cap_log2, fast_reciprocal(e + 1.0F), cap_log2));  // cap tanh(s / cap)
-          }
-        } else {
+        for (int part = 0; part < kKeys; part += 16) {
+          float lowered[16];  // what the distance takes off
+          if (bias_row == nullptr) {
 #pragma unroll
-          for (int i = 0; i < kKeys; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * score_scale);
-        }
-        if (bias_row != nullptr) {
-          const int distance0 = min(position, total_keys - 1) - key0;
-          const float *const bias = bias_row - key0;
-          if (partial) {
+            for (int i = 0; i < 16; ++i) lowered[i] = 0.0F;
+          } else if (partial) {
 #pragma unroll
-            for (int i = 0; i < kKeys; ++i)
-              v[i] = __float_as_uint(fmaf(-kLog2e, __ldg(bias - min(i, distance0)), __uint_as_float(v[i])));
+            for (int i = 0; i < 16; ++i) lowered[i] = __ldg(bias - min(part + i, distance0));
           } else {
 #pragma unroll
-            for (int i = 0; i < kKeys; ++i)
-              v[i] = __float_as_uint(fmaf(-kLog2e, __ldg(bias - i), __uint_as_float(v[i])));
+            for (int i = 0; i < 16; ++i) lowered[i] = __ldg(bias - (part + i));
+          }
+          unsigned long long x[8];
+          float largest = 0.0F;
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            float low, high;
+            x[i] = mul_f32x2(pack_f32x2(__uint_as_float(v[part + 2 * i]), __uint_as_float(v[part + 2 * i + 1])), ratio_pair);
+            unpack_f32x2(x[i], low, high);
+            largest = max3(largest, fabsf(low), fabsf(high));
+          }
+          unsigned long long t[8];
+          if (__any_sync(0xffffffffU, largest > kSeriesLimit)) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              float y[2];
+              unpack_f32x2(x[i], y[0], y[1]);
+#pragma unroll
+              for (int h = 0; h < 2; ++h) {
+                const float e = fast_exp2(y[h] * (2.0F * kLog2e));  // e^(2x)
+                y[h] = fmaf(-2.0F * cap_log2, fast_reciprocal(e + 1.0F), cap_log2);
+              }
+              t[i] = pack_f32x2(y[0], y[1]);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              const unsigned long long square = mul_f32x2(x[i], x[i]);
+              unsigned long long y = fma_f32x2(square, series[5], series[4]);
+              y = fma_f32x2(y, square, series[3]);
+              y = fma_f32x2(y, square, series[2]);
+              y = fma_f32x2(y, square, series[1]);
+              y = fma_f32x2(y, square, series[0]);
+              t[i] = mul_f32x2(y, x[i]);
+            }
+          }
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            float p[2];
+            unpack_f32x2(fma_f32x2(pack_f32x2(lowered[2 * i], lowered[2 * i + 1]), minus_log2e_pair, t[i]), p[0], p[1]);
+            p[0] = fast_exp2(p[0]);
+            p[1] = fast_exp2(p[1]);
+            if (partial) {
+#pragma unroll
+              for (int h = 0; h < 2; ++h) {
+                const int key = key0 + part + 2 * i + h;
+                const bool seen = key <= position && (w.window == 0 || position - key < w.window || key < w.keep_first);
+                if (!seen) p[h] = 0.0F;
+              }
+            }
+            partial_sum[i % 2] = add_f32x2(partial_sum[i % 2], pack_f32x2(p[0], p[1]));
+            packed[part / 2 + i] = round_pair_bf16(p[0], p[1]);
           }
         }
-        if (partial) {
+        float even, odd;
+        unpack_f32x2(add_f32x2(partial_sum[0], partial_sum[1]), even, odd);
+        running_sum += even + odd;
+      } else {
+        if constexpr (kWindow) {
+          const int key0 = first_key(j);
+          const bool partial = key0 + kKeys - 1 > prefix + q0 ||
+                               (w.window > 0 && prefix + q0 + kRows - 1 - key0 >= w.window && key0 + kKeys > w.keep_first);
+          if (w.softcap > 0.0F) {
 #pragma unroll
-          for (int i = 0; i < kKeys; ++i) {
-            const int key = key0 + i;
-            const bool seen = key <= position && (w.window == 0 || position - key < w.window || key < w.keep_first);
-            if (!seen) v[i] = 0xff800000U;  // -inf
+            for (int i = 0; i < kKeys; ++i) {
+              const float e = fast_exp2(__uint_as_float(v[i]) * score_scale);
+              v[i] = __float_as_uint(fmaf(-2.0F * cap_log2, fast_reciprocal(e + 1.0F), cap_log2));  // cap tanh(s / cap)
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < kKeys; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * score_scale);
           }
+          if (bias_row != nullptr) {
+            const int distance0 = min(position, total_keys - 1) - key0;
+            const float *const bias = bias_row - key0;
+            if (partial) {
+#pragma unroll
+              for (int i = 0; i < kKeys; ++i)
+                v[i] = __float_as_uint(fmaf(-kLog2e, __ldg(bias - min(i, distance0)), __uint_as_float(v[i])));
+            } else {
+#pragma unroll
+              for (int i = 0; i < kKeys; ++i)
+                v[i] = __float_as_uint(fmaf(-kLog2e, __ldg(bias - i), __uint_as_float(v[i])));
+            }
+          }
+          if (partial) {
+#pragma unroll
+            for (int i = 0; i < kKeys; ++i) {
+              const int key = key0 + i;
+              const bool seen = key <= position && (w.window == 0 || position - key < w.window || key < w.keep_first);
+              if (!seen) v[i] = 0xff800000U;  // -inf
+            }
+          }
+        } else if (j * kKeys + kKeys - 1 > prefix + q0) {     // some key hidden from some row
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i)
+            if (j * kKeys + i > position) v[i] = 0xff800000U;  // -inf
         }
-      } else if (j * kKeys + kKeys - 1 > prefix + q0) {     // some key hidden from some row
+        float partial_max[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-        for (int i = 0; i < kKeys; ++i)
-          if (j * kKeys + i > position) v[i] = 0xff800000U;  // -inf
+        for (int i = 0; i < kKeys; i += 2)
+          partial_max[(i / 2) % 4] = max3(partial_max[(i / 2) % 4], __uint_as_float(v[i]), __uint_as_float(v[i + 1]));
+        const float tile_max = fmaxf(fmaxf(partial_max[0], partial_max[1]), fmaxf(partial_max[2], partial_max[3]));
+        moved = tile_max > reference + slack;  // true on the first tile: reference = -inf
+        alpha = moved ? fast_exp2((reference - tile_max) * scale_log2) : 1.0F;
+        if (moved) reference = tile_max;
+        const float bias = -reference * scale_log2;
+        const unsigned long long bias_pair = pack_f32x2(bias, bias);
+        // probabilities and the row sum first: they need nothing from the previous tile's P V
+        unsigned long long partial_sum[4] = {0ULL, 0ULL, 0ULL, 0ULL};  // (even key, odd key) pairs of F32 sums
+        // in three sweeps, so that no instruction waits for the one before it
+        float t[kKeys];
+#pragma unroll
+        for (int i = 0; i < kKeys; i += 2)
+          unpack_f32x2(fma_f32x2(pack_f32x2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), scale_pair, bias_pair),
+                       t[i], t[i + 1]);
+#pragma unroll
+        for (int i = 0; i < kKeys; ++i) t[i] = fast_exp2(t[i]);
+#pragma unroll
+        for (int i = 0; i < kKeys; i += 2) {
+          partial_sum[(i / 2) % 4] = add_f32x2(partial_sum[(i / 2) % 4], pack_f32x2(t[i], t[i + 1]));
+          packed[i / 2] = round_pair_bf16(t[i], t[i + 1]);
+        }
+        partial_sum[0] = add_f32x2(partial_sum[0], partial_sum[2]);
+        partial_sum[1] = add_f32x2(partial_sum[1], partial_sum[3]);
+        float sum_even, sum_odd, sum_even_b, sum_odd_b;
+        unpack_f32x2(partial_sum[0], sum_even, sum_odd);
+        unpack_f32x2(partial_sum[1], sum_even_b, sum_odd_b);
+        running_sum = fmaf(running_sum, alpha, (sum_even + sum_odd) + (sum_even_b + sum_odd_b));
       }
-      float partial_max[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-#pragma unroll
-      for (int i = 0; i < kKeys; i += 2)
-        partial_max[(i / 2) % 4] = max3(partial_max[(i / 2) % 4], __uint_as_float(v[i]), __uint_as_float(v[i + 1]));
-      const float tile_max = fmaxf(fmaxf(partial_max[0], partial_max[1]), fmaxf(partial_max[2], partial_max[3]));
-      const bool moved = tile_max > reference + slack;  // true on the first tile: reference = -inf
-      const float alpha = moved ? fast_exp2((reference - tile_max) * scale_log2) : 1.0F;
-      if (moved) reference = tile_max;
-      const float bias = -reference * scale_log2;
-      const unsigned long long bias_pair = pack_f32x2(bias, bias);
-      // probabilities and the row sum first: they need nothing from the previous tile's P V
-      unsigned long long partial_sum[4] = {0ULL, 0ULL, 0ULL, 0ULL};  // (even key, odd key) pairs of F32 sums
-      std::uint32_t packed[kKeys / 2];
-      // in three sweeps, so that no instruction waits for the one before it
-      float t[kKeys];
-#pragma unroll
-      for (int i = 0; i < kKeys; i += 2)
-        unpack_f32x2(fma_f32x2(pack_f32x2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), scale_pair, bias_pair),
-                     t[i], t[i + 1]);
-#pragma unroll
-      for (int i = 0; i < kKeys; ++i) t[i] = fast_exp2(t[i]);
-#pragma unroll
-      for (int i = 0; i < kKeys; i += 2) {
-        partial_sum[(i / 2) % 4] = add_f32x2(partial_sum[(i / 2) % 4], pack_f32x2(t[i], t[i + 1]));
-        packed[i / 2] = round_pair_bf16(t[i], t[i + 1]);
-      }
-      partial_sum[0] = add_f32x2(partial_sum[0], partial_sum[2]);
-      partial_sum[1] = add_f32x2(partial_sum[1], partial_sum[3]);
-      float sum_even, sum_odd, sum_even_b, sum_odd_b;
-      unpack_f32x2(partial_sum[0], sum_even, sum_odd);
-      unpack_f32x2(partial_sum[1], sum_even_b, sum_odd_b);
-      running_sum = fmaf(running_sum, alpha, (sum_even + sum_odd) + (sum_even_b + sum_odd_b));
       if (j > 0) {
         // Every warp follows the O-ready barrier tile by tile, whether it has to rescale or not: a parity
         // wait cannot tell a phase from the one two before or two after it, so a waiter that skipped
@@ -442,7 +547,7 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           break;
         }
         tc_fence_after();
-        if (__any_sync(0xffffffffU, moved)) {
+        if (kForm != Form::kCapped && __any_sync(0xffffffffU, moved)) {
 #pragma unroll
           for (int c = 0; c < kRows / 16; ++c) {
             std::uint32_t o[16];
@@ -542,13 +647,13 @@ int flash_tcgen05_attention_k64(const void *query, const void *key_cache, const 
       (status = tc::make_bf16_tile_map(&map_k, key_cache, total_keys, width, kKeys)) != kOk ||
       (status = tc::make_bf16_tile_map(&map_v, value_cache, total_keys, width, kKeys)) != kOk)
     return status;
-  if (cudaFuncSetAttribute(flash_tcgen05_k64_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+  if (cudaFuncSetAttribute(flash_tcgen05_k64_kernel<Form::kCausal>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                            kSmemBytes) != cudaSuccess ||
-      cudaFuncSetAttribute(flash_tcgen05_k64_kernel<false>, cudaFuncAttributePreferredSharedMemoryCarveout,
+      cudaFuncSetAttribute(flash_tcgen05_k64_kernel<Form::kCausal>, cudaFuncAttributePreferredSharedMemoryCarveout,
                            cudaSharedmemCarveoutMaxShared) != cudaSuccess)
     return fail(kCuda, "cannot raise the attention shared-memory limit");
   const dim3 grid(ceil_div_u(rows, kRows), static_cast<unsigned int>(heads));
-  flash_tcgen05_k64_kernel<false><<<grid, kThreads, kSmemBytes, stream>>>(
+  flash_tcgen05_k64_kernel<Form::kCausal><<<grid, kThreads, kSmemBytes, stream>>>(
       map_q, map_k, map_v, static_cast<bf16 *>(output), static_cast<int>(rows), static_cast<int>(total_keys),
       static_cast<int>(heads), WindowParams{}, error);
   return check_launch("tcgen05 attention kernel (64-key tiles)");
@@ -571,10 +676,11 @@ int window_attention_tcgen05(const WindowAttentionArgs &a, cudaStream_t stream) 
       (status = tc::make_bf16_head_map(&map_k, a.key_cache, total_keys, a.kv_heads, a.dim, kKeys)) != kOk ||
       (status = tc::make_bf16_head_map(&map_v, a.value_cache, total_keys, a.kv_heads, a.value_dim, kKeys)) != kOk)
     return status;
-  if (cudaFuncSetAttribute(flash_tcgen05_k64_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
-          cudaSuccess ||
-      cudaFuncSetAttribute(flash_tcgen05_k64_kernel<true>, cudaFuncAttributePreferredSharedMemoryCarveout,
-                           cudaSharedmemCarveoutMaxShared) != cudaSuccess)
+  const bool capped = a.softcap > 0.0F && a.softcap * 1.4426950408889634F <= kMaxCap;
+  const auto kernel = capped ? flash_tcgen05_k64_kernel<Form::kCapped> : flash_tcgen05_k64_kernel<Form::kWindow>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) != cudaSuccess ||
+      cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared) !=
+          cudaSuccess)
     return fail(kCuda, "cannot raise the attention shared-memory limit");
   WindowParams w{};
   w.kv_heads = static_cast<int>(a.kv_heads);
@@ -590,7 +696,7 @@ int window_attention_tcgen05(const WindowAttentionArgs &a, cudaStream_t stream) 
   w.gate_stride = a.gate_stride;
   w.sink = a.sink ? 1 : 0;
   const dim3 grid(ceil_div_u(a.rows, kRows), static_cast<unsigned int>(a.heads));
-  flash_tcgen05_k64_kernel<true><<<grid, kThreads, kSmemBytes, stream>>>(
+  kernel<<<grid, kThreads, kSmemBytes, stream>>>(
       map_q, map_k, map_v, static_cast<bf16 *>(a.output), static_cast<int>(a.rows), static_cast<int>(total_keys),
       static_cast<int>(a.heads), w, error);
   return check_launch("tcgen05 window attention kernel");

@@ -2,7 +2,7 @@
 // delta rule (a scalar decay per head, values corrected by what the state already holds for the key).
 // Everything that enters the recurrences is F32.
 //
-// A prompt portion runs in three launches:
+// One token (cached decode) is one launch: decode_kernel.  A prompt portion runs in three:
 //   1. preparation: per token the decays and the queries / keys the recurrence reads (F32), for the delta
 //      rule also the short convolutions, the unit vectors, the step sizes, and the scalars of the blocked
 //      form below;
@@ -20,11 +20,14 @@
 //   S'  = G_3 S + sum_s D_3s k_s u_s^T
 // so the eight products with S are taken at once and summed over the lanes together; the scalars
 // depend on the head only and come from the preparation.
+#include <cooperative_groups.h>
+
 #include "decoder_types.cuh"
 #include "ops_internal.hpp"
 
 namespace evob {
 namespace {
+namespace cg = cooperative_groups;
 
 constexpr int kBlock = 4;              // tokens per block of the delta rule
 constexpr int kTile = 16;              // tokens per shared-memory tile
@@ -561,6 +564,196 @@ norm_gate_kernel(const float *__restrict__ input, const float *__restrict__ gain
     out[d] = from_float<T>(o[d] * factor * gain[d] * silu_f32(to_float(g[d])));
 }
 
+// ---------------------------------------------------------------- one token
+// A cluster of CTAs per key head: each owns a slice of the value columns of the heads that share the key, keeps
+// its part of the state in registers between the read-out and the update (a warp per set of channels, a lane
+// per column), and the output norm's sums meet in distributed shared memory.
+constexpr int kDecodeRanks = 8, kDecodeThreads = 256, kDecodeWarps = kDecodeThreads / 32;
+constexpr int kDecodeMaxGroup = 64;  // heads per key head
+
+struct DecodeParams {
+  int heads, kv_heads, dim, value_dim, taps, channels, rank;
+  int key_column, value_column, gate_column, beta_column, decay_column;
+  float inverse_tau, epsilon;
+  int fresh;
+};
+
+template <bool kDelta, typename T>
+__global__ void __launch_bounds__(kDecodeThreads)
+decode_kernel(const T *__restrict__ projection, T *const history, const float *__restrict__ conv,
+              const float *__restrict__ decay_rate, const float *__restrict__ decay_shift,
+              const float *__restrict__ decay_weight, const float *__restrict__ decay_bias,
+              const float *__restrict__ gain, float *const state, T *__restrict__ output, const DecodeParams p) {
+  // a one-row projection launched with programmatic stream serialisation may start under this kernel
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  __shared__ float key[kDecoderMaxHeadDim], query[kDecoderMaxHeadDim], alpha[kDecoderMaxHeadDim];
+  __shared__ float partial[2][kDecodeWarps][32], scratch[kDecodeWarps];
+  __shared__ float squares[kDecodeMaxGroup];  // this CTA's part of every head's sum of squares
+  extern __shared__ float outputs[];          // this CTA's columns
+  cg::cluster_group cluster = cg::this_cluster();
+  const int rank = static_cast<int>(cluster.block_rank()), g = blockIdx.y;
+  const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+  const int group = kDelta ? p.heads / p.kv_heads : 1;
+  const int columns = group * p.value_dim, share = (columns + kDecodeRanks - 1) / kDecodeRanks;
+  const int begin = rank * share, count = max(0, min(columns, begin + share) - begin);
+  const auto convolved = [&](const int column) {
+    return conv_silu(projection, 0, history, p.channels, conv, p.taps, p.fresh != 0, 0, column);
+  };
+  float k = 0.0F, q = 0.0F;
+  const int d = threadIdx.x;  // kDecodeThreads == kDecoderMaxHeadDim: a thread per key channel
+  if (d < p.dim) {
+    if constexpr (kDelta) {
+      k = convolved(p.key_column + g * p.dim + d);
+      q = convolved(g * p.dim + d);
+    } else {
+      const int channel = g * p.dim + d;
+      k = to_float(projection[p.key_column + channel]);
+      q = to_float(projection[channel]);
+      float z = decay_bias[channel];
+      for (int r = 0; r < p.rank; ++r)
+        z = fmaf(decay_weight[static_cast<std::size_t>(r) * p.heads * p.dim + channel], to_float(projection[p.beta_column + r]), z);
+      alpha[d] = expf(-softplus_f32(-z) * p.inverse_tau);
+    }
+  }
+  const float inverse_root = 1.0F / sqrtf(static_cast<float>(p.dim));
+  if constexpr (kDelta) {
+    k *= 1.0F / sqrtf(block_sum<kDecodeThreads>(k * k, scratch) + 1e-6F);
+    q *= 1.0F / sqrtf(block_sum<kDecodeThreads>(q * q, scratch) + 1e-6F);
+  }
+  q *= inverse_root;
+  if (d < p.dim) {
+    key[d] = k;
+    query[d] = q;
+  }
+  const float key_query = block_sum<kDecodeThreads>(k * q, scratch);  // (its barriers also publish key and query)
+  constexpr int kHeld = static_cast<int>(kDecoderMaxHeadDim) / kDecodeWarps;
+  for (int c0 = 0; c0 < count; c0 += 32) {
+    const int c = begin + c0 + lane;
+    const bool live = c0 + lane < count;
+    const int head = g * group + (live ? c / p.value_dim : 0), column = live ? c % p.value_dim : 0;
+    float *const cells = state + static_cast<std::size_t>(head) * p.dim * p.value_dim + column;
+    float v = 0.0F, beta = 0.0F, decay = 1.0F;
+    if (live) {
+      if constexpr (kDelta) {
+        v = convolved(p.value_column + head * p.value_dim + column);
+        v = to_float(from_float<T>(v));  // the prompt's kernels keep convolved values in the activation type
+        beta = sigmoid_f32(to_float(projection[p.beta_column + head]));
+        decay = expf(decay_rate[head] * softplus_f32(to_float(projection[p.decay_column + head]) + decay_shift[head]));
+      } else {
+        v = to_float(projection[p.value_column + head * p.value_dim + column]);
+      }
+    }
+    float held[kHeld], with_key = 0.0F, with_query = 0.0F;
+#pragma unroll
+    for (int i = 0; i < kHeld; ++i) {
+      const int row = warp + kDecodeWarps * i;
+      held[i] = live && row < p.dim && p.fresh == 0 ? cells[static_cast<std::size_t>(row) * p.value_dim] : 0.0F;
+    }
+#pragma unroll
+    for (int i = 0; i < kHeld; ++i) {
+      const int row = warp + kDecodeWarps * i;
+      if (row < p.dim) {
+        if constexpr (kDelta) {
+          held[i] *= decay;
+          with_key = fmaf(held[i], key[row], with_key);
+        } else {
+          held[i] = fmaf(key[row], v, alpha[row] * held[i]);
+        }
+        with_query = fmaf(held[i], query[row], with_query);
+      }
+    }
+    partial[0][warp][lane] = with_key;
+    partial[1][warp][lane] = with_query;
+    __syncthreads();
+    with_key = with_query = 0.0F;
+#pragma unroll
+    for (int w = 0; w < kDecodeWarps; ++w) {
+      with_key += partial[0][w][lane];
+      with_query += partial[1][w][lane];
+    }
+    const float u = kDelta ? beta * (v - with_key) : 0.0F;
+    const float o = kDelta ? fmaf(u, key_query, with_query) : with_query;
+#pragma unroll
+    for (int i = 0; i < kHeld; ++i) {
+      const int row = warp + kDecodeWarps * i;
+      if (live && row < p.dim)
+        cells[static_cast<std::size_t>(row) * p.value_dim] = kDelta ? fmaf(key[row], u, held[i]) : held[i];
+    }
+    if (warp == 0 && live) outputs[c0 + lane] = o;
+    __syncthreads();
+  }
+  for (int local = 0; local < group; ++local) {
+    const int from = max(local * p.value_dim, begin) - begin, to = min((local + 1) * p.value_dim, begin + count) - begin;
+    float square = 0.0F;
+    if (from < to) {  // the same for every thread
+      for (int c = from + threadIdx.x; c < to; c += kDecodeThreads) square = fmaf(outputs[c], outputs[c], square);
+      square = block_sum<kDecodeThreads>(square, scratch);
+    }
+    if (threadIdx.x == 0) squares[local] = square;
+  }
+  cluster.sync();  // every part of the norms is there, and every CTA has read the history of the shared channels
+  for (int c = threadIdx.x; c < count; c += kDecodeThreads) {
+    const int local = (begin + c) / p.value_dim, column = (begin + c) % p.value_dim, head = g * group + local;
+    float total = 0.0F;
+    for (int r = 0; r < kDecodeRanks; ++r) total += cluster.map_shared_rank(squares, r)[local];
+    const float factor = 1.0F / sqrtf(total / static_cast<float>(p.value_dim) + p.epsilon);
+    const int at = head * p.value_dim + column;
+    output[at] = from_float<T>(outputs[c] * factor * gain[column] * silu_f32(to_float(projection[p.gate_column + at])));
+  }
+  if constexpr (kDelta) {
+    const auto advance = [&](const int column) {
+      for (int i = 0; i + 1 < p.taps; ++i)
+        history[static_cast<std::size_t>(i) * p.channels + column] =
+            i + 2 < p.taps ? (p.fresh == 0 ? history[static_cast<std::size_t>(i + 1) * p.channels + column] : from_float<T>(0.0F))
+                           : projection[column];
+    };
+    for (int c = threadIdx.x; c < count; c += kDecodeThreads) advance(p.value_column + g * columns + begin + c);
+    if (rank == 0 && d < p.dim) {
+      advance(g * p.dim + d);
+      advance(p.key_column + g * p.dim + d);
+    }
+  }
+  cluster.sync();  // remote shared memory stays alive until everybody has read it
+}
+
+template <bool kDelta, typename T>
+int launch_decode(const RecurrentArgs &a, cudaStream_t stream) {
+  DecodeParams p{};
+  p.heads = static_cast<int>(a.heads);
+  p.kv_heads = static_cast<int>(a.kv_heads);
+  p.dim = static_cast<int>(a.dim);
+  p.value_dim = static_cast<int>(a.value_dim);
+  p.taps = static_cast<int>(a.conv_taps);
+  p.channels = static_cast<int>(a.gate_column);
+  p.rank = static_cast<int>(a.decay_rank);
+  p.key_column = static_cast<int>(a.key_column);
+  p.value_column = static_cast<int>(a.value_column);
+  p.gate_column = static_cast<int>(a.gate_column);
+  p.beta_column = static_cast<int>(a.beta_column);
+  p.decay_column = static_cast<int>(a.decay_column);
+  p.inverse_tau = 1.0F / a.tau;
+  p.epsilon = a.epsilon;
+  p.fresh = a.fresh ? 1 : 0;
+  cudaLaunchAttribute attribute{};
+  attribute.id = cudaLaunchAttributeClusterDimension;
+  attribute.val.clusterDim.x = kDecodeRanks;
+  attribute.val.clusterDim.y = attribute.val.clusterDim.z = 1;
+  cudaLaunchConfig_t config{};
+  config.gridDim = dim3(kDecodeRanks, static_cast<unsigned int>(kDelta ? a.kv_heads : a.heads));
+  config.blockDim = dim3(kDecodeThreads);
+  const std::size_t columns = (kDelta ? a.heads / a.kv_heads : 1) * a.value_dim;
+  config.dynamicSmemBytes = (columns + kDecodeRanks - 1) / kDecodeRanks * sizeof(float);
+  config.stream = stream;
+  config.attrs = &attribute;
+  config.numAttrs = 1;
+  if (cudaLaunchKernelEx(&config, decode_kernel<kDelta, T>, static_cast<const T *>(a.projection),
+                         static_cast<T *>(a.conv_history), a.conv, a.decay_rate, a.decay_shift, a.decay_weight,
+                         a.decay_bias, a.output_norm, a.state, static_cast<T *>(a.output), p) != cudaSuccess)
+    return fail(kCuda, std::string("cannot launch the recurrent decode kernel: ") +
+                           cudaGetErrorString(cudaGetLastError()));
+  return check_launch("recurrent decode kernel");
+}
+
 template <bool kDelta, int kElements, typename T>
 int launch_recurrence(const float *queries, const float *keys, const float *alpha, const T *values,
                       const float *scalars, float *state, float *output, const RecurrenceParams &p,
@@ -672,6 +865,12 @@ int recurrent_mixer(const RecurrentArgs &a, cudaStream_t stream) {
                    !(a.tau > 0.0F)))
     return fail(kInvalidArgument, "linear attention arguments are invalid");
   if (a.rows == 0) return kOk;
+  const std::size_t decode_columns = (a.delta ? a.heads / a.kv_heads : 1) * a.value_dim;
+  if (a.rows == 1 && (!a.delta || a.heads / a.kv_heads <= static_cast<std::size_t>(kDecodeMaxGroup)) &&
+      decode_columns <= 8192 * static_cast<std::size_t>(kDecodeRanks)) {
+    if (a.type == Activation::kBf16) return a.delta ? launch_decode<true, bf16>(a, stream) : launch_decode<false, bf16>(a, stream);
+    return a.delta ? launch_decode<true, float>(a, stream) : launch_decode<false, float>(a, stream);
+  }
   return a.type == Activation::kBf16 ? run<bf16>(a, stream) : run<float>(a, stream);
 }
 

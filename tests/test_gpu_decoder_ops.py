@@ -184,7 +184,7 @@ def test_attention_tensor_cores(pkg, ops, dim, vdim, rows, position, window, kee
 
 
 @pytest.mark.parametrize("kernel", [ROW, TILE, TENSOR])
-@pytest.mark.parametrize("softcap, sink, gated, biased", [(0.0, 1, True, True), (3.0, 0, True, True), (15.0, 1, False, True),
+@pytest.mark.parametrize("softcap, sink, gated, biased", [(0.0, 1, True, True), (90.0, 1, True, True), (1.5, 1, True, True), (3.0, 0, True, True), (15.0, 1, False, True),
                                                            (15.0, 1, True, False), (0.0, 0, False, False)])
 def test_attention_options(pkg, ops, kernel, softcap, sink, gated, biased):
     out, expected = window_case(pkg, ops, rows=70, position=90, heads=4, kv_heads=1, dim=64, vdim=80, window=33, keep_first=2,
