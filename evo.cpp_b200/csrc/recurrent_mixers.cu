@@ -2,7 +2,8 @@
 // delta rule (a scalar decay per head, values corrected by what the state already holds for the key).
 // Everything that enters the recurrences is F32.
 //
-// One token (cached decode) is one launch: decode_kernel.  A prompt portion runs in three:
+// One token (cached decode) is one launch: decode_kernel.  BF16 prompt portions of 32 rows and more take the
+// tensor-core form (recurrent_chunks.cu); shorter ones, and the F32 profile, run in three launches:
 //   1. preparation: per token the decays and the queries / keys the recurrence reads (F32), for the delta
 //      rule also the short convolutions, the unit vectors, the step sizes, and the scalars of the blocked
 //      form below;
@@ -24,6 +25,7 @@
 
 #include "decoder_types.cuh"
 #include "ops_internal.hpp"
+#include "recurrent_chunks.hpp"
 
 namespace evob {
 namespace {
@@ -779,6 +781,30 @@ int dispatch_recurrence(const float *queries, const float *keys, const float *al
 }
 
 template <typename T>
+int advance_history(const RecurrentArgs &a, cudaStream_t stream) {
+  if (!a.delta || a.conv_taps <= 1) return kOk;
+  conv_history_kernel<T><<<ceil_div_u(a.gate_column, 256), 256, 0, stream>>>(
+      static_cast<const T *>(a.projection), a.stride, static_cast<T *>(a.conv_history), static_cast<int>(a.gate_column),
+      static_cast<int>(a.conv_taps) - 1, static_cast<int>(a.rows), a.fresh);
+  return check_launch("convolution history kernel");
+}
+
+template <typename T>
+int norm_gate(const RecurrentArgs &a, const float *input, cudaStream_t stream) {
+  norm_gate_kernel<T><<<ceil_div_u(a.rows * a.heads, 8), 256, 0, stream>>>(
+      input, a.output_norm, static_cast<const T *>(a.projection) + a.gate_column, a.stride, static_cast<int>(a.rows),
+      static_cast<int>(a.heads), static_cast<int>(a.value_dim), a.epsilon, static_cast<T *>(a.output));
+  return check_launch("output norm and gate kernel");
+}
+
+int run_chunks(const RecurrentArgs &a, cudaStream_t stream) {
+  float *output = nullptr;
+  int status = recurrent_chunks(a, &output, stream);
+  if (status == kOk) status = advance_history<bf16>(a, stream);
+  return status == kOk ? norm_gate<bf16>(a, output, stream) : status;
+}
+
+template <typename T>
 int run(const RecurrentArgs &a, cudaStream_t stream) {
   const Workspace w = workspace_layout(a.delta, a.rows, a.heads, a.kv_heads, a.dim, a.value_dim, a.type);
   unsigned char *const base = static_cast<unsigned char *>(a.workspace);
@@ -818,11 +844,7 @@ int run(const RecurrentArgs &a, cudaStream_t stream) {
         projection, static_cast<const T *>(a.conv_history), a.conv, a.decay_rate, a.decay_shift, queries, keys, values,
         scalars, d);
     if ((status = check_launch("delta preparation kernel")) != kOk) return status;
-    if (a.conv_taps > 1) {
-      conv_history_kernel<T><<<ceil_div_u(a.gate_column, 256), 256, 0, stream>>>(
-          projection, a.stride, static_cast<T *>(a.conv_history), d.channels, d.taps - 1, p.rows, a.fresh);
-      if ((status = check_launch("convolution history kernel")) != kOk) return status;
-    }
+    if ((status = advance_history<T>(a, stream)) != kOk) return status;
     p.value_stride = a.heads * a.value_dim;
     status = dispatch_recurrence<true, T>(queries, keys, nullptr, values, scalars, a.state, output, p, stream);
   } else {
@@ -838,10 +860,7 @@ int run(const RecurrentArgs &a, cudaStream_t stream) {
                                            stream);
   }
   if (status != kOk) return status;
-  norm_gate_kernel<T><<<ceil_div_u(a.rows * a.heads, 8), 256, 0, stream>>>(
-      output, a.output_norm, projection + a.gate_column, a.stride, p.rows, p.heads, p.value_dim, a.epsilon,
-      static_cast<T *>(a.output));
-  return check_launch("output norm and gate kernel");
+  return norm_gate<T>(a, output, stream);
 }
 
 }  // namespace
@@ -849,7 +868,9 @@ int run(const RecurrentArgs &a, cudaStream_t stream) {
 std::size_t recurrent_workspace_bytes(const bool delta, const std::size_t rows, const std::size_t heads,
                                       const std::size_t kv_heads, const std::size_t dim, const std::size_t value_dim,
                                       const Activation type) {
-  return workspace_layout(delta, rows, heads, kv_heads, dim, value_dim, type).bytes;
+  const std::size_t blocks = workspace_layout(delta, rows, heads, kv_heads, dim, value_dim, type).bytes;
+  const std::size_t chunks = recurrent_chunks_workspace(delta, rows, heads, kv_heads, dim, value_dim);
+  return blocks > chunks ? blocks : chunks;
 }
 
 int recurrent_mixer(const RecurrentArgs &a, cudaStream_t stream) {
@@ -871,6 +892,7 @@ int recurrent_mixer(const RecurrentArgs &a, cudaStream_t stream) {
     if (a.type == Activation::kBf16) return a.delta ? launch_decode<true, bf16>(a, stream) : launch_decode<false, bf16>(a, stream);
     return a.delta ? launch_decode<true, float>(a, stream) : launch_decode<false, float>(a, stream);
   }
+  if (recurrent_chunks_applicable(a)) return run_chunks(a, stream);
   return a.type == Activation::kBf16 ? run<bf16>(a, stream) : run<float>(a, stream);
 }
 
