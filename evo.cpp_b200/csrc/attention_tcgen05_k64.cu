@@ -343,6 +343,7 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     float reference = -INFINITY, running_sum = 0.0F;
     float cap_log2 = 0.0F, score_scale = 0.0F;
     unsigned long long ratio_pair = 0ULL, minus_log2e_pair = 0ULL, series[6] = {};
+    float series_scale = 0.0F;
     const float *bias_row = nullptr;
     if constexpr (kWindow) {
       if (w.sink != 0) {  // the sink is a score of 0 without a value
@@ -359,6 +360,7 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         running_sum = w.sink != 0 ? 1.0F : 0.0F;
         const float ratio = w.scale / w.softcap;
         ratio_pair = pack_f32x2(ratio, ratio);
+        series_scale = fabsf(ratio);
         minus_log2e_pair = pack_f32x2(-kLog2e, -kLog2e);
         const float coefficients[6] = {1.0F, -1.0F / 3.0F, 2.0F / 15.0F, -17.0F / 315.0F, 62.0F / 2835.0F, -1382.0F / 155925.0F};
 #pragma unroll
@@ -370,6 +372,31 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 
     for (int j = 0; j < tiles; ++j) {
       const int s = j & 1;
+      // capped form: what the distance takes off, infinity for a key that the row does not see; fetched while the
+      // scores are still being multiplied
+      float lowered[kForm == Form::kCapped ? kKeys : 1];
+      if constexpr (kForm == Form::kCapped) {
+        const int key0 = first_key(j);
+        const bool partial = key0 + kKeys - 1 > prefix + q0 ||
+                             (w.window > 0 && prefix + q0 + kRows - 1 - key0 >= w.window && key0 + kKeys > w.keep_first);
+        const float *const bias = bias_row - key0;
+        if (partial) {
+          // seen: key <= position, and in the window or kept
+          const int own = position - key0, oldest = w.window > 0 ? own - w.window : -1, kept = w.keep_first - key0;
+          const int distance0 = min(position, total_keys - 1) - key0;
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) {
+            const float value = bias_row != nullptr ? __ldg(bias - min(i, distance0)) : 0.0F;
+            lowered[i] = i <= own && (i > oldest || i < kept) ? value : INFINITY;
+          }
+        } else if (bias_row != nullptr) {
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) lowered[i] = __ldg(bias - i);
+        } else {
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) lowered[i] = 0.0F;
+        }
+      }
       if (!mbar_wait(bar(kSFull + s), (j >> 1) & 1U, abort_flag)) {
         ok = false;
         break;
@@ -388,75 +415,43 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       bool moved = false;
       float alpha = 1.0F;
       if constexpr (kForm == Form::kCapped) {
-        const int key0 = first_key(j);
-        const bool partial = key0 + kKeys - 1 > prefix + q0 ||
-                             (w.window > 0 && prefix + q0 + kRows - 1 - key0 >= w.window && key0 + kKeys > w.keep_first);
-        const int distance0 = min(position, total_keys - 1) - key0;
-        const float *const bias = bias_row - key0;
         unsigned long long partial_sum[2] = {0ULL, 0ULL};
+        float largest[4] = {};
 #pragma unroll
-        for (int part = 0; part < kKeys; part += 16) {
-          float lowered[16];  // what the distance takes off
-          if (bias_row == nullptr) {
+        for (int i = 0; i < kKeys; i += 2)
+          largest[(i / 2) % 4] = max3(largest[(i / 2) % 4], fabsf(__uint_as_float(v[i])), fabsf(__uint_as_float(v[i + 1])));
+        const bool wide = fmaxf(fmaxf(largest[0], largest[1]), fmaxf(largest[2], largest[3])) * series_scale > kSeriesLimit;
+        const auto finish = [&](const int i, const unsigned long long capped) {
+          float low, high;
+          unpack_f32x2(fma_f32x2(pack_f32x2(lowered[i], lowered[i + 1]), minus_log2e_pair, capped), low, high);
+          low = fast_exp2(low);
+          high = fast_exp2(high);
+          partial_sum[(i / 2) % 2] = add_f32x2(partial_sum[(i / 2) % 2], pack_f32x2(low, high));
+          packed[i / 2] = round_pair_bf16(low, high);
+        };
+        if (__any_sync(0xffffffffU, wide)) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) lowered[i] = 0.0F;
-          } else if (partial) {
+          for (int i = 0; i < kKeys; i += 2) {
+            float y[2];
 #pragma unroll
-            for (int i = 0; i < 16; ++i) lowered[i] = __ldg(bias - min(part + i, distance0));
-          } else {
-#pragma unroll
-            for (int i = 0; i < 16; ++i) lowered[i] = __ldg(bias - (part + i));
-          }
-          unsigned long long x[8];
-          float largest = 0.0F;
-#pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            float low, high;
-            x[i] = mul_f32x2(pack_f32x2(__uint_as_float(v[part + 2 * i]), __uint_as_float(v[part + 2 * i + 1])), ratio_pair);
-            unpack_f32x2(x[i], low, high);
-            largest = max3(largest, fabsf(low), fabsf(high));
-          }
-          unsigned long long t[8];
-          if (__any_sync(0xffffffffU, largest > kSeriesLimit)) {
-#pragma unroll
-            for (int i = 0; i < 8; ++i) {
-              float y[2];
-              unpack_f32x2(x[i], y[0], y[1]);
-#pragma unroll
-              for (int h = 0; h < 2; ++h) {
-                const float e = fast_exp2(y[h] * (2.0F * kLog2e));  // e^(2x)
-                y[h] = fmaf(-2.0F * cap_log2, fast_reciprocal(e + 1.0F), cap_log2);
-              }
-              t[i] = pack_f32x2(y[0], y[1]);
+            for (int h = 0; h < 2; ++h) {
+              const float e = fast_exp2(__uint_as_float(v[i + h]) * score_scale);  // e^(2 s / cap)
+              y[h] = fmaf(-2.0F * cap_log2, fast_reciprocal(e + 1.0F), cap_log2);
             }
-          } else {
-#pragma unroll
-            for (int i = 0; i < 8; ++i) {
-              const unsigned long long square = mul_f32x2(x[i], x[i]);
-              unsigned long long y = fma_f32x2(square, series[5], series[4]);
-              y = fma_f32x2(y, square, series[3]);
-              y = fma_f32x2(y, square, series[2]);
-              y = fma_f32x2(y, square, series[1]);
-              y = fma_f32x2(y, square, series[0]);
-              t[i] = mul_f32x2(y, x[i]);
-            }
+            finish(i, pack_f32x2(y[0], y[1]));
           }
+        } else {
 #pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            float p[2];
-            unpack_f32x2(fma_f32x2(pack_f32x2(lowered[2 * i], lowered[2 * i + 1]), minus_log2e_pair, t[i]), p[0], p[1]);
-            p[0] = fast_exp2(p[0]);
-            p[1] = fast_exp2(p[1]);
-            if (partial) {
-#pragma unroll
-              for (int h = 0; h < 2; ++h) {
-                const int key = key0 + part + 2 * i + h;
-                const bool seen = key <= position && (w.window == 0 || position - key < w.window || key < w.keep_first);
-                if (!seen) p[h] = 0.0F;
-              }
-            }
-            partial_sum[i % 2] = add_f32x2(partial_sum[i % 2], pack_f32x2(p[0], p[1]));
-            packed[part / 2 + i] = round_pair_bf16(p[0], p[1]);
+          for (int i = 0; i < kKeys; i += 2) {
+            const unsigned long long x =
+                mul_f32x2(pack_f32x2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), ratio_pair);
+            const unsigned long long square = mul_f32x2(x, x);
+            unsigned long long y = fma_f32x2(square, series[5], series[4]);
+            y = fma_f32x2(y, square, series[3]);
+            y = fma_f32x2(y, square, series[2]);
+            y = fma_f32x2(y, square, series[1]);
+            y = fma_f32x2(y, square, series[0]);
+            finish(i, mul_f32x2(y, x));
           }
         }
         float even, odd;

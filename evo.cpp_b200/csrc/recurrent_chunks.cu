@@ -77,15 +77,15 @@ __device__ __forceinline__ void convolve_chunk(const T *const projection, const 
 }
 
 template <int kTaps, typename T>
-__global__ void __launch_bounds__(kPrepThreads)
+__global__ void __launch_bounds__(kPrepThreads, 2)
 delta_chunks_kernel(const T *__restrict__ projection, const T *__restrict__ history, const float *__restrict__ conv,
                     const float *__restrict__ decay_rate, const float *__restrict__ decay_shift,
                     float *__restrict__ queries, float *__restrict__ keys, T *__restrict__ values,
                     float *__restrict__ matrices, const DeltaParams p) {
-  extern __shared__ float smem[];  // keys [16][dim + 1], queries [16][dim + 1], then decay products per slot of heads
+  extern __shared__ __align__(16) float smem[];  // per slot of heads two 16 x 16 matrices, then keys and queries [16][dim + 1]
   const int stride = p.dim + 1;
-  float *const ks = smem, *const qs = ks + kChunk * stride;
-  float *const heads_base = qs + kChunk * stride;
+  float *const heads_base = smem;
+  float *const ks = heads_base + kPrepThreads / kChunk * 2 * kChunk * kMatrixStride, *const qs = ks + kChunk * stride;
   __shared__ float kk[kChunk][kChunk + 1], kq[kChunk][kChunk + 1];  // [t][s]
   const int chunk = blockIdx.x, g = blockIdx.y, row0 = chunk * kChunk;
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
@@ -125,10 +125,11 @@ delta_chunks_kernel(const T *__restrict__ projection, const T *__restrict__ hist
   }
   __syncthreads();
   // inner products: one (t, s) pair per thread
-  for (int item = threadIdx.x; item < kChunk * kChunk; item += kPrepThreads) {
-    const int t = item / kChunk, s = item % kChunk;
+  {
+    const int t = threadIdx.x / kChunk, s = threadIdx.x % kChunk;
     float a = 0.0F, b = 0.0F;
     if (s <= t) {
+#pragma unroll 4
       for (int d = 0; d < p.dim; ++d) {
         const float k = ks[s * stride + d];
         a = fmaf(k, ks[t * stride + d], a);
@@ -139,11 +140,12 @@ delta_chunks_kernel(const T *__restrict__ projection, const T *__restrict__ hist
     kq[t][s] = b;
   }
   __syncthreads();
-  // heads that share the key: 16 threads each, thread j owns column j of the inverse
-  const int j = threadIdx.x % kChunk, slot = threadIdx.x / kChunk;
+  // heads that share the key, two per warp: thread j of sixteen owns column j of the inverse
+  const int j = lane % kChunk, slot = threadIdx.x / kChunk;
   constexpr int kSlots = kPrepThreads / kChunk;
-  float *const decay = heads_base + slot * (kChunk * (kChunk + 1));  // D [t][s]
-  for (int first = 0; first < group; first += kSlots) {
+  float *const below = heads_base + slot * (2 * kChunk * kMatrixStride);  // A [t][s], rows of whole 16-byte words
+  float *const reads = below + kChunk * kMatrixStride;                    // D (k.q) [t][s]
+  for (int first = 0; first + 2 * warp < group; first += kSlots) {
     const int local = first + slot, head = g * group + local;
     const bool live = local < group;
     float gate = 1.0F, beta = 0.0F;  // of token j
@@ -152,43 +154,52 @@ delta_chunks_kernel(const T *__restrict__ projection, const T *__restrict__ hist
       beta = sigmoid_f32(to_float(source[p.beta_column + head]));
       gate = expf(decay_rate[head] * softplus_f32(to_float(source[p.decay_column + head]) + decay_shift[head]));
     }
-    float product = 1.0F, cumulative = 1.0F, last_decay = 1.0F;
-    const unsigned int half = 0xffffffffU;
-    float betas[kChunk];
+    float product = 1.0F, cumulative = 1.0F;
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      const float g_t = __shfl_sync(half, gate, t, kChunk);
-      betas[t] = __shfl_sync(half, beta, t, kChunk);
+      const float g_t = __shfl_sync(0xffffffffU, gate, t, kChunk), beta_t = __shfl_sync(0xffffffffU, beta, t, kChunk);
       if (t > j) product *= g_t;      // D_tj
       if (t <= j) cumulative *= g_t;  // G_j
-      decay[t * (kChunk + 1) + j] = t >= j ? product : 0.0F;
+      below[t * kMatrixStride + j] = t > j ? beta_t * product * kk[t][j] : 0.0F;
+      reads[t * kMatrixStride + j] = t >= j ? product * kq[t][j] : 0.0F;
     }
-    last_decay = product;  // D_15,j
+    const float last_decay = product;  // D_15,j
     __syncwarp();
+    const auto row_of = [](const float *const matrix, const int t, float (&v)[kChunk]) {
+      load_floats<kChunk>(matrix + t * kMatrixStride, v);
+    };
     float column[kChunk];  // N_tj
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      float x = t == j ? 1.0F : 0.0F;
+      float row[kChunk], x[2] = {t == j ? 1.0F : 0.0F, 0.0F};
+      row_of(below, t, row);
 #pragma unroll
-      for (int s = 0; s < t; ++s) x = fmaf(-betas[t] * decay[t * (kChunk + 1) + s] * kk[t][s], column[s], x);
-      column[t] = x;
+      for (int s = 0; s < t; ++s) x[s % 2] = fmaf(-row[s], column[s], x[s % 2]);
+      column[t] = x[0] + x[1];
     }
     float *const out = matrices + (static_cast<std::size_t>(chunk) * p.heads + head) * kDeltaFloats;
+    float updates[kChunk], readouts[kChunk];
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      const float tail = __shfl_sync(half, last_decay, t, kChunk);  // D_15,t
-      if (live) out[j * kMatrixStride + t] = tail * column[t];
-      float x = 0.0F;
+      updates[t] = __shfl_sync(0xffffffffU, last_decay, t, kChunk) * column[t];  // D_15,t N_tj
+      float row[kChunk], x[2] = {0.0F, 0.0F};
+      row_of(reads, t, row);
 #pragma unroll
-      for (int r = 0; r <= t; ++r) x = fmaf(decay[t * (kChunk + 1) + r] * kq[t][r], column[r], x);
-      if (live) out[kMatrix + j * kMatrixStride + t] = x;
+      for (int r = 0; r <= t; ++r) x[r % 2] = fmaf(row[r], column[r], x[r % 2]);
+      readouts[t] = x[0] + x[1];
     }
     if (live) {
+#pragma unroll
+      for (int t = 0; t < kChunk; t += 4) {
+        *reinterpret_cast<float4 *>(out + j * kMatrixStride + t) = make_float4(updates[t], updates[t + 1], updates[t + 2], updates[t + 3]);
+        *reinterpret_cast<float4 *>(out + kMatrix + j * kMatrixStride + t) =
+            make_float4(readouts[t], readouts[t + 1], readouts[t + 2], readouts[t + 3]);
+      }
+      *reinterpret_cast<float4 *>(out + j * kMatrixStride + kChunk) = make_float4(0.0F, 0.0F, 0.0F, 0.0F);
+      *reinterpret_cast<float4 *>(out + kMatrix + j * kMatrixStride + kChunk) = make_float4(0.0F, 0.0F, 0.0F, 0.0F);
       out[2 * kMatrix + j] = beta;
       out[2 * kMatrix + kChunk + j] = beta * cumulative;
       out[2 * kMatrix + 2 * kChunk + j] = cumulative;
-#pragma unroll
-      for (int t = kChunk; t < kMatrixStride; ++t) out[j * kMatrixStride + t] = out[kMatrix + j * kMatrixStride + t] = 0.0F;
     }
     __syncwarp();
   }
@@ -289,9 +300,10 @@ linear_chunks_kernel(const T *__restrict__ projection, const std::size_t stride,
 struct Split {
   std::uint32_t big, small;
 };
+// big: x rounded to TF32 (10 mantissa bits, halves away from zero), small: the exact rest
 __device__ __forceinline__ Split split(const float x) {
   Split s;
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(s.big) : "f"(x));
+  s.big = (__float_as_uint(x) + 0x1000U) & 0xffffe000U;
   s.small = __float_as_uint(x - __uint_as_float(s.big));
   return s;
 }
@@ -317,11 +329,16 @@ __device__ __forceinline__ Operand operand_of(const float (&c)[4]) {
   }
   return a;
 }
-__device__ __forceinline__ void mma_f32(float (&d)[4], const Operand &a, const float b0, const float b1) {
+// Main and correction sums in separate accumulators: shorter chains of dependent MMAs.
+struct Sum {
+  float main[4] = {}, first[4] = {}, second[4] = {};
+  __device__ __forceinline__ float get(const int i) const { return main[i] + (first[i] + second[i]); }
+};
+__device__ __forceinline__ void mma_f32(Sum &d, const Operand &a, const float b0, const float b1) {
   const Split x = split(b0), y = split(b1);
-  mma_tf32(d, a.small, x.big, y.big);
-  mma_tf32(d, a.big, x.small, y.small);
-  mma_tf32(d, a.big, x.big, y.big);
+  mma_tf32(d.first, a.small, x.big, y.big);
+  mma_tf32(d.second, a.big, x.small, y.small);
+  mma_tf32(d.main, a.big, x.big, y.big);
 }
 
 struct WalkParams {
@@ -369,8 +386,11 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
   const auto fetch = [&](const int chunk) {
     float *const b = smem + (chunk & 1) * L::kBuffer;
     const int words = p.head_stride / 4;
-    for (int i = threadIdx.x; i < kChunk * words; i += kThreads) {
-      const int row = i / words, word = i % words;
+    constexpr int kWords = L::kWidth / 4;
+#pragma unroll
+    for (int i = 0; i < kChunk * kWords / kThreads; ++i) {
+      const int row = (i * kThreads + threadIdx.x) / kWords, word = (i * kThreads + threadIdx.x) % kWords;
+      if (word >= words) continue;
       const std::size_t source = (static_cast<std::size_t>(chunk * kChunk + row) * key_heads + key_head) * p.head_stride + word * 4;
       copy16(b + L::kKeys + row * L::kRow + word * 4, keys + source);
       copy16(b + L::kQueries + row * L::kRow + word * 4, queries + source);
@@ -421,7 +441,7 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
       load_values(chunk + 1);
     }
     // this warp's channels of S^T K^T and S^T Q^T, two halves of eight tokens each
-    float products[kProducts][4] = {};
+    Sum products[kProducts];
 #pragma unroll
     for (int n = 0; n < kTiles; ++n) {
       const Operand a = operand_of(S[n]);
@@ -438,7 +458,7 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
     }
 #pragma unroll
     for (int i = 0; i < kProducts; ++i)
-      parts[(warp * kProducts + i) * 32 + lane] = make_float4(products[i][0], products[i][1], products[i][2], products[i][3]);
+      parts[(warp * kProducts + i) * 32 + lane] = make_float4(products[i].get(0), products[i].get(1), products[i].get(2), products[i].get(3));
     const auto gathered = [&](const int product, float (&sum)[4]) {
       float4 total = parts[product * 32 + lane];
 #pragma unroll
@@ -475,13 +495,14 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
     if constexpr (kDelta) {
 #pragma unroll
       for (int out = 0; out < 2; ++out) {
-        float u[4] = {};
+        Sum u;
 #pragma unroll
         for (int half = 0; half <= out; ++half) {  // later tokens do not reach earlier ones
           const float *const x = m + (8 * half + 2 * t) * kMatrixStride + 8 * out + g;
           mma_f32(u, right[half], x[0], x[kMatrixStride]);
         }
-        update[out] = operand_of(u);
+        const float sums[4] = {u.get(0), u.get(1), u.get(2), u.get(3)};
+        update[out] = operand_of(sums);
       }
     } else {
       update[0] = right[0];
@@ -497,23 +518,26 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
         const float2 decay = *reinterpret_cast<const float2 *>(b + L::kLast + channel0 + 8 * n + 2 * t);
         S[n][0] *= decay.x, S[n][1] *= decay.y, S[n][2] *= decay.x, S[n][3] *= decay.y;
       }
+      Sum added;
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const float *const k = b + L::kKeys + (8 * half + 2 * t) * L::kRow + channel0 + 8 * n + g;
-        mma_f32(S[n], update[half], k[0], k[L::kRow]);
+        mma_f32(added, update[half], k[0], k[L::kRow]);
       }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) S[n][i] += added.get(i);
     }
     if constexpr (!kDelta) __syncthreads();
     if (warp < 2) {  // outputs of token half `warp`
       float o[4];
       gathered(warp, o);
-      if constexpr (kDelta) {
-#pragma unroll
-        for (int i = 0; i < 4; ++i) o[i] *= cumulative[8 * warp + 2 * t + (i & 1)];
-      }
       const float *const x = m + (kDelta ? kMatrix : 0) + 2 * t * kMatrixStride + 8 * warp + g;
-      mma_f32(o, right[0], x[0], x[kMatrixStride]);
-      if (warp == 1) mma_f32(o, right[1], x[8 * kMatrixStride], x[9 * kMatrixStride]);
+      Sum inside;
+      mma_f32(inside, right[0], x[0], x[kMatrixStride]);
+      if (warp == 1) mma_f32(inside, right[1], x[8 * kMatrixStride], x[9 * kMatrixStride]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        o[i] = kDelta ? fmaf(o[i], cumulative[8 * warp + 2 * t + (i & 1)], inside.get(i)) : o[i] + inside.get(i);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int row = chunk * kChunk + 8 * warp + 2 * t + (i & 1), column = column0 + g + (i & 2) * 4;
@@ -621,7 +645,7 @@ int recurrent_chunks(const RecurrentArgs &a, float **output, cudaStream_t stream
     p.beta_column = static_cast<int>(a.beta_column);
     p.decay_column = static_cast<int>(a.decay_column);
     p.fresh = w.fresh;
-    const std::size_t bytes = (2 * kChunk * (a.dim + 1) + kPrepThreads / kChunk * kChunk * (kChunk + 1)) * sizeof(float);
+    const std::size_t bytes = (2 * kChunk * (a.dim + 1) + kPrepThreads / kChunk * 2 * kChunk * kMatrixStride) * sizeof(float);
     bf16 *const values = reinterpret_cast<bf16 *>(base + l.value);
     const auto kernel = a.conv_taps <= 4 ? delta_chunks_kernel<4, bf16> : delta_chunks_kernel<8, bf16>;
     if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)) != cudaSuccess)

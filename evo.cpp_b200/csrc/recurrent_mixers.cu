@@ -566,6 +566,58 @@ norm_gate_kernel(const float *__restrict__ input, const float *__restrict__ gain
     out[d] = from_float<T>(o[d] * factor * gain[d] * silu_f32(to_float(g[d])));
 }
 
+// The same for value sizes that are multiples of four up to 512: a lane owns runs of four.
+__device__ __forceinline__ void load_quad(const float *const p, float (&v)[4]) {
+  const float4 w = *reinterpret_cast<const float4 *>(p);
+  v[0] = w.x, v[1] = w.y, v[2] = w.z, v[3] = w.w;
+}
+__device__ __forceinline__ void load_quad(const bf16 *const p, float (&v)[4]) {
+  const uint2 w = *reinterpret_cast<const uint2 *>(p);
+  v[0] = __uint_as_float(w.x << 16U), v[1] = __uint_as_float(w.x & 0xffff0000U);
+  v[2] = __uint_as_float(w.y << 16U), v[3] = __uint_as_float(w.y & 0xffff0000U);
+}
+__device__ __forceinline__ void store_quad(float *const p, const float (&v)[4]) {
+  *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void store_quad(bf16 *const p, const float (&v)[4]) {
+  *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+
+template <int kQuads, typename T>
+__global__ void __launch_bounds__(256)
+norm_gate_quads_kernel(const float *__restrict__ input, const float *__restrict__ gain, const T *__restrict__ gate,
+                       const std::size_t gate_stride, const int rows, const int heads, const int value_dim,
+                       const float epsilon, T *__restrict__ output) {
+  const std::size_t item = static_cast<std::size_t>(blockIdx.x) * 8 + threadIdx.x / 32;
+  const int lane = threadIdx.x % 32;
+  if (item >= static_cast<std::size_t>(rows) * heads) return;
+  const std::size_t row = item / heads, head = item % heads;
+  const float *const o = input + item * value_dim;
+  const T *const g = gate + row * gate_stride + head * value_dim;
+  float v[kQuads][4] = {}, z[kQuads][4] = {}, square = 0.0F;
+#pragma unroll
+  for (int i = 0; i < kQuads; ++i) {
+    const int d = 4 * (lane + 32 * i);
+    if (d < value_dim) {
+      load_quad(o + d, v[i]);
+      load_quad(g + d, z[i]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) square = fmaf(v[i][e], v[i][e], square);
+  }
+  const float factor = 1.0F / sqrtf(warp_sum(square) / static_cast<float>(value_dim) + epsilon);
+#pragma unroll
+  for (int i = 0; i < kQuads; ++i) {
+    const int d = 4 * (lane + 32 * i);
+    if (d >= value_dim) continue;
+    float w[4], y[4];
+    load_quad(gain + d, w);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[e] = v[i][e] * factor * w[e] * silu_f32(z[i][e]);
+    store_quad(output + item * value_dim + d, y);
+  }
+}
+
 // ---------------------------------------------------------------- one token
 // A cluster of CTAs per key head: each owns a slice of the value columns of the heads that share the key, keeps
 // its part of the state in registers between the read-out and the update (a warp per set of channels, a lane
@@ -791,9 +843,15 @@ int advance_history(const RecurrentArgs &a, cudaStream_t stream) {
 
 template <typename T>
 int norm_gate(const RecurrentArgs &a, const float *input, cudaStream_t stream) {
-  norm_gate_kernel<T><<<ceil_div_u(a.rows * a.heads, 8), 256, 0, stream>>>(
-      input, a.output_norm, static_cast<const T *>(a.projection) + a.gate_column, a.stride, static_cast<int>(a.rows),
-      static_cast<int>(a.heads), static_cast<int>(a.value_dim), a.epsilon, static_cast<T *>(a.output));
+  const T *const gate = static_cast<const T *>(a.projection) + a.gate_column;
+  const bool quads = a.value_dim % 4 == 0 && a.value_dim <= 512 && a.stride % 8 == 0 && a.gate_column % 8 == 0 &&
+                     aligned16(a.projection) && aligned16(a.output) && aligned16(a.output_norm);
+  const auto kernel = !quads ? norm_gate_kernel<T>
+                      : a.value_dim <= 128 ? norm_gate_quads_kernel<1, T>
+                      : a.value_dim <= 256 ? norm_gate_quads_kernel<2, T> : norm_gate_quads_kernel<4, T>;
+  kernel<<<ceil_div_u(a.rows * a.heads, 8), 256, 0, stream>>>(
+      input, a.output_norm, gate, a.stride, static_cast<int>(a.rows), static_cast<int>(a.heads),
+      static_cast<int>(a.value_dim), a.epsilon, static_cast<T *>(a.output));
   return check_launch("output norm and gate kernel");
 }
 
