@@ -9,7 +9,7 @@
 //     N = (I + A)^-1, XW_st = D_15,t N_ts, XM_st = sum_r D_tr (k_r.q_t) N_rs
 // (tokens in rows of K, Q, columns of O, R; decay products only, no quotients, so extreme decays stay finite).
 // A first kernel prepares Q~, K~ and the 16 x 16 matrices for all chunks at once; the second walks the chunks
-// of one head and 16 value columns per CTA.  Its four warps split the key channels: each keeps S^T for its
+// of one head and 16 value columns per CTA.  Its eight warps split the key channels: each keeps S^T for its
 // channels as MMA accumulators and uses them in place as the A operand of the next chunk (the contraction
 // may run over the channels in any order, so the accumulator layout is a valid operand layout).
 //
@@ -23,7 +23,7 @@
 namespace evob {
 namespace {
 
-constexpr int kChunk = 16, kColumns = 16, kThreads = 128;
+constexpr int kChunk = 16, kColumns = 16, kWarps = 8, kThreads = 32 * kWarps;
 constexpr int kMatrixStride = 20;                       // floats between rows of a 16 x 16 matrix
 constexpr int kMatrix = kChunk * kMatrixStride;
 // per chunk and head: XW | XM | beta | beta G | G (delta), X (linear)
@@ -40,6 +40,8 @@ struct DeltaParams {
 };
 
 constexpr int kPrepThreads = 256;
+// Floats between rows of keys or queries in shared memory: whole 16-byte words, four banks from row to row.
+__host__ __device__ constexpr int pair_stride(const int dim) { return (dim + 31) / 32 * 32 + 4; }
 
 // 16 tokens of one channel of the convolution with SiLU, handed to emit(token, value).
 template <int kTaps, typename T, typename Emit>
@@ -53,17 +55,30 @@ __device__ __forceinline__ void convolve_chunk(const T *const projection, const 
     const int tap = j - (kTaps - n);
     taps[j] = tap >= 0 ? conv[static_cast<std::size_t>(column) * n + tap] : 0.0F;
   }
-  const auto input = [&](const int row) -> float {
-    if (row >= p.rows) return 0.0F;
-    if (row >= 0) return to_float(projection[static_cast<std::size_t>(row) * p.stride + column]);
-    if (p.fresh != 0 || row + n - 1 < 0) return 0.0F;
-    return to_float(history[static_cast<std::size_t>(row + n - 1) * p.channels + column]);
-  };
-#pragma unroll
-  for (int j = 0; j < kTaps; ++j) window[j] = j == 0 ? 0.0F : input(row0 - kTaps + j);
   float next[kChunk];
+  if (row0 >= kTaps - 1 && row0 + kChunk <= p.rows) {
+    const T *const source = projection + static_cast<std::size_t>(row0) * p.stride + column;
+    T raw[kTaps - 1 + kChunk];
 #pragma unroll
-  for (int t = 0; t < kChunk; ++t) next[t] = input(row0 + t);
+    for (int i = 0; i < kTaps - 1 + kChunk; ++i)
+      raw[i] = source[(static_cast<long long>(i) - (kTaps - 1)) * static_cast<long long>(p.stride)];
+    window[0] = 0.0F;
+#pragma unroll
+    for (int j = 1; j < kTaps; ++j) window[j] = to_float(raw[j - 1]);
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) next[t] = to_float(raw[kTaps - 1 + t]);
+  } else {
+    const auto input = [&](const int row) -> float {
+      if (row >= p.rows) return 0.0F;
+      if (row >= 0) return to_float(projection[static_cast<std::size_t>(row) * p.stride + column]);
+      if (p.fresh != 0 || row + n - 1 < 0) return 0.0F;
+      return to_float(history[static_cast<std::size_t>(row + n - 1) * p.channels + column]);
+    };
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j) window[j] = j == 0 ? 0.0F : input(row0 - kTaps + j);
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) next[t] = input(row0 + t);
+  }
 #pragma unroll
   for (int t = 0; t < kChunk; ++t) {
 #pragma unroll
@@ -72,7 +87,7 @@ __device__ __forceinline__ void convolve_chunk(const T *const projection, const 
     float sum = 0.0F;
 #pragma unroll
     for (int j = 0; j < kTaps; ++j) sum = fmaf(taps[j], window[j], sum);
-    emit(t, row0 + t < p.rows ? silu_f32(sum) : 0.0F);
+    emit(t, row0 + t < p.rows ? __fdividef(sum, 1.0F + expf(-fmaxf(sum, -80.0F))) : 0.0F);  // SiLU
   }
 }
 
@@ -82,15 +97,18 @@ delta_chunks_kernel(const T *__restrict__ projection, const T *__restrict__ hist
                     const float *__restrict__ decay_rate, const float *__restrict__ decay_shift,
                     float *__restrict__ queries, float *__restrict__ keys, T *__restrict__ values,
                     float *__restrict__ matrices, const DeltaParams p) {
-  extern __shared__ __align__(16) float smem[];  // per slot of heads two 16 x 16 matrices, then keys and queries [16][dim + 1]
-  const int stride = p.dim + 1;
+  extern __shared__ __align__(16) float smem[];  // per slot of heads two 16 x 16 matrices, then keys and queries [16][pair_stride]
+  const int stride = pair_stride(p.dim);
   float *const heads_base = smem;
   float *const ks = heads_base + kPrepThreads / kChunk * 2 * kChunk * kMatrixStride, *const qs = ks + kChunk * stride;
   __shared__ float kk[kChunk][kChunk + 1], kq[kChunk][kChunk + 1];  // [t][s]
+  __shared__ float part[4][2][kChunk][kChunk];
   const int chunk = blockIdx.x, g = blockIdx.y, row0 = chunk * kChunk;
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
   const int group = p.heads / p.kv_heads;
   const int total = 2 * p.dim + group * p.value_dim;
+  for (int i = threadIdx.x; i < 2 * kChunk * (stride - p.dim); i += kPrepThreads)  // padding behind the channels
+    ks[i / (stride - p.dim) * stride + p.dim + i % (stride - p.dim)] = 0.0F;
   for (int c = threadIdx.x; c < total; c += kPrepThreads) {
     if (c < 2 * p.dim) {
       const bool is_key = c < p.dim;
@@ -124,20 +142,43 @@ delta_chunks_kernel(const T *__restrict__ projection, const T *__restrict__ hist
     }
   }
   __syncthreads();
-  // inner products: one (t, s) pair per thread
+  // inner products: a quarter of the channels of 2 x 2 (t, s) pairs per thread, rows eight apart so that the
+  // 16-byte reads of a warp spread over the banks
+  {
+    const int quarter = threadIdx.x / 64, pair = threadIdx.x % 64, t = pair / 8, s = pair % 8;
+    float a[2][2] = {}, b[2][2] = {};
+    const int words = stride / 4;
+    for (int word = quarter; word < words; word += 4) {
+      float k[2][4], kt[2][4], q[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        load_floats<4>(ks + (s + 8 * i) * stride + 4 * word, k[i]);
+        load_floats<4>(ks + (t + 8 * i) * stride + 4 * word, kt[i]);
+        load_floats<4>(qs + (t + 8 * i) * stride + 4 * word, q[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int l = 0; l < 2; ++l)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            a[i][l] = fmaf(kt[i][e], k[l][e], a[i][l]);
+            b[i][l] = fmaf(q[i][e], k[l][e], b[i][l]);
+          }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int l = 0; l < 2; ++l) {
+        part[quarter][0][t + 8 * i][s + 8 * l] = a[i][l];
+        part[quarter][1][t + 8 * i][s + 8 * l] = b[i][l];
+      }
+  }
+  __syncthreads();
   {
     const int t = threadIdx.x / kChunk, s = threadIdx.x % kChunk;
-    float a = 0.0F, b = 0.0F;
-    if (s <= t) {
-#pragma unroll 4
-      for (int d = 0; d < p.dim; ++d) {
-        const float k = ks[s * stride + d];
-        a = fmaf(k, ks[t * stride + d], a);
-        b = fmaf(k, qs[t * stride + d], b);
-      }
-    }
-    kk[t][s] = a;
-    kq[t][s] = b;
+    kk[t][s] = (part[0][0][t][s] + part[1][0][t][s]) + (part[2][0][t][s] + part[3][0][t][s]);
+    kq[t][s] = (part[0][1][t][s] + part[1][1][t][s]) + (part[2][1][t][s] + part[3][1][t][s]);
   }
   __syncthreads();
   // heads that share the key, two per warp: thread j of sixteen owns column j of the inverse
@@ -240,6 +281,22 @@ linear_chunks_kernel(const T *__restrict__ projection, const std::size_t stride,
   const int channel = head * dim + d, channels = heads * dim;
   const bool inside = d < dim;
   float a[kChunk], q[kChunk], k[kChunk];
+  if (inside && row0 + kChunk <= rows) {
+    const T *const source = projection + static_cast<std::size_t>(row0) * stride + channel;
+    T raw_q[kChunk], raw_k[kChunk];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      raw_q[t] = source[t * stride];
+      raw_k[t] = source[t * stride + key_column];
+    }
+    const float offset = bias[channel];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      a[t] = offset;
+      q[t] = to_float(raw_q[t]);
+      k[t] = to_float(raw_k[t]);
+    }
+  } else
 #pragma unroll
   for (int t = 0; t < kChunk; ++t) {
     a[t] = inside ? bias[channel] : 0.0F;
@@ -355,7 +412,7 @@ __device__ __forceinline__ void copy16(float *const dst, const float *const src)
 
 template <bool kDelta, int kTiles>
 struct WalkLayout {
-  static constexpr int kWidth = kTiles * 32;      // key channels, eight per tile and warp
+  static constexpr int kWidth = kTiles * 8 * kWarps;  // key channels, eight per tile and warp
   static constexpr int kRow = kWidth + 8;         // floats: the 64-bit operand reads hit every bank once
   static constexpr int kValueStride = 20;
   static constexpr int kKeys = 0, kQueries = kChunk * kRow, kLast = 2 * kChunk * kRow;
@@ -363,7 +420,8 @@ struct WalkLayout {
   static constexpr int kValues = kMatrices + (kDelta ? kDeltaFloats : kLinearFloats);
   static constexpr int kBuffer = kValues + kChunk * kValueStride;
   static constexpr int kParts = 2 * kBuffer;      // [warp][product][lane] float4
-  static constexpr int kFloats = kParts + 4 * (kDelta ? 4 : 2) * 32 * 4;
+  static constexpr int kRight = kParts + kWarps * (kDelta ? 4 : 2) * 32 * 4;  // delta: R, two halves of 32 float4
+  static constexpr int kFloats = kRight + (kDelta ? 2 * 32 * 4 : 0);
 };
 
 template <bool kDelta, int kTiles, typename T>
@@ -403,15 +461,12 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
       copy16(b + L::kMatrices + 4 * i, matrices + (static_cast<std::size_t>(chunk) * p.heads + head) * kFloats + 4 * i);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  T staged[2];  // widened only when they are stored: the loads stay in flight until then
+  T staged;  // widened only when they are stored: the loads stay in flight until then
+  static_assert(kThreads == kChunk * kColumns, "one value of the chunk per thread");
   const auto load_values = [&](const int chunk) {
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int index = i * kThreads + threadIdx.x, row = chunk * kChunk + index / kColumns, c = column0 + index % kColumns;
-      staged[i] = row < p.rows && c < p.value_dim
-                      ? values[static_cast<std::size_t>(row) * p.value_stride + head * p.value_dim + c]
-                      : from_float<T>(0.0F);
-    }
+    const int row = chunk * kChunk + threadIdx.x / kColumns, c = column0 + threadIdx.x % kColumns;
+    staged = row < p.rows && c < p.value_dim ? values[static_cast<std::size_t>(row) * p.value_stride + head * p.value_dim + c]
+                                             : from_float<T>(0.0F);
   };
 
   float S[kTiles][4];  // S^T: rows = value columns g, g + 8; columns = channels channel0 + 8 tile + 2t, + 1
@@ -429,11 +484,7 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
   float4 *const parts = reinterpret_cast<float4 *>(smem + L::kParts);
   for (int chunk = 0; chunk < chunks; ++chunk) {
     float *const b = smem + (chunk & 1) * L::kBuffer;
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int index = i * kThreads + threadIdx.x;
-      b[L::kValues + index / kColumns * L::kValueStride + index % kColumns] = to_float(staged[i]);
-    }
+    b[L::kValues + threadIdx.x / kColumns * L::kValueStride + threadIdx.x % kColumns] = to_float(staged);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();  // the chunk is here, and everybody is done with the one before
     if (chunk + 1 < chunks) {
@@ -462,34 +513,37 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
     const auto gathered = [&](const int product, float (&sum)[4]) {
       float4 total = parts[product * 32 + lane];
 #pragma unroll
-      for (int w = 1; w < 4; ++w) {
+      for (int w = 1; w < kWarps; ++w) {
         const float4 v = parts[(w * kProducts + product) * 32 + lane];
         total.x += v.x, total.y += v.y, total.z += v.z, total.w += v.w;
       }
       sum[0] = total.x, sum[1] = total.y, sum[2] = total.z, sum[3] = total.w;
     };
-    // rows of the right-hand side in the accumulator layout: values [column][token]
-    float R[2][4];
-#pragma unroll
-    for (int half = 0; half < 2; ++half)
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-        R[half][i] = b[L::kValues + (8 * half + 2 * t + (i & 1)) * L::kValueStride + g + (i & 2) * 4];
     const float *const m = b + L::kMatrices;
     const float *const beta = m + 2 * kMatrix, *const beta_g = beta + kChunk, *const cumulative = beta_g + kChunk;
     Operand update[2];  // what is added to the state, by token half
+    // the right-hand side in the accumulator layout, [column][token]: the values, for the delta rule corrected
+    float R[2][4];
     if constexpr (kDelta) {
       __syncthreads();
+      // one element per thread: (token half, lane, accumulator register)
+      const int half = threadIdx.x / 128, at = threadIdx.x % 128, i = at % 4;
+      const int token = 8 * half + 2 * (at / 4 % 4) + (i & 1), column = at / 16 + (i & 2) * 4;
+      const float *const held = smem + L::kParts + (2 + half) * 128 + at;
+      float sum[2] = {0.0F, 0.0F};
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        float held[4];
-        gathered(2 + half, held);
+      for (int w = 0; w < kWarps; ++w) sum[w % 2] += held[w * kProducts * 128];
+      smem[L::kRight + threadIdx.x] =
+          fmaf(-beta_g[token], sum[0] + sum[1], beta[token] * b[L::kValues + token * L::kValueStride + column]);
+      __syncthreads();
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int token = 8 * half + 2 * t + (i & 1);
-          R[half][i] = fmaf(-beta_g[token], held[i], beta[token] * R[half][i]);
-        }
-      }
+      for (int half = 0; half < 2; ++half) load_floats<4>(smem + L::kRight + half * 128 + lane * 4, R[half]);
+    } else {
+#pragma unroll
+      for (int half = 0; half < 2; ++half)
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          R[half][i] = b[L::kValues + (8 * half + 2 * t + (i & 1)) * L::kValueStride + g + (i & 2) * 4];
     }
     Operand right[2] = {operand_of(R[0]), operand_of(R[1])};
     if constexpr (kDelta) {
@@ -571,10 +625,9 @@ int launch_walk(const float *queries, const float *keys, const float *last, cons
 template <bool kDelta>
 int dispatch_walk(const float *queries, const float *keys, const float *last, const float *matrices, const bf16 *values,
                   float *state, float *output, const WalkParams &p, cudaStream_t stream) {
-  if (p.dim <= 32) return launch_walk<kDelta, 1>(queries, keys, last, matrices, values, state, output, p, stream);
-  if (p.dim <= 64) return launch_walk<kDelta, 2>(queries, keys, last, matrices, values, state, output, p, stream);
-  if (p.dim <= 128) return launch_walk<kDelta, 4>(queries, keys, last, matrices, values, state, output, p, stream);
-  return launch_walk<kDelta, 8>(queries, keys, last, matrices, values, state, output, p, stream);
+  if (p.dim <= 64) return launch_walk<kDelta, 1>(queries, keys, last, matrices, values, state, output, p, stream);
+  if (p.dim <= 128) return launch_walk<kDelta, 2>(queries, keys, last, matrices, values, state, output, p, stream);
+  return launch_walk<kDelta, 4>(queries, keys, last, matrices, values, state, output, p, stream);
 }
 
 struct Layout {
@@ -645,7 +698,7 @@ int recurrent_chunks(const RecurrentArgs &a, float **output, cudaStream_t stream
     p.beta_column = static_cast<int>(a.beta_column);
     p.decay_column = static_cast<int>(a.decay_column);
     p.fresh = w.fresh;
-    const std::size_t bytes = (2 * kChunk * (a.dim + 1) + kPrepThreads / kChunk * 2 * kChunk * kMatrixStride) * sizeof(float);
+    const std::size_t bytes = (2 * kChunk * pair_stride(static_cast<int>(a.dim)) + kPrepThreads / kChunk * 2 * kChunk * kMatrixStride) * sizeof(float);
     bf16 *const values = reinterpret_cast<bf16 *>(base + l.value);
     const auto kernel = a.conv_taps <= 4 ? delta_chunks_kernel<4, bf16> : delta_chunks_kernel<8, bf16>;
     if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)) != cudaSuccess)
