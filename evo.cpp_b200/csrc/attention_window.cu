@@ -20,7 +20,8 @@ namespace cg = cooperative_groups;
 // ---------------------------------------------------------------- head norms and cache append
 constexpr int kAppendThreads = 256;
 
-template <typename T>
+// kQuads: head sizes that are multiples of four, all columns at multiples of four; a lane owns runs of four.
+template <typename T, bool kQuads>
 __global__ void __launch_bounds__(kAppendThreads)
 head_norm_append_kernel(const T *__restrict__ projection, const std::size_t stride, const int key_column,
                         const int value_column, const float *__restrict__ query_gain,
@@ -38,7 +39,15 @@ head_norm_append_kernel(const T *__restrict__ projection, const std::size_t stri
       const int g = head - heads - kv_heads;
       T *const out = value_cache + (at * kv_heads + g) * value_dim;
       const T *const in = source + value_column + g * value_dim;
-      for (int i = lane; i < value_dim; i += 32) out[i] = in[i];
+      if constexpr (kQuads) {
+        for (int i = 4 * lane; i < value_dim; i += 128) {
+          float v[4];
+          load_quad(in + i, v);
+          store_quad(out + i, v);
+        }
+      } else {
+        for (int i = lane; i < value_dim; i += 32) out[i] = in[i];
+      }
       continue;
     }
     const bool is_query = head < heads;
@@ -46,20 +55,43 @@ head_norm_append_kernel(const T *__restrict__ projection, const std::size_t stri
     const T *const in = source + (is_query ? 0 : key_column) + local * dim;
     const float *const gain = is_query ? query_gain : key_gain;
     T *const out = is_query ? query + (row * heads + local) * dim : key_cache + (at * kv_heads + local) * dim;
-    float v[kDecoderMaxHeadDim / 32];
-    float square = 0.0F;
+    if constexpr (kQuads) {
+      constexpr int kRuns = static_cast<int>(kDecoderMaxHeadDim) / 128;
+      float v[kRuns][4] = {}, square = 0.0F;
 #pragma unroll
-    for (int i = 0; i < static_cast<int>(kDecoderMaxHeadDim) / 32; ++i) {
-      const int d = lane + 32 * i;
-      v[i] = d < dim ? to_float(in[d]) : 0.0F;
-      square = fmaf(v[i], v[i], square);
-    }
-    square = warp_sum(square);
-    const float factor = 1.0F / sqrtf(square / static_cast<float>(dim) + epsilon);
+      for (int i = 0; i < kRuns; ++i) {
+        const int d = 4 * lane + 128 * i;
+        if (d < dim) load_quad(in + d, v[i]);
 #pragma unroll
-    for (int i = 0; i < static_cast<int>(kDecoderMaxHeadDim) / 32; ++i) {
-      const int d = lane + 32 * i;
-      if (d < dim) out[d] = from_float<T>(v[i] * factor * gain[d]);
+        for (int e = 0; e < 4; ++e) square = fmaf(v[i][e], v[i][e], square);
+      }
+      const float factor = 1.0F / sqrtf(warp_sum(square) / static_cast<float>(dim) + epsilon);
+#pragma unroll
+      for (int i = 0; i < kRuns; ++i) {
+        const int d = 4 * lane + 128 * i;
+        if (d >= dim) continue;
+        float w[4], y[4];
+        load_quad(gain + d, w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] = v[i][e] * factor * w[e];
+        store_quad(out + d, y);
+      }
+    } else {
+      float v[kDecoderMaxHeadDim / 32];
+      float square = 0.0F;
+#pragma unroll
+      for (int i = 0; i < static_cast<int>(kDecoderMaxHeadDim) / 32; ++i) {
+        const int d = lane + 32 * i;
+        v[i] = d < dim ? to_float(in[d]) : 0.0F;
+        square = fmaf(v[i], v[i], square);
+      }
+      square = warp_sum(square);
+      const float factor = 1.0F / sqrtf(square / static_cast<float>(dim) + epsilon);
+#pragma unroll
+      for (int i = 0; i < static_cast<int>(kDecoderMaxHeadDim) / 32; ++i) {
+        const int d = lane + 32 * i;
+        if (d < dim) out[d] = from_float<T>(v[i] * factor * gain[d]);
+      }
     }
   }
 }
@@ -90,7 +122,7 @@ __device__ __forceinline__ void merge(float &m, float &l, float &acc, const floa
 
 // ---------------------------------------------------------------- row kernel
 constexpr int kSplits = 8;  // CTAs per cluster
-constexpr int kRowThreads = 128;
+constexpr int kRowThreads = 256;
 constexpr int kRowWarps = kRowThreads / 32;
 
 struct RowParams {
@@ -413,9 +445,13 @@ int head_norm_append(const HeadNormArgs &a, cudaStream_t stream) {
       a.stride > 0x7fffff00U)
     return fail(kInvalidArgument, "head norm arguments are invalid");
   if (a.rows == 0) return kOk;
+  const bool quads = a.dim % 4 == 0 && a.value_dim % 4 == 0 && a.stride % 4 == 0 && a.key_column % 4 == 0 &&
+                     a.value_column % 4 == 0 && aligned16(a.projection) && aligned16(a.query) && aligned16(a.key_cache) &&
+                     aligned16(a.value_cache) && aligned16(a.query_gain) && aligned16(a.key_gain);
   const auto launch = [&](auto tag) {
     using T = decltype(tag);
-    head_norm_append_kernel<T><<<static_cast<unsigned int>(a.rows), kAppendThreads, 0, stream>>>(
+    const auto kernel = quads ? head_norm_append_kernel<T, true> : head_norm_append_kernel<T, false>;
+    kernel<<<static_cast<unsigned int>(a.rows), kAppendThreads, 0, stream>>>(
         static_cast<const T *>(a.projection), a.stride, static_cast<int>(a.key_column),
         static_cast<int>(a.value_column), a.query_gain, a.key_gain, static_cast<T *>(a.query),
         static_cast<T *>(a.key_cache), static_cast<T *>(a.value_cache), static_cast<int>(a.position),

@@ -49,6 +49,23 @@ __device__ __forceinline__ void store_floats(bf16 *const p, const float (&v)[8])
                                              pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
 }
 
+// Four consecutive elements.
+__device__ __forceinline__ void load_quad(const float *const p, float (&v)[4]) {
+  const float4 w = *reinterpret_cast<const float4 *>(p);
+  v[0] = w.x, v[1] = w.y, v[2] = w.z, v[3] = w.w;
+}
+__device__ __forceinline__ void load_quad(const bf16 *const p, float (&v)[4]) {
+  const uint2 w = *reinterpret_cast<const uint2 *>(p);
+  v[0] = __uint_as_float(w.x << 16U), v[1] = __uint_as_float(w.x & 0xffff0000U);
+  v[2] = __uint_as_float(w.y << 16U), v[3] = __uint_as_float(w.y & 0xffff0000U);
+}
+__device__ __forceinline__ void store_quad(float *const p, const float (&v)[4]) {
+  *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void store_quad(bf16 *const p, const float (&v)[4]) {
+  *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+
 __device__ __forceinline__ float sigmoid_f32(const float x) { return 1.0F / (1.0F + expf(-x)); }
 __device__ __forceinline__ float silu_f32(const float x) { return x / (1.0F + expf(-x)); }
 // ln(1 + e^x) without overflow or cancellation

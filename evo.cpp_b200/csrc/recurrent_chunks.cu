@@ -487,10 +487,6 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
     b[L::kValues + threadIdx.x / kColumns * L::kValueStride + threadIdx.x % kColumns] = to_float(staged);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();  // the chunk is here, and everybody is done with the one before
-    if (chunk + 1 < chunks) {
-      fetch(chunk + 1);
-      load_values(chunk + 1);
-    }
     // this warp's channels of S^T K^T and S^T Q^T, two halves of eight tokens each
     Sum products[kProducts];
 #pragma unroll
@@ -507,9 +503,14 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
         }
       }
     }
+    const float *const m = b + L::kMatrices;
 #pragma unroll
     for (int i = 0; i < kProducts; ++i)
       parts[(warp * kProducts + i) * 32 + lane] = make_float4(products[i].get(0), products[i].get(1), products[i].get(2), products[i].get(3));
+    if (chunk + 1 < chunks) {
+      fetch(chunk + 1);
+      load_values(chunk + 1);
+    }
     const auto gathered = [&](const int product, float (&sum)[4]) {
       float4 total = parts[product * 32 + lane];
 #pragma unroll
@@ -519,10 +520,9 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
       }
       sum[0] = total.x, sum[1] = total.y, sum[2] = total.z, sum[3] = total.w;
     };
-    const float *const m = b + L::kMatrices;
     const float *const beta = m + 2 * kMatrix, *const beta_g = beta + kChunk, *const cumulative = beta_g + kChunk;
-    Operand update[2];  // what is added to the state, by token half
-    // the right-hand side in the accumulator layout, [column][token]: the values, for the delta rule corrected
+    Operand right[2], update[2];  // the right-hand side, and what is added to the state, by token half
+    // in the accumulator layout, [column][token]: the values, for the delta rule corrected
     float R[2][4];
     if constexpr (kDelta) {
       __syncthreads();
@@ -545,7 +545,8 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
         for (int i = 0; i < 4; ++i)
           R[half][i] = b[L::kValues + (8 * half + 2 * t + (i & 1)) * L::kValueStride + g + (i & 2) * 4];
     }
-    Operand right[2] = {operand_of(R[0]), operand_of(R[1])};
+    right[0] = operand_of(R[0]);
+    right[1] = operand_of(R[1]);
     if constexpr (kDelta) {
 #pragma unroll
       for (int out = 0; out < 2; ++out) {
@@ -590,13 +591,11 @@ chunk_walk_kernel(const float *__restrict__ queries, const float *__restrict__ k
       mma_f32(inside, right[0], x[0], x[kMatrixStride]);
       if (warp == 1) mma_f32(inside, right[1], x[8 * kMatrixStride], x[9 * kMatrixStride]);
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        o[i] = kDelta ? fmaf(o[i], cumulative[8 * warp + 2 * t + (i & 1)], inside.get(i)) : o[i] + inside.get(i);
-#pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int row = chunk * kChunk + 8 * warp + 2 * t + (i & 1), column = column0 + g + (i & 2) * 4;
+        const int token = 8 * warp + 2 * t + (i & 1), row = chunk * kChunk + token, column = column0 + g + (i & 2) * 4;
         if (row < p.rows && column < p.value_dim)
-          output[(static_cast<std::size_t>(row) * p.heads + head) * p.value_dim + column] = o[i];
+          output[(static_cast<std::size_t>(row) * p.heads + head) * p.value_dim + column] =
+              kDelta ? fmaf(o[i], cumulative[token], inside.get(i)) : o[i] + inside.get(i);
       }
     }
   }

@@ -567,22 +567,6 @@ norm_gate_kernel(const float *__restrict__ input, const float *__restrict__ gain
 }
 
 // The same for value sizes that are multiples of four up to 512: a lane owns runs of four.
-__device__ __forceinline__ void load_quad(const float *const p, float (&v)[4]) {
-  const float4 w = *reinterpret_cast<const float4 *>(p);
-  v[0] = w.x, v[1] = w.y, v[2] = w.z, v[3] = w.w;
-}
-__device__ __forceinline__ void load_quad(const bf16 *const p, float (&v)[4]) {
-  const uint2 w = *reinterpret_cast<const uint2 *>(p);
-  v[0] = __uint_as_float(w.x << 16U), v[1] = __uint_as_float(w.x & 0xffff0000U);
-  v[2] = __uint_as_float(w.y << 16U), v[3] = __uint_as_float(w.y & 0xffff0000U);
-}
-__device__ __forceinline__ void store_quad(float *const p, const float (&v)[4]) {
-  *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]);
-}
-__device__ __forceinline__ void store_quad(bf16 *const p, const float (&v)[4]) {
-  *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
-}
-
 template <int kQuads, typename T>
 __global__ void __launch_bounds__(256)
 norm_gate_quads_kernel(const float *__restrict__ input, const float *__restrict__ gain, const T *__restrict__ gate,
