@@ -33,6 +33,7 @@ head_norm_append_kernel(const T *__restrict__ projection, const std::size_t stri
   const std::size_t at = (dynamic_position != nullptr ? *dynamic_position : static_position) + row;
   const T *const source = projection + row * stride;
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+  const float inverse_dim = 1.0F / static_cast<float>(dim);
   if (at >= static_cast<std::size_t>(capacity)) return;  // the host checks the capacity; nothing is written past it
   for (int head = warp; head < heads + 2 * kv_heads; head += kAppendThreads / 32) {
     if (head >= heads + kv_heads) {
@@ -65,7 +66,7 @@ head_norm_append_kernel(const T *__restrict__ projection, const std::size_t stri
 #pragma unroll
         for (int e = 0; e < 4; ++e) square = fmaf(v[i][e], v[i][e], square);
       }
-      const float factor = 1.0F / sqrtf(warp_sum(square) / static_cast<float>(dim) + epsilon);
+      const float factor = rsqrtf(fmaf(warp_sum(square), inverse_dim, epsilon));
 #pragma unroll
       for (int i = 0; i < kRuns; ++i) {
         const int d = 4 * lane + 128 * i;

@@ -159,9 +159,9 @@ poly_norm_kernel(const T *input, const float *__restrict__ coefficients, const i
   second = block_sum<kThreads>(second, scratch);
   fourth = block_sum<kThreads>(fourth, scratch);
   sixth = block_sum<kThreads>(sixth, scratch);
-  const float a = coefficients[0] / sqrtf(second * inverse_width + epsilon);
-  const float b = coefficients[1] / sqrtf(fourth * inverse_width + epsilon);
-  const float c3 = coefficients[2] / sqrtf(sixth * inverse_width + epsilon);
+  const float a = coefficients[0] * rsqrtf(second * inverse_width + epsilon);
+  const float b = coefficients[1] * rsqrtf(fourth * inverse_width + epsilon);
+  const float c3 = coefficients[2] * rsqrtf(sixth * inverse_width + epsilon);
   const float e = coefficients[3];
   const auto emit = [&](const int group, const float (&v)[8]) {
     float y[8];

@@ -67,7 +67,8 @@ __device__ __forceinline__ void store_quad(bf16 *const p, const float (&v)[4]) {
 }
 
 __device__ __forceinline__ float sigmoid_f32(const float x) { return 1.0F / (1.0F + expf(-x)); }
-__device__ __forceinline__ float silu_f32(const float x) { return x / (1.0F + expf(-x)); }
+// (the quotient is good to two units in the last place and wants a divisor below 2^126)
+__device__ __forceinline__ float silu_f32(const float x) { return __fdividef(x, 1.0F + expf(-fmaxf(x, -80.0F))); }
 // ln(1 + e^x) without overflow or cancellation
 __device__ __forceinline__ float softplus_f32(const float x) { return fmaxf(x, 0.0F) + log1pf(expf(-fabsf(x))); }
 

@@ -87,7 +87,7 @@ __device__ __forceinline__ void convolve_chunk(const T *const projection, const 
     float sum = 0.0F;
 #pragma unroll
     for (int j = 0; j < kTaps; ++j) sum = fmaf(taps[j], window[j], sum);
-    emit(t, row0 + t < p.rows ? __fdividef(sum, 1.0F + expf(-fmaxf(sum, -80.0F))) : 0.0F);  // SiLU
+    emit(t, row0 + t < p.rows ? silu_f32(sum) : 0.0F);
   }
 }
 

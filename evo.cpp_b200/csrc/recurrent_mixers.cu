@@ -589,7 +589,7 @@ norm_gate_quads_kernel(const float *__restrict__ input, const float *__restrict_
 #pragma unroll
     for (int e = 0; e < 4; ++e) square = fmaf(v[i][e], v[i][e], square);
   }
-  const float factor = 1.0F / sqrtf(warp_sum(square) / static_cast<float>(value_dim) + epsilon);
+  const float factor = rsqrtf(warp_sum(square) / static_cast<float>(value_dim) + epsilon);
 #pragma unroll
   for (int i = 0; i < kQuads; ++i) {
     const int d = 4 * (lane + 32 * i);
