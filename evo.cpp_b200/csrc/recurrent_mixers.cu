@@ -214,6 +214,7 @@ conv_history_kernel(const T *__restrict__ projection, const std::size_t stride, 
 
 // ---------------------------------------------------------------- linear: preparation
 constexpr int kPrepTokens = 16;
+constexpr std::size_t kMaxDecayRank = 512;  // bottleneck rows of a preparation step in shared memory
 
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -924,9 +925,11 @@ int recurrent_mixer(const RecurrentArgs &a, cudaStream_t stream) {
   if (a.delta && (a.conv == nullptr || a.conv_taps == 0 || (a.conv_taps > 1 && a.conv_history == nullptr) ||
                   a.decay_rate == nullptr || a.decay_shift == nullptr))
     return fail(kInvalidArgument, "delta mixer arguments are invalid");
-  if (!a.delta && (a.decay_weight == nullptr || a.decay_bias == nullptr || a.decay_rank == 0 || a.decay_rank > 2048 ||
+  if (!a.delta && (a.decay_weight == nullptr || a.decay_bias == nullptr || a.decay_rank == 0 ||
                    !(a.tau > 0.0F)))
     return fail(kInvalidArgument, "linear attention arguments are invalid");
+  if (!a.delta && a.decay_rank > kMaxDecayRank)
+    return fail(kUnsupported, "decay bottlenecks wider than " + std::to_string(kMaxDecayRank) + " are not supported");
   if (a.rows == 0) return kOk;
   const std::size_t decode_columns = (a.delta ? a.heads / a.kv_heads : 1) * a.value_dim;
   if (a.rows == 1 && (!a.delta || a.heads / a.kv_heads <= static_cast<std::size_t>(kDecodeMaxGroup)) &&

@@ -142,6 +142,28 @@ def test_values_that_are_one(pkg, rt, tmp_path):
     model.close()
 
 
+def test_odd_sizes_everywhere(pkg, rt, tmp_path):
+    """No width is a multiple of eight: the scalar forms of every operator, rows of every kernel's range."""
+    layers = [attention(heads=5, kv_heads=5, dim=33, vdim=7, size=19, keep_first=2, ff=37), delta(heads=3, kv_heads=1, dim=65, vdim=9,
+              conv=9, ff=None), gla(heads=3, dim=130, vdim=11, tau=0.7, ff=51), delta(heads=2, kv_heads=2, dim=7, vdim=70, conv=5, ff=29)]
+    directory, config, weights = make_model(pkg, tmp_path / "m", layers, vocab=101, width=51, max_positions=163, eps=1e-3,
+                                            decay_rank=9, edit=sharpen)
+    tokens = np.random.default_rng(9).integers(0, 101, 163).tolist()
+    expected = oracle.forward(config, weights, tokens)
+    model = rt.EvoLibrary(pkg.EVO_LIBRARY).load(directory)
+    for flags, limit in ((rt.CONTEXT_FLAG_FLOAT32, F32_LIMIT), (0, BF16_LIMIT)):
+        c = model.context(163, flags=flags)
+        assert error(c.prefill_tokens(tokens), expected) < limit
+        got, at = [], 0
+        for n in (3, 40, 1, 12, 2, 64, 1, 40):
+            got.append(c.prefill_tokens(tokens[:n]) if at == 0 else c.decode(tokens[at])[None] if n == 1
+                       else c.prefill_tokens(tokens[at:at + n], c.PREFILL_CHUNK))
+            at += n
+        assert at == 163 and error(np.concatenate(got), expected) < limit
+        c.close()
+    model.close()
+
+
 def test_larger_heads_on_the_tensor_cores(pkg, rt, tmp_path):
     layers = [attention(heads=4, kv_heads=2, dim=128, vdim=96, size=100, keep_first=5, ff=320), delta(heads=4, kv_heads=2, dim=128,
               vdim=64, ff=512), gla(heads=2, dim=128, vdim=128, ff=None)]
