@@ -35,11 +35,12 @@ KERNEL_SOURCES = [
     "errors.cu", "elementwise.cu", "qgmma_emulation.cu", "gemm_tcgen05.cu", "gemv.cu",
     "hyena_fir.cu", "hyena_fir_fused.cu", "hyena_fir_tcgen05.cu", "hyena_modal.cu", "hyena_decode.cu", "attention.cu", "attention_flash.cu", "attention_tcgen05.cu", "attention_tcgen05_k64.cu", "attention_decode.cu", "kv_q8.cu", "linear_executor.cu", "fp8_codec.cpp",
     "decoder_rows.cu", "attention_window.cu", "recurrent_mixers.cu", "recurrent_chunks.cu",
+    "latent_attention.cu", "experts.cu",
 ]
 OPS_SOURCES = KERNEL_SOURCES + ["ops_api.cu"]
 RUNTIME_SOURCES = KERNEL_SOURCES + [
     "runtime/safetensors.cpp", "runtime/model_load.cpp", "runtime/model_weights.cpp",
-    "runtime/gigusun.cpp",
+    "runtime/gigusun.cpp", "runtime/kikepel.cpp",
     "runtime/model.cu", "runtime/decoder.cu", "runtime/sampler.cpp", "runtime/variant.cpp", "runtime/variant_io.cpp", "runtime/scheduler.cpp", "runtime/c_api.cpp",
 ]
 

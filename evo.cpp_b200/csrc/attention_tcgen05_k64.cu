@@ -171,6 +171,7 @@ struct WindowParams {
   const bf16 *gate;            // [rows, gate_stride] or null
   std::size_t gate_stride;
   int sink;
+  const float *sink_logit;     // [heads] or null: zeros
 };
 
 __device__ __forceinline__ float fast_reciprocal(const float x) {
@@ -346,8 +347,8 @@ flash_tcgen05_k64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     float series_scale = 0.0F;
     const float *bias_row = nullptr;
     if constexpr (kWindow) {
-      if (w.sink != 0) {  // the sink is a score of 0 without a value
-        reference = 0.0F;
+      if (w.sink != 0) {  // the sink is a score without a value
+        reference = w.sink_logit != nullptr ? w.sink_logit[head] * kLog2e : 0.0F;
         running_sum = 1.0F;
       } else {
         reference = -3.0e38F;  // finite: a tile may hide every key from a row
@@ -671,7 +672,9 @@ int window_attention_tcgen05(const WindowAttentionArgs &a, cudaStream_t stream) 
       (status = tc::make_bf16_head_map(&map_k, a.key_cache, total_keys, a.kv_heads, a.dim, kKeys)) != kOk ||
       (status = tc::make_bf16_head_map(&map_v, a.value_cache, total_keys, a.kv_heads, a.value_dim, kKeys)) != kOk)
     return status;
-  const bool capped = a.softcap > 0.0F && a.softcap * 1.4426950408889634F <= kMaxCap;
+  // (a sink of any size needs the running reference)
+  const bool capped = a.softcap > 0.0F && a.softcap * 1.4426950408889634F <= kMaxCap &&
+                      !(a.sink && a.sink_logit != nullptr);
   const auto kernel = capped ? flash_tcgen05_k64_kernel<Form::kCapped> : flash_tcgen05_k64_kernel<Form::kWindow>;
   if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) != cudaSuccess ||
       cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared) !=
@@ -690,6 +693,7 @@ int window_attention_tcgen05(const WindowAttentionArgs &a, cudaStream_t stream) 
   w.gate = static_cast<const bf16 *>(a.gate);
   w.gate_stride = a.gate_stride;
   w.sink = a.sink ? 1 : 0;
+  w.sink_logit = a.sink ? a.sink_logit : nullptr;
   const dim3 grid(ceil_div_u(a.rows, kRows), static_cast<unsigned int>(a.heads));
   kernel<<<grid, kThreads, kSmemBytes, stream>>>(
       map_q, map_k, map_v, static_cast<bf16 *>(a.output), static_cast<int>(a.rows), static_cast<int>(total_keys),

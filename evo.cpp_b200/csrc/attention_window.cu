@@ -134,14 +134,15 @@ struct RowParams {
   const float *distance_bias;
   std::size_t bias_stride, gate_stride;
   int sink;
+  const float *sink_logit;  // [heads] or null: zeros
 };
 
-// Elements of a head that a lane holds: runs of kVec at ((chunk * 8 + part) * kVec), part = lane % 8.
-template <typename T, int kVec, int kElements>
+// Elements of a head that a lane holds: runs of kVec at ((chunk * kLanes + part) * kVec), part = lane % kLanes.
+template <typename T, int kVec, int kElements, int kLanes>
 __device__ __forceinline__ void load_part(const T *const head, const int part, const int dim, float (&v)[kElements]) {
 #pragma unroll
   for (int c = 0; c < kElements / kVec; ++c) {
-    const int base = (c * 8 + part) * kVec;
+    const int base = (c * kLanes + part) * kVec;
     if constexpr (kVec == 8) {
       if (base < dim) {
         float w[8];
@@ -158,15 +159,15 @@ __device__ __forceinline__ void load_part(const T *const head, const int part, c
   }
 }
 
-// kElements * 8 >= max(dim, value_dim)
-template <typename T, int kVec, int kElements>
+// kLanes lanes share a key; kElements * kLanes >= max(dim, value_dim)
+template <typename T, int kVec, int kElements, int kLanes>
 __global__ void __launch_bounds__(kRowThreads)
 window_attention_row_kernel(const T *__restrict__ query, const T *__restrict__ key_cache,
                             const T *__restrict__ value_cache, const T *__restrict__ gate, T *__restrict__ output,
                             const RowParams p) {
   // a one-row projection launched with programmatic stream serialisation may start under this kernel
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  constexpr int kWidth = kElements * 8;
+  constexpr int kWidth = kElements * kLanes, kGroups = 32 / kLanes;  // keys that a warp takes at once
   __shared__ float warp_partials[kRowWarps][kWidth + 2];
   __shared__ float cta_partial[kWidth + 2];
   cg::cluster_group cluster = cg::this_cluster();
@@ -174,7 +175,7 @@ window_attention_row_kernel(const T *__restrict__ query, const T *__restrict__ k
   const int head = blockIdx.y, row = blockIdx.z;
   const int kv = head / (p.heads / p.kv_heads);
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
-  const int group = lane / 8, part = lane % 8;
+  const int group = lane / kLanes, part = lane % kLanes;
   const int position = (p.dynamic_position != nullptr ? *p.dynamic_position : p.position) + row;
   const int low = p.window > 0 ? max(0, position - p.window + 1) : 0;
   const int kept = min(p.keep_first, low);
@@ -185,19 +186,20 @@ window_attention_row_kernel(const T *__restrict__ query, const T *__restrict__ k
                           p.distance_bias != nullptr ? p.distance_bias + head * p.bias_stride : nullptr};
 
   float q[kElements];
-  load_part<T, kVec, kElements>(query + (static_cast<std::size_t>(row) * p.heads + head) * p.dim, part, p.dim, q);
+  load_part<T, kVec, kElements, kLanes>(query + (static_cast<std::size_t>(row) * p.heads + head) * p.dim, part, p.dim, q);
   float running_max = -INFINITY, running_sum = 0.0F, acc[kElements];
 #pragma unroll
   for (int i = 0; i < kElements; ++i) acc[i] = 0.0F;
-  for (int n0 = begin + warp * 4; n0 < end; n0 += kRowWarps * 4) {
+  for (int n0 = begin + warp * kGroups; n0 < end; n0 += kRowWarps * kGroups) {
     const int n = n0 + group;
     const bool live = n < end;
     const int key = n < kept ? n : low + (n - kept);
     float k[kElements], v[kElements];
     if (live) {
-      load_part<T, kVec, kElements>(key_cache + (static_cast<std::size_t>(key) * p.kv_heads + kv) * p.dim, part, p.dim, k);
-      load_part<T, kVec, kElements>(value_cache + (static_cast<std::size_t>(key) * p.kv_heads + kv) * p.value_dim, part,
-                                    p.value_dim, v);
+      load_part<T, kVec, kElements, kLanes>(key_cache + (static_cast<std::size_t>(key) * p.kv_heads + kv) * p.dim, part,
+                                            p.dim, k);
+      load_part<T, kVec, kElements, kLanes>(value_cache + (static_cast<std::size_t>(key) * p.kv_heads + kv) * p.value_dim,
+                                            part, p.value_dim, v);
     } else {
 #pragma unroll
       for (int i = 0; i < kElements; ++i) k[i] = v[i] = 0.0F;
@@ -205,9 +207,8 @@ window_attention_row_kernel(const T *__restrict__ query, const T *__restrict__ k
     float dot = 0.0F;
 #pragma unroll
     for (int i = 0; i < kElements; ++i) dot = fmaf(q[i], k[i], dot);
-    dot += __shfl_xor_sync(0xffffffffU, dot, 1);
-    dot += __shfl_xor_sync(0xffffffffU, dot, 2);
-    dot += __shfl_xor_sync(0xffffffffU, dot, 4);
+#pragma unroll
+    for (int offset = 1; offset < kLanes; offset *= 2) dot += __shfl_xor_sync(0xffffffffU, dot, offset);
     if (live) {
       const float s = capped_score(dot, score, position - key);
       const float next = fmaxf(running_max, s);
@@ -219,9 +220,9 @@ window_attention_row_kernel(const T *__restrict__ query, const T *__restrict__ k
       running_max = next;
     }
   }
-  // the four key groups of a warp hold partials over the same elements per part
+  // the key groups of a warp hold partials over the same elements per part
 #pragma unroll
-  for (int offset = 8; offset <= 16; offset *= 2) {
+  for (int offset = kLanes; offset <= 16; offset *= 2) {
     const float other_m = __shfl_xor_sync(0xffffffffU, running_max, offset);
     const float other_l = __shfl_xor_sync(0xffffffffU, running_sum, offset);
     const float merged = fmaxf(running_max, other_m);
@@ -235,7 +236,7 @@ window_attention_row_kernel(const T *__restrict__ query, const T *__restrict__ k
   }
   if (group == 0) {
 #pragma unroll
-    for (int i = 0; i < kElements; ++i) warp_partials[warp][((i / kVec) * 8 + part) * kVec + i % kVec] = acc[i];
+    for (int i = 0; i < kElements; ++i) warp_partials[warp][((i / kVec) * kLanes + part) * kVec + i % kVec] = acc[i];
     if (part == 0) {
       warp_partials[warp][kWidth] = running_max;
       warp_partials[warp][kWidth + 1] = running_sum;
@@ -260,7 +261,7 @@ window_attention_row_kernel(const T *__restrict__ query, const T *__restrict__ k
         const float *const remote = cluster.map_shared_rank(cta_partial, other);
         merge(m, l, a, remote[kWidth], remote[kWidth + 1], remote[i]);
       }
-      if (p.sink != 0) merge(m, l, a, 0.0F, 1.0F, 0.0F);
+      if (p.sink != 0) merge(m, l, a, p.sink_logit != nullptr ? p.sink_logit[head] : 0.0F, 1.0F, 0.0F);
       float y = a / l;
       if (gate != nullptr) y *= sigmoid_f32(to_float(gate[static_cast<std::size_t>(row) * p.gate_stride + head]));
       output[(static_cast<std::size_t>(row) * p.heads + head) * p.value_dim + i] = from_float<T>(y);
@@ -302,7 +303,7 @@ window_attention_tile_kernel(const T *__restrict__ query, const T *__restrict__ 
   }
   for (int i = threadIdx.x; i < kTileRows * p.value_dim; i += kTileThreads) os[i] = 0.0F;
   if (threadIdx.x < kTileRows) {
-    row_max[threadIdx.x] = p.sink != 0 ? 0.0F : -INFINITY;
+    row_max[threadIdx.x] = p.sink == 0 ? -INFINITY : p.sink_logit != nullptr ? p.sink_logit[head] : 0.0F;
     row_sum[threadIdx.x] = p.sink != 0 ? 1.0F : 0.0F;
   }
   const int low = p.window > 0 ? max(0, first - p.window + 1) : 0;
@@ -386,10 +387,11 @@ RowParams row_params(const WindowAttentionArgs &a) {
   p.bias_stride = a.bias_stride;
   p.gate_stride = a.gate_stride;
   p.sink = a.sink ? 1 : 0;
+  p.sink_logit = a.sink ? a.sink_logit : nullptr;
   return p;
 }
 
-template <typename T, int kVec, int kElements>
+template <typename T, int kVec, int kElements, int kLanes = 8>
 int launch_rows(const WindowAttentionArgs &a, cudaStream_t stream) {
   cudaLaunchAttribute attribute{};
   attribute.id = cudaLaunchAttributeClusterDimension;
@@ -401,7 +403,7 @@ int launch_rows(const WindowAttentionArgs &a, cudaStream_t stream) {
   config.stream = stream;
   config.attrs = &attribute;
   config.numAttrs = 1;
-  if (cudaLaunchKernelEx(&config, window_attention_row_kernel<T, kVec, kElements>, static_cast<const T *>(a.query),
+  if (cudaLaunchKernelEx(&config, window_attention_row_kernel<T, kVec, kElements, kLanes>, static_cast<const T *>(a.query),
                          static_cast<const T *>(a.key_cache), static_cast<const T *>(a.value_cache),
                          static_cast<const T *>(a.gate), static_cast<T *>(a.output), row_params(a)) != cudaSuccess)
     return fail(kCuda, std::string("cannot launch the window attention row kernel: ") +
@@ -417,11 +419,14 @@ int dispatch_rows(const WindowAttentionArgs &a, cudaStream_t stream) {
   if (vector) {
     if (widest <= 64) return launch_rows<T, 8, 8>(a, stream);
     if (widest <= 128) return launch_rows<T, 8, 16>(a, stream);
-    return launch_rows<T, 8, 32>(a, stream);
+    if (widest <= 256) return launch_rows<T, 8, 32>(a, stream);
+    if (widest <= 512) return launch_rows<T, 8, 16, 32>(a, stream);
+    return launch_rows<T, 8, 32, 32>(a, stream);
   }
   if (widest <= 64) return launch_rows<T, 1, 8>(a, stream);
   if (widest <= 128) return launch_rows<T, 1, 16>(a, stream);
-  return launch_rows<T, 1, 32>(a, stream);
+  if (widest <= 256) return launch_rows<T, 1, 32>(a, stream);
+  return launch_rows<T, 1, 32, 32>(a, stream);
 }
 
 template <typename T>
@@ -467,7 +472,7 @@ int head_norm_append(const HeadNormArgs &a, cudaStream_t stream) {
 int window_attention(const WindowAttentionArgs &a, cudaStream_t stream) {
   if (a.query == nullptr || a.key_cache == nullptr || a.value_cache == nullptr || a.output == nullptr ||
       a.heads == 0 || a.heads > 65535 || a.kv_heads == 0 || a.heads % a.kv_heads != 0 || a.dim == 0 ||
-      a.value_dim == 0 || a.dim > kDecoderMaxHeadDim || a.value_dim > kDecoderMaxHeadDim ||
+      a.value_dim == 0 || a.dim > kDecoderMaxLatent || a.value_dim > kDecoderMaxLatent ||
       a.position + a.rows > a.capacity || a.capacity > 0x7fffff00U || a.softcap < 0.0F ||
       (a.distance_bias != nullptr && a.bias_stride < a.position + a.rows))
     return fail(kInvalidArgument, "window attention arguments are invalid");
@@ -476,11 +481,13 @@ int window_attention(const WindowAttentionArgs &a, cudaStream_t stream) {
     if (window_attention_tcgen05_applicable(a)) return window_attention_tcgen05(a, stream);
     if (a.force == 3) return fail(kUnsupported, "the tensor-core attention kernel does not take these sizes");
   }
-  if (a.force == 1 || (a.force == 0 && a.rows <= 8)) {
+  const bool wide = a.dim > kDecoderMaxHeadDim || a.value_dim > kDecoderMaxHeadDim;
+  if (a.force == 1 || (a.force == 0 && (a.rows <= 8 || wide))) {
     if (a.rows > 65535) return fail(kInvalidArgument, "too many rows for the row kernel");
     return a.type == Activation::kBf16 ? dispatch_rows<bf16>(a, stream) : dispatch_rows<float>(a, stream);
   }
   if (a.dynamic_position != nullptr) return fail(kInvalidArgument, "replayed attention launches take few rows");
+  if (wide) return fail(kUnsupported, "the tile kernel does not take heads of this size");
   return a.type == Activation::kBf16 ? launch_tiles<bf16>(a, stream) : launch_tiles<float>(a, stream);
 }
 

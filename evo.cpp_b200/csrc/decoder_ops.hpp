@@ -13,6 +13,8 @@
 namespace evob {
 
 constexpr std::size_t kDecoderMaxHeadDim = 256;
+constexpr std::size_t kDecoderMaxLatent = 1024;  // widest latent of latent attention (row kernel)
+constexpr std::size_t kDecoderMaxExperts = 1024;
 
 enum class Activation { kBf16, kF32 };
 inline std::size_t activation_bytes(const Activation a) { return a == Activation::kBf16 ? 2 : 4; }
@@ -33,9 +35,112 @@ int poly_norm(const void *input, const float *coefficients, std::size_t rows, st
 // table[h, d] = r1[h] ln(1 + r2[h] d), d < distances.
 int distance_bias_table(const float *r1, const float *r2, std::size_t heads, std::size_t distances, float *table,
                         cudaStream_t stream);
-// F32 [rows, in] x BF16 [out, in]^T in F32 fused multiply-adds: output (+)= product.
+// [rows, in] (F32 or BF16) x BF16 [out, in]^T in F32 fused multiply-adds.  output = [output +] alpha *
+// row_scale[r] * product + bias, then softcap tanh(output / softcap) where softcap > 0.  Grouped weights
+// [groups, out, in]: see LinearArgs (row_group / row_fanout, or tile_group / tile_count / tile_rows).
+struct LinearF32Args {
+  const void *input = nullptr;
+  Activation input_type = Activation::kF32;
+  const void *weight = nullptr;
+  float *output = nullptr;
+  std::size_t rows = 0, in_features = 0, out_features = 0;
+  bool accumulate = false;
+  float alpha = 1.0F, softcap = 0.0F;
+  const float *row_scale = nullptr, *bias = nullptr;
+  const int *row_group = nullptr;
+  std::size_t row_fanout = 1;
+  const int *tile_group = nullptr, *tile_count = nullptr;
+  std::size_t tile_rows = 128;
+};
+int linear_f32(const LinearF32Args &args, cudaStream_t stream);
 int linear_f32(const float *input, const void *weight, std::size_t rows, std::size_t in_features,
                std::size_t out_features, float *output, bool accumulate, cudaStream_t stream);
+// stream[r, :] = table[token[r], :] in F32, and the same row in `copy` (optional).  Ids >= vocabulary: see embedding().
+int embed_rows(const std::uint32_t *tokens, const void *table, std::size_t rows, std::size_t width,
+               std::size_t vocabulary, float *stream_rows, void *copy, Activation type, cudaStream_t stream);
+// Row r of the input is y = the sum of its `parts` rows (row slots[r * parts + k], or r * parts + k without
+// slots); n = (y - mean) / sqrt(variance + epsilon) * gain.  With a residual: residual[r, :] += n, and the new
+// residual row goes to `output` (optional); without: n goes to `output`.
+struct LayerNormArgs {
+  const void *input = nullptr;
+  Activation input_type = Activation::kF32;
+  const int *slots = nullptr;
+  std::size_t parts = 1;
+  const float *gain = nullptr;
+  float *residual = nullptr;
+  void *output = nullptr;
+  Activation output_type = Activation::kF32;
+  std::size_t rows = 0, width = 0;
+  float epsilon = 1e-6F;
+};
+int layer_norm(const LayerNormArgs &args, cudaStream_t stream);
+// F32 rows in the activation type.
+int convert_rows(const float *input, std::size_t elements, void *output, Activation type, cudaStream_t stream);
+// Gated activation of row-interleaved products [rows, 2 * inner] (blocks of 128 gate columns followed by the
+// matching 128 up columns), `gate` as LinearArgs::gate_mode 3 and 4; with tile_count only its tiles' rows are live.
+int gated_activation(const float *input, int gate, float limit, std::size_t rows, std::size_t inner, void *output,
+                     Activation type, const int *tile_count, std::size_t tile_rows, cudaStream_t stream);
+
+// ---- experts.cu
+// Router of a mixture of experts: scores sigmoid(x . router[e]) in F32, the `top` largest, best first, ties to
+// the lower index.  The products come from `logits` [rows, logit_stride] where given; else the kernel makes
+// them itself (few rows).  Results per (row, place): expert id and score.
+struct RouteArgs {
+  const void *input = nullptr;    // [rows, width], without logits
+  Activation type = Activation::kBf16;
+  const void *router = nullptr;   // [experts, width] BF16
+  const float *logits = nullptr;
+  std::size_t logit_stride = 0;
+  std::size_t rows = 0, width = 0, experts = 0, top = 0;
+  int *expert = nullptr;          // [rows * top]
+  float *score = nullptr;         // [rows * top]
+  // with counts (zeroed by the launch): counts[e] = rows that chose e, rank = a pair's place among them
+  int *counts = nullptr, *rank = nullptr;
+};
+int route_rows(const RouteArgs &args, cudaStream_t stream);
+// Rows grouped by expert: expert e owns whole tiles of tile_rows rows of `grouped`, in the order of the experts.
+// grouped[slot[pair], :] = input[pair / top, :], slot_score[slot[pair]] = score[pair]; tile_group[t] = expert of
+// tile t, *tile_count = tiles in use (at most grouped_tiles()).  Rows that fill up a tile are left as they are.
+struct GroupRowsArgs {
+  const void *input = nullptr;
+  Activation type = Activation::kBf16;
+  std::size_t rows = 0, width = 0, experts = 0, top = 0, tile_rows = 128;
+  const int *expert = nullptr, *rank = nullptr, *counts = nullptr;
+  const float *score = nullptr;
+  void *grouped = nullptr;
+  float *slot_score = nullptr;
+  int *slot = nullptr, *tile_group = nullptr, *tile_count = nullptr;
+};
+int group_rows(const GroupRowsArgs &args, cudaStream_t stream);
+inline std::size_t grouped_tiles(const std::size_t rows, const std::size_t top, const std::size_t experts,
+                                 const std::size_t tile_rows) {
+  const std::size_t pairs = rows * top;
+  return pairs / tile_rows + (pairs < experts ? pairs : experts);
+}
+
+// ---- latent_attention.cu
+// Row r of `projection` ([rows, stride]) holds the query latent at column 0 and the key/value latent at
+// latent_column.  Both are RMS-normed with their gains: the first goes to query_latent [rows, query_rank], the
+// second to row position + r of the cache [capacity, latent_rank].
+struct LatentNormArgs {
+  const void *projection = nullptr;
+  std::size_t stride = 0, latent_column = 0;
+  const float *query_gain = nullptr, *latent_gain = nullptr;
+  void *query_latent = nullptr, *cache = nullptr;
+  std::size_t rows = 0, position = 0, capacity = 0, query_rank = 0, latent_rank = 0;
+  float epsilon = 1e-6F;
+  Activation type = Activation::kBf16;
+  const int *dynamic_position = nullptr;
+};
+int latent_norm_append(const LatentNormArgs &args, cudaStream_t stream);
+// Few rows: the per-head up projections moved to the query and output side, so that attention runs on the
+// cached latents themselves.  absorbed[r, h, :] = sum_d query[r, h, d] key_up[h * dim + d, :], and
+// output[r, h, d] = value_up[h * value_dim + d, :] . mixed[r, h, :].  At most kLatentRows rows.
+constexpr std::size_t kLatentRows = 8;
+int absorb_queries(const void *query, const void *key_up, std::size_t rows, std::size_t heads, std::size_t dim,
+                   std::size_t latent_rank, void *absorbed, Activation type, cudaStream_t stream);
+int expand_values(const void *mixed, const void *value_up, std::size_t rows, std::size_t heads, std::size_t value_dim,
+                  std::size_t latent_rank, void *output, Activation type, cudaStream_t stream);
 
 // ---- attention_window.cu
 // Row r of `projection` ([rows, stride]) holds query heads at column 0, key heads at key_column, value heads
@@ -56,8 +161,9 @@ int head_norm_append(const HeadNormArgs &args, cudaStream_t stream);
 // Softmax attention of `rows` queries at positions position .. against the cached keys.  Query i sees key
 // j <= i if i - j < window (window 0: no limit) or j < keep_first.  score = softcap tanh(q.k scale / softcap)
 // (softcap 0: plain) - distance_bias[head, i - j] (optional); with `sink` the softmax denominator has one
-// more term exp(0) without a value.  Head h uses key/value head h / (heads / kv_heads).  output[r, h, :] is
-// multiplied by sigmoid(gate[r * gate_stride + h]) when a gate is given.
+// more term exp(sink_logit[head]) (exp(0) without sink_logit) that has no value.  Head h uses key/value head h / (heads / kv_heads).  output[r, h, :] is
+// multiplied by sigmoid(gate[r * gate_stride + h]) when a gate is given.  Heads above kDecoderMaxHeadDim (up to
+// kDecoderMaxLatent) run in the row kernel only.
 struct WindowAttentionArgs {
   const void *query = nullptr, *key_cache = nullptr, *value_cache = nullptr;
   const void *gate = nullptr;
@@ -69,6 +175,7 @@ struct WindowAttentionArgs {
   std::size_t window = 0, keep_first = 0;
   float scale = 1.0F, softcap = 0.0F;
   bool sink = false;
+  const float *sink_logit = nullptr;  // [heads]
   Activation type = Activation::kBf16;
   const int *dynamic_position = nullptr;
   int force = 0;  // tests: 1 the row kernel, 2 the tile kernel, 3 the tcgen05 kernel (refused where it does not apply)

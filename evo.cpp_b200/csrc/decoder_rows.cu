@@ -1,6 +1,8 @@
-// Row operators of the decoder graph: embedding with learned positions, the norm of the F32 residual
-// stream, the normalised polynomial activation, and the F32 projection of the F32 profile.
+// Row operators of the decoder graph: embeddings (with and without learned positions), the norms of the F32
+// residual stream and of what is added to it, the activations of the feed-forwards, and the F32 projection of
+// the F32 profile.
 #include "decoder_types.cuh"
+#include "gates.cuh"
 #include "ops_internal.hpp"
 
 namespace evob {
@@ -189,23 +191,192 @@ distance_bias_kernel(const float *__restrict__ r1, const float *__restrict__ r2,
     table[static_cast<std::size_t>(head) * distances + d] = r1[head] * logf(fmaf(r2[head], static_cast<float>(d), 1.0F));
 }
 
+template <typename T, bool kVector>
+__global__ void __launch_bounds__(kThreads)
+embed_rows_kernel(const std::uint32_t *__restrict__ tokens, const bf16 *__restrict__ table, const int width,
+                  const std::uint32_t vocabulary, float *__restrict__ stream_rows, T *__restrict__ copy,
+                  int *const error_word) {
+  const std::size_t row = blockIdx.x;
+  const std::uint32_t token = tokens[row];
+  const bool known = token < vocabulary;
+  if (!known && threadIdx.x == 0) atomicOr(error_word, 2);
+  const bf16 *const word = table + static_cast<std::size_t>(known ? token : 0U) * width;
+  for (int group = threadIdx.x; group < (width + 7) / 8; group += kThreads) {
+    float v[8];
+    load_group<bf16, kVector>(word, group, width, v);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = known ? v[i] : 0.0F;
+    store_group<float, kVector>(stream_rows + row * width, group, width, v);
+    if (copy != nullptr) store_group<T, kVector>(copy + row * width, group, width, v);
+  }
+}
+
+struct LayerNormParams {
+  const int *slots;
+  int parts;
+  const float *gain;
+  float *residual;
+  int width;
+  float epsilon;
+};
+
+// Mean and variance from the row itself (two sweeps over registers), one read and one write of the residual.
+template <typename In, typename Out, bool kVector>
+__global__ void __launch_bounds__(kThreads)
+layer_norm_kernel(const In *__restrict__ input, Out *__restrict__ output, const LayerNormParams p) {
+  // a one-row projection launched with programmatic stream serialisation may start under this kernel
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  __shared__ float scratch[kThreads / 32];
+  const std::size_t row = blockIdx.x;
+  const int groups = (p.width + 7) / 8;
+  const float inverse_width = 1.0F / static_cast<float>(p.width);
+  const auto load = [&](const int group, float (&v)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = 0.0F;
+    for (int k = 0; k < p.parts; ++k) {
+      const std::size_t pair = row * p.parts + k;
+      const std::size_t at = p.slots != nullptr ? static_cast<std::size_t>(p.slots[pair]) : pair;
+      float w[8];
+      load_group<In, kVector>(input + at * p.width, group, p.width, w);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[i] += w[i];
+    }
+  };
+  const auto live = [&](const int group, const int i) { return kVector || 8 * group + i < p.width; };
+  float cached[kCached][8], old[kCached][8];
+  float sum = 0.0F;
+#pragma unroll
+  for (int c = 0; c < kCached; ++c) {
+    const int group = threadIdx.x + c * kThreads;
+    if (group < groups) {
+      load(group, cached[c]);
+      if (p.residual != nullptr) load_group<float, kVector>(p.residual + row * p.width, group, p.width, old[c]);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) sum += cached[c][i];
+    }
+  }
+  for (int group = threadIdx.x + kCached * kThreads; group < groups; group += kThreads) {
+    float v[8];
+    load(group, v);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) sum += v[i];
+  }
+  const float mean = block_sum<kThreads>(sum, scratch) * inverse_width;
+  float square = 0.0F;
+  const auto deviate = [&](const int group, const float (&v)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float d = live(group, i) ? v[i] - mean : 0.0F;
+      square = fmaf(d, d, square);
+    }
+  };
+#pragma unroll
+  for (int c = 0; c < kCached; ++c) {
+    const int group = threadIdx.x + c * kThreads;
+    if (group < groups) deviate(group, cached[c]);
+  }
+  for (int group = threadIdx.x + kCached * kThreads; group < groups; group += kThreads) {
+    float v[8];
+    load(group, v);
+    deviate(group, v);
+  }
+  const float factor = 1.0F / sqrtf(block_sum<kThreads>(square, scratch) * inverse_width + p.epsilon);
+  const auto emit = [&](const int group, const float (&v)[8], const float (&before)[8]) {
+    float g[8], y[8];
+    load_group<float, kVector>(p.gain, group, p.width, g);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = (v[i] - mean) * factor * g[i];
+    if (p.residual != nullptr) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] += before[i];
+      store_group<float, kVector>(p.residual + row * p.width, group, p.width, y);
+    }
+    if (output != nullptr) store_group<Out, kVector>(output + row * p.width, group, p.width, y);
+  };
+#pragma unroll
+  for (int c = 0; c < kCached; ++c) {
+    const int group = threadIdx.x + c * kThreads;
+    if (group < groups) emit(group, cached[c], old[c]);
+  }
+  for (int group = threadIdx.x + kCached * kThreads; group < groups; group += kThreads) {
+    float v[8], before[8] = {};
+    load(group, v);
+    if (p.residual != nullptr) load_group<float, kVector>(p.residual + row * p.width, group, p.width, before);
+    emit(group, v, before);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+convert_kernel(const float *__restrict__ input, T *__restrict__ output, const std::size_t elements) {
+  const std::size_t stride = static_cast<std::size_t>(gridDim.x) * kThreads;
+  for (std::size_t i = static_cast<std::size_t>(blockIdx.x) * kThreads + threadIdx.x; i < elements; i += stride)
+    output[i] = from_float<T>(input[i]);
+}
+
+// One row of one 128-column block of the output per iteration.
+template <typename T>
+__global__ void __launch_bounds__(128)
+gated_activation_kernel(const float *__restrict__ input, T *__restrict__ output, const int gate, const float limit,
+                        const std::size_t rows, const int inner, const int *__restrict__ tile_count, const int tile_rows) {
+  std::size_t live = rows;
+  if (tile_count != nullptr) {
+    const std::size_t used = static_cast<std::size_t>(*tile_count) * tile_rows;
+    live = used < rows ? used : rows;
+  }
+  const int block = blockIdx.y, column = block * 128 + static_cast<int>(threadIdx.x);
+  for (std::size_t row = blockIdx.x; row < live; row += gridDim.x) {
+    const float *const pair = input + row * 2 * inner + 256 * block + threadIdx.x;
+    output[row * inner + column] = from_float<T>(gated_value(gate, limit, pair[0], pair[128]));
+  }
+}
+
+struct F32Params {
+  const bf16 *weight;
+  float *output;
+  int rows, out_features, in_features, accumulate;
+  float alpha, softcap;
+  const float *row_scale, *bias;
+  const int *row_group;
+  int row_fanout;
+  const int *tile_group, *tile_count;
+  int tile_rows;
+};
+
+__device__ __forceinline__ void store_f32_result(const F32Params &p, const std::size_t row, const int column,
+                                                 const float product) {
+  float *const out = p.output + row * p.out_features + column;
+  float value = product * (p.row_scale != nullptr ? p.alpha * p.row_scale[row] : p.alpha);
+  if (p.accumulate != 0) value += *out;
+  if (p.bias != nullptr) value += p.bias[column];
+  *out = soft_cap(value, p.softcap);
+}
+
 // 64 x 64 output tile, 16 inputs per step, 4 x 4 products per thread; plain F32 multiply-adds, every step's 16
 // products summed on their own before they join the running sum.
+template <typename T>
 __global__ void __launch_bounds__(256)
-linear_f32_kernel(const float *__restrict__ input, const bf16 *__restrict__ weight, float *__restrict__ output,
-                  const int rows, const int out_features, const int in_features, const bool accumulate) {
+linear_f32_kernel(const T *__restrict__ input, const F32Params p) {
   __shared__ float x_tile[16][68];
   __shared__ float w_tile[16][68];
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const bf16 *weight = p.weight;
+  if (p.tile_group != nullptr) {
+    const int tile = m0 / p.tile_rows;
+    if (tile >= *p.tile_count) return;
+    weight += static_cast<std::size_t>(p.tile_group[tile]) * p.out_features * p.in_features;
+  }
   float acc[4][4] = {};
-  for (int k0 = 0; k0 < in_features; k0 += 16) {
+  for (int k0 = 0; k0 < p.in_features; k0 += 16) {
     for (int i = threadIdx.x; i < 64 * 16; i += 256) {
       const int r = i / 16, k = i % 16;
-      const bool inside = k0 + k < in_features;
-      x_tile[k][r] = m0 + r < rows && inside ? input[static_cast<std::size_t>(m0 + r) * in_features + k0 + k] : 0.0F;
-      w_tile[k][r] =
-          n0 + r < out_features && inside ? bf2f(weight[static_cast<std::size_t>(n0 + r) * in_features + k0 + k]) : 0.0F;
+      const bool inside = k0 + k < p.in_features;
+      x_tile[k][r] =
+          m0 + r < p.rows && inside ? to_float(input[static_cast<std::size_t>(m0 + r) * p.in_features + k0 + k]) : 0.0F;
+      w_tile[k][r] = n0 + r < p.out_features && inside
+                         ? bf2f(weight[static_cast<std::size_t>(n0 + r) * p.in_features + k0 + k])
+                         : 0.0F;
     }
     __syncthreads();
     float step[4][4] = {};
@@ -228,25 +399,24 @@ linear_f32_kernel(const float *__restrict__ input, const bf16 *__restrict__ weig
   for (int i = 0; i < 4; ++i)
     for (int j = 0; j < 4; ++j) {
       const int row = m0 + ty * 4 + i, col = n0 + tx * 4 + j;
-      if (row >= rows || col >= out_features) continue;
-      float *const out = output + static_cast<std::size_t>(row) * out_features + col;
-      *out = accumulate ? *out + acc[i][j] : acc[i][j];
+      if (row < p.rows && col < p.out_features) store_f32_result(p, static_cast<std::size_t>(row), col, acc[i][j]);
     }
 }
 
 // Few rows: a warp per (row, output).
+template <typename T>
 __global__ void __launch_bounds__(256)
-linear_f32_rows_kernel(const float *__restrict__ input, const bf16 *__restrict__ weight, float *__restrict__ output,
-                       const int out_features, const int in_features, const bool accumulate) {
+linear_f32_rows_kernel(const T *__restrict__ input, const F32Params p) {
   const int column = blockIdx.x * 8 + threadIdx.x / 32, lane = threadIdx.x % 32;
-  if (column >= out_features) return;
-  const float *const x = input + static_cast<std::size_t>(blockIdx.y) * in_features;
-  const bf16 *const w = weight + static_cast<std::size_t>(column) * in_features;
+  if (column >= p.out_features) return;
+  const std::size_t row = blockIdx.y;
+  const T *const x = input + row / p.row_fanout * p.in_features;
+  const std::size_t group = p.row_group != nullptr ? static_cast<std::size_t>(p.row_group[row]) : 0;
+  const bf16 *const w = p.weight + (group * p.out_features + column) * p.in_features;
   float sum = 0.0F;
-  for (int k = lane; k < in_features; k += 32) sum = fmaf(x[k], bf2f(w[k]), sum);
+  for (int k = lane; k < p.in_features; k += 32) sum = fmaf(to_float(x[k]), bf2f(w[k]), sum);
   sum = warp_sum(sum);
-  float *const out = output + static_cast<std::size_t>(blockIdx.y) * out_features + column;
-  if (lane == 0) *out = accumulate ? *out + sum : sum;
+  if (lane == 0) store_f32_result(p, row, column, sum);
 }
 
 bool row_vector_ok(const std::size_t width, const void *a, const void *b, const void *c) {
@@ -325,24 +495,137 @@ int distance_bias_table(const float *r1, const float *r2, const std::size_t head
   return check_launch("distance bias kernel");
 }
 
+int embed_rows(const std::uint32_t *tokens, const void *table, const std::size_t rows, const std::size_t width,
+               const std::size_t vocabulary, float *stream_rows, void *copy, const Activation type, cudaStream_t stream) {
+  if (tokens == nullptr || table == nullptr || stream_rows == nullptr || width == 0 || width > 0x7fffff00U ||
+      rows > 0x7fffffffU)
+    return fail(kInvalidArgument, "embedding arguments are invalid");
+  if (rows == 0) return kOk;
+  int status = kOk;
+  int *const error = device_error_word(&status);
+  if (error == nullptr) return status;
+  const bool vector = row_vector_ok(width, table, stream_rows, copy);
+  const auto launch = [&](auto tag) {
+    using T = decltype(tag);
+    const auto kernel = vector ? embed_rows_kernel<T, true> : embed_rows_kernel<T, false>;
+    kernel<<<static_cast<unsigned int>(rows), kThreads, 0, stream>>>(tokens, static_cast<const bf16 *>(table),
+                                                                     static_cast<int>(width),
+                                                                     static_cast<std::uint32_t>(vocabulary), stream_rows,
+                                                                     static_cast<T *>(copy), error);
+  };
+  if (type == Activation::kBf16) launch(bf16{});
+  else launch(float{});
+  return check_launch("embedding kernel of the residual stream");
+}
+
+int layer_norm(const LayerNormArgs &a, cudaStream_t stream) {
+  if (a.input == nullptr || a.gain == nullptr || (a.residual == nullptr && a.output == nullptr) || a.parts == 0 ||
+      a.parts > 0x7fffffffU || a.width == 0 || a.width > 0x7fffff00U || a.rows > 0x7fffffffU)
+    return fail(kInvalidArgument, "layer norm arguments are invalid");
+  if (a.rows == 0) return kOk;
+  const bool vector = row_vector_ok(a.width, a.input, a.gain, a.output) && aligned16(a.residual);
+  LayerNormParams p{};
+  p.slots = a.slots;
+  p.parts = static_cast<int>(a.parts);
+  p.gain = a.gain;
+  p.residual = a.residual;
+  p.width = static_cast<int>(a.width);
+  p.epsilon = a.epsilon;
+  const auto launch = [&](auto in_tag, auto out_tag) {
+    using In = decltype(in_tag);
+    using Out = decltype(out_tag);
+    const auto kernel = vector ? layer_norm_kernel<In, Out, true> : layer_norm_kernel<In, Out, false>;
+    kernel<<<static_cast<unsigned int>(a.rows), kThreads, 0, stream>>>(static_cast<const In *>(a.input),
+                                                                       static_cast<Out *>(a.output), p);
+  };
+  if (a.input_type == Activation::kBf16) {
+    if (a.output_type == Activation::kBf16) launch(bf16{}, bf16{});
+    else launch(bf16{}, float{});
+  } else {
+    if (a.output_type == Activation::kBf16) launch(float{}, bf16{});
+    else launch(float{}, float{});
+  }
+  return check_launch("layer norm kernel");
+}
+
+int convert_rows(const float *input, const std::size_t elements, void *output, const Activation type, cudaStream_t stream) {
+  if (input == nullptr || output == nullptr) return fail(kInvalidArgument, "conversion arguments are invalid");
+  if (elements == 0) return kOk;
+  const std::size_t blocks = (elements + kThreads - 1) / kThreads;
+  const unsigned int grid = static_cast<unsigned int>(blocks < 8 * kSmCount ? blocks : 8 * kSmCount);
+  if (type == Activation::kBf16)
+    convert_kernel<<<grid, kThreads, 0, stream>>>(input, static_cast<bf16 *>(output), elements);
+  else
+    convert_kernel<<<grid, kThreads, 0, stream>>>(input, static_cast<float *>(output), elements);
+  return check_launch("conversion kernel");
+}
+
+int gated_activation(const float *input, const int gate, const float limit, const std::size_t rows,
+                     const std::size_t inner, void *output, const Activation type, const int *tile_count,
+                     const std::size_t tile_rows, cudaStream_t stream) {
+  if (input == nullptr || output == nullptr || (gate != kGateRelu && gate != kGateClamped) || inner == 0 || inner % 128 != 0 ||
+      inner / 128 > 65535 || inner > 0x3fffff00U || tile_rows > 0x7fffffffU)
+    return fail(kInvalidArgument, "gated activation arguments are invalid");
+  if (rows == 0) return kOk;
+  const dim3 grid(static_cast<unsigned int>(rows < 65536 ? rows : 65536), static_cast<unsigned int>(inner / 128));
+  if (type == Activation::kBf16)
+    gated_activation_kernel<<<grid, 128, 0, stream>>>(input, static_cast<bf16 *>(output), gate, limit, rows,
+                                                      static_cast<int>(inner), tile_count, static_cast<int>(tile_rows));
+  else
+    gated_activation_kernel<<<grid, 128, 0, stream>>>(input, static_cast<float *>(output), gate, limit, rows,
+                                                      static_cast<int>(inner), tile_count, static_cast<int>(tile_rows));
+  return check_launch("gated activation kernel");
+}
+
+int linear_f32(const LinearF32Args &a, cudaStream_t stream) {
+  if (a.input == nullptr || a.weight == nullptr || a.output == nullptr || a.in_features == 0 || a.out_features == 0 ||
+      a.in_features > 0x7fffff00U || a.out_features > 0x7fffff00U || a.rows > 64 * 65535U || a.row_fanout == 0 ||
+      (a.tile_group != nullptr && (a.tile_count == nullptr || a.tile_rows % 64 != 0 || a.row_group != nullptr)) ||
+      (a.row_group != nullptr && a.rows > 65535U))
+    return fail(kInvalidArgument, "F32 linear arguments are invalid");
+  if (a.rows == 0) return kOk;
+  F32Params p{};
+  p.weight = static_cast<const bf16 *>(a.weight);
+  p.output = a.output;
+  p.rows = static_cast<int>(a.rows);
+  p.out_features = static_cast<int>(a.out_features);
+  p.in_features = static_cast<int>(a.in_features);
+  p.accumulate = a.accumulate ? 1 : 0;
+  p.alpha = a.alpha;
+  p.softcap = a.softcap;
+  p.row_scale = a.row_scale;
+  p.bias = a.bias;
+  p.row_group = a.row_group;
+  p.row_fanout = static_cast<int>(a.row_fanout);
+  p.tile_group = a.tile_group;
+  p.tile_count = a.tile_count;
+  p.tile_rows = static_cast<int>(a.tile_rows);
+  const auto launch = [&](auto tag) {
+    using T = decltype(tag);
+    const T *const input = static_cast<const T *>(a.input);
+    if (a.row_group != nullptr || (a.rows <= 16 && a.tile_group == nullptr)) {
+      const dim3 grid(ceil_div_u(a.out_features, 8), static_cast<unsigned int>(a.rows));
+      linear_f32_rows_kernel<T><<<grid, 256, 0, stream>>>(input, p);
+      return check_launch("F32 linear kernel (few rows)");
+    }
+    const dim3 grid(ceil_div_u(a.out_features, 64), ceil_div_u(a.rows, 64));
+    linear_f32_kernel<T><<<grid, 256, 0, stream>>>(input, p);
+    return check_launch("F32 linear kernel");
+  };
+  return a.input_type == Activation::kBf16 ? launch(bf16{}) : launch(float{});
+}
+
 int linear_f32(const float *input, const void *weight, const std::size_t rows, const std::size_t in_features,
                const std::size_t out_features, float *output, const bool accumulate, cudaStream_t stream) {
-  if (input == nullptr || weight == nullptr || output == nullptr || in_features == 0 || out_features == 0 ||
-      in_features > 0x7fffff00U || out_features > 0x7fffff00U || rows > 64 * 65535U)
-    return fail(kInvalidArgument, "F32 linear arguments are invalid");
-  if (rows == 0) return kOk;
-  if (rows <= 16) {
-    const dim3 grid(ceil_div_u(out_features, 8), static_cast<unsigned int>(rows));
-    linear_f32_rows_kernel<<<grid, 256, 0, stream>>>(input, static_cast<const bf16 *>(weight), output,
-                                                     static_cast<int>(out_features), static_cast<int>(in_features),
-                                                     accumulate);
-    return check_launch("F32 linear kernel (few rows)");
-  }
-  const dim3 grid(ceil_div_u(out_features, 64), ceil_div_u(rows, 64));
-  linear_f32_kernel<<<grid, 256, 0, stream>>>(input, static_cast<const bf16 *>(weight), output, static_cast<int>(rows),
-                                              static_cast<int>(out_features), static_cast<int>(in_features),
-                                              accumulate);
-  return check_launch("F32 linear kernel");
+  LinearF32Args a;
+  a.input = input;
+  a.weight = weight;
+  a.rows = rows;
+  a.in_features = in_features;
+  a.out_features = out_features;
+  a.output = output;
+  a.accumulate = accumulate;
+  return linear_f32(a, stream);
 }
 
 }  // namespace evob

@@ -30,6 +30,7 @@
 #include <type_traits>
 
 #include "common.cuh"
+#include "gates.cuh"
 #include "ops_internal.hpp"
 #include "tcgen05.cuh"
 
@@ -49,7 +50,8 @@ struct EpilogueParams {
   float alpha;
   const float *row_scale;  // optional [M]: row r's accumulator is also multiplied by row_scale[r]
   int bias_mode;  // 0 none, 1 fused into the F32 sum, 2 separate BF16 add
-  int gate_mode;  // 0 none, 1 first*second halves, 2 gelu(first)*second
+  int gate_mode;  // LinearArgs::gate_mode
+  float gate_limit;
   // F32 result mode (split-precision products): out_f32 = [out_f32 +] alpha*acc [+ bias_f32]
   float *out_f32;
   const float *bias_f32;
@@ -62,6 +64,9 @@ struct EpilogueParams {
   // partial sums to out_f32 + split * partial_stride; a second kernel adds them up in order.
   int split_k;
   std::size_t partial_stride;
+  float softcap;
+  // Grouped weights: row tile t multiplies the N weight rows of group tile_group[t]; *tile_count row tiles exist.
+  const int *tile_group, *tile_count;
 };
 
 using namespace tc;
@@ -177,9 +182,13 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const int r = m0 + quarter * 32 + 4 * i + lane / 8;
-            if (r < M)
-              *reinterpret_cast<float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at) =
-                  make_float4(sums[i].x + shift.x, sums[i].y + shift.y, sums[i].z + shift.z, sums[i].w + shift.w);
+            if (r >= M) continue;
+            float4 result =
+                make_float4(sums[i].x + shift.x, sums[i].y + shift.y, sums[i].z + shift.z, sums[i].w + shift.w);
+            if (ep.softcap > 0.0F)
+              result = make_float4(soft_cap(result.x, ep.softcap), soft_cap(result.y, ep.softcap),
+                                   soft_cap(result.z, ep.softcap), soft_cap(result.w, ep.softcap));
+            *reinterpret_cast<float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at) = result;
           }
         }
         continue;
@@ -192,7 +201,7 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
             float value = __uint_as_float(v[j]) * scale;
             if (ep.bias_f32 != nullptr) value += ep.bias_f32[col + j];
             if (ep.accumulate_f32 != 0) value += out_row[col + j];
-            out_row[col + j] = value;
+            out_row[col + j] = soft_cap(value, ep.softcap);
           }
         }
       }
@@ -204,7 +213,15 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
         float value = __uint_as_float(v[j]) * scale;
-        if (gated) {
+        if (ep.gate_mode >= kGateRelu) {
+          // (the weight rows of this output column: n0 + c * 32 + j, and 128 further on)
+          float up = __uint_as_float(w[j]) * scale;
+          if (ep.bias_f32 != nullptr) {
+            value += __ldg(ep.bias_f32 + n0 + c * 32 + j);
+            up += __ldg(ep.bias_f32 + n0 + BN / 2 + c * 32 + j);
+          }
+          r[j] = gated_value(ep.gate_mode, ep.gate_limit, value, up);
+        } else if (gated) {
           const float first =
               ep.gate_mode == 2 ? bf2f(gelu_round(value)) : rbf(value);
           const float second = rbf(__uint_as_float(w[j]) * scale);
@@ -326,7 +343,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
   tc_fence_after();
   const std::uint32_t tmem_base = *tmem_ptr;
 
-  const int tiles_m = (M + kBlockM - 1) / kBlockM;
+  const int tiles_m = ep.tile_count != nullptr ? min(*ep.tile_count, (M + kBlockM - 1) / kBlockM) : (M + kBlockM - 1) / kBlockM;
   const int tiles_n = (N + BN - 1) / BN;
   const int splits = ep.split_k > 1 ? ep.split_k : 1;
   const int tiles_mn = tiles_m * tiles_n;
@@ -343,7 +360,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
         int tile_m, tile_n;
         tile_coordinates(tile % tiles_mn, tiles_m, tiles_n, &tile_m, &tile_n);
         const int m0 = tile_m * kBlockM;
-        const int n0 = tile_n * BN;
+        const int n0 = tile_n * BN + (ep.tile_group != nullptr ? __ldg(ep.tile_group + tile_m) * N : 0);
         const int kb_begin = (tile / tiles_mn) * k_per_split;
         for (int kb = kb_begin; kb < kb_begin + k_per_split; ++kb) {
           if (!mbar_wait(empty_bar(stage), phase ^ 1U, abort_flag)) {
@@ -575,7 +592,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
   tc_fence_after();
   const std::uint32_t tmem_base = *tmem_ptr;
 
-  const int tiles_m = (M + 255) / 256;
+  const int tiles_m = ep.tile_count != nullptr ? min(*ep.tile_count, (M + 255) / 256) : (M + 255) / 256;
   const int tiles_n = (N + kPairN - 1) / kPairN;
   const int splits = ep.split_k > 1 ? ep.split_k : 1;
   const int tiles_mn = tiles_m * tiles_n;
@@ -593,7 +610,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
         int tile_m, tile_n;
         tile_coordinates(tile % tiles_mn, tiles_m, tiles_n, &tile_m, &tile_n);
         const int m0 = tile_m * 256 + static_cast<int>(rank) * 128;
-        const int n0 = tile_n * kPairN + static_cast<int>(rank) * 128;
+        const int n0 = tile_n * kPairN + static_cast<int>(rank) * 128 +
+                       (ep.tile_group != nullptr ? __ldg(ep.tile_group + tile_m) * N : 0);
         const int kb_begin = (tile / tiles_mn) * k_per_split;
         for (int kb = kb_begin; kb < kb_begin + k_per_split; ++kb) {
           if (!mbar_wait(empty_bar(stage), phase ^ 1U, abort_flag)) {
@@ -897,7 +915,7 @@ gemm_simt_kernel(const void *__restrict__ a_raw, const void *__restrict__ b_raw,
       if (ep.out_f32 != nullptr) {
         float *const slot = ep.out_f32 + static_cast<std::size_t>(row) * ep.ld_out + col;
         if (ep.bias_f32 != nullptr) value += ep.bias_f32[col];
-        *slot = ep.accumulate_f32 != 0 ? *slot + value : value;
+        *slot = soft_cap(ep.accumulate_f32 != 0 ? *slot + value : value, ep.softcap);
         continue;
       }
       if (ep.bias_mode == 1) value += bf2f(ep.bias[col]);
@@ -931,7 +949,16 @@ splitk_finish_kernel(const float *__restrict__ partials, const int splits, const
     float result;
     if (gated) {
       const int first_column = (col / 128) * 256 + col % 128;
-      const float value = sum(first_column);
+      float value = sum(first_column);
+      if (ep.gate_mode >= kGateRelu) {
+        float up = sum(first_column + 128);
+        if (ep.bias_f32 != nullptr) {
+          value += ep.bias_f32[first_column];
+          up += ep.bias_f32[first_column + 128];
+        }
+        ep.out[static_cast<std::size_t>(row) * ep.ld_out + col] = f2bf(gated_value(ep.gate_mode, ep.gate_limit, value, up));
+        continue;
+      }
       const float first = ep.gate_mode == 2 ? bf2f(gelu_round(value)) : rbf(value);
       const float second = rbf(sum(first_column + 128));
       result = rbf(first * second);
@@ -939,7 +966,7 @@ splitk_finish_kernel(const float *__restrict__ partials, const int splits, const
       float *const slot = ep.out_f32 + static_cast<std::size_t>(row) * ep.ld_out + col;
       float value = sum(col);
       if (ep.bias_f32 != nullptr) value += ep.bias_f32[col];
-      *slot = ep.accumulate_f32 != 0 ? *slot + value : value;
+      *slot = soft_cap(ep.accumulate_f32 != 0 ? *slot + value : value, ep.softcap);
       continue;
     } else {
       float value = sum(col);
@@ -1031,7 +1058,7 @@ DeviceState *device_state(int *status) {
 template <bool kFp8, int BN>
 int launch_tc(const void *a, const void *b, const EpilogueParams &ep,
               const std::size_t M, const std::size_t N, const std::size_t K,
-              cudaStream_t stream) {
+              cudaStream_t stream, const std::size_t groups = 1) {
   // the weight is [N, K], or [N, wrap width] when its K coordinate wraps
   const std::size_t weight_k = ep.weight_wrap_blocks > 0 ? static_cast<std::size_t>(ep.weight_wrap_blocks) * 64 : K;
   int status = kOk;
@@ -1040,7 +1067,7 @@ int launch_tc(const void *a, const void *b, const EpilogueParams &ep,
   CUtensorMap map_a, map_b;
   status = make_map(&map_a, a, kFp8, M, K, kBlockM);
   if (status != kOk) return status;
-  status = make_map(&map_b, b, kFp8, N, weight_k, BN);
+  status = make_map(&map_b, b, kFp8, N * groups, weight_k, BN);
   if (status != kOk) return status;
   using L = SharedLayout<BN>;
   static bool configured[64] = {};
@@ -1066,7 +1093,7 @@ int launch_tc(const void *a, const void *b, const EpilogueParams &ep,
 
 template <bool kFp8>
 int launch_tc_pair(const void *a, const void *b, const EpilogueParams &ep, const std::size_t M, const std::size_t N,
-                   const std::size_t K, cudaStream_t stream) {
+                   const std::size_t K, cudaStream_t stream, const std::size_t groups = 1) {
   const std::size_t weight_k = ep.weight_wrap_blocks > 0 ? static_cast<std::size_t>(ep.weight_wrap_blocks) * 64 : K;
   int status = kOk;
   DeviceState *const state = device_state(&status);
@@ -1074,7 +1101,7 @@ int launch_tc_pair(const void *a, const void *b, const EpilogueParams &ep, const
   CUtensorMap map_a, map_b;
   status = make_map(&map_a, a, kFp8, M, K, kBlockM);
   if (status != kOk) return status;
-  status = make_map(&map_b, b, kFp8, N, weight_k, 128);  // a CTA loads its 128 of the tile's 256 weight rows
+  status = make_map(&map_b, b, kFp8, N * groups, weight_k, 128);  // a CTA loads its 128 of the tile's 256 weight rows
   if (status != kOk) return status;
   static bool configured[64] = {};
   int device = 0;
@@ -1180,6 +1207,13 @@ int gemm_error_state(cudaStream_t stream) {
 
 int *device_error_word(int *status) { return tc::error_word(status, nullptr); }
 
+bool grouped_linear_applicable(const LinearArgs &a) {
+  return a.operand_type == OperandType::kBf16 && a.in_features % 8 == 0 && a.in_features >= 64 && a.out_features >= 32 &&
+         (a.gate_mode == 0 || a.out_features % 256 == 0) && a.groups > 0 && a.groups * a.out_features <= 0x7fffffffU &&
+         a.out_features < 0x7fffffffU && (a.tile_rows == 128 || a.tile_rows == 256) && !a.force_simt &&
+         (reinterpret_cast<std::uintptr_t>(a.input) & 15U) == 0 && (reinterpret_cast<std::uintptr_t>(a.weight) & 15U) == 0;
+}
+
 int linear(const LinearArgs &args, cudaStream_t stream) {
   const bool fp8 = args.operand_type == OperandType::kE4m3;
   if (args.input == nullptr || args.weight == nullptr ||
@@ -1196,12 +1230,17 @@ int linear(const LinearArgs &args, cudaStream_t stream) {
       args.in_features > 0x3fffffffU)
     return fail(kInvalidArgument, "linear dimensions are too large");
   if (args.rows == 0) return kOk;
+  if (args.gate_mode >= kGateRelu && (fp8 || args.output_f32 != nullptr))
+    return fail(kInvalidArgument, "the F32 gates take BF16 operands and give BF16 results");
   if (args.output_f32 != nullptr &&
       (fp8 || args.gate_mode != 0 || args.bias_mode != 0 || args.residual != nullptr))
     return fail(kInvalidArgument, "the F32-result mode takes BF16 operands and no BF16 epilogue");
+  if (args.row_group != nullptr)
+    return small_batch_linear_applicable(args) ? small_batch_linear(args, stream)
+                                               : fail(kUnsupported, "grouped rows do not take these sizes");
   // (an F32 result keeps the tile kernel unless the caller gave a split workspace, i.e. wants the weight-stream forms)
   if ((args.output_f32 == nullptr || args.split_workspace != nullptr) && args.weight_wrap_features == 0 &&
-      args.row_scale == nullptr && small_batch_linear_applicable(args))
+      args.row_scale == nullptr && args.tile_group == nullptr && small_batch_linear_applicable(args))
     return small_batch_linear(args, stream);
   const std::size_t out_columns =
       args.gate_mode != 0 ? args.out_features / 2 : args.out_features;
@@ -1214,6 +1253,10 @@ int linear(const LinearArgs &args, cudaStream_t stream) {
   ep.row_scale = args.row_scale;
   ep.bias_mode = args.bias_mode;
   ep.gate_mode = args.gate_mode;
+  ep.gate_limit = args.gate_limit;
+  ep.softcap = args.softcap;
+  ep.tile_group = args.tile_group;
+  ep.tile_count = args.tile_count;
   ep.out_f32 = args.output_f32;
   ep.bias_f32 = args.bias_f32;
   ep.accumulate_f32 = args.accumulate_f32 ? 1 : 0;
@@ -1221,6 +1264,21 @@ int linear(const LinearArgs &args, cudaStream_t stream) {
     if (args.weight_wrap_features % 64 != 0 || args.output_f32 == nullptr)
       return fail(kInvalidArgument, "weight wrap needs whole K blocks and the F32-result mode");
     ep.weight_wrap_blocks = static_cast<int>(args.weight_wrap_features / 64);
+  }
+  if (args.tile_group != nullptr) {
+    if (!grouped_linear_applicable(args) || args.tile_count == nullptr || args.weight_wrap_features != 0)
+      return fail(kUnsupported, "grouped weights do not take these sizes");
+    if (args.tile_rows == 256)
+      return launch_tc_pair<false>(args.input, args.weight, ep, args.rows, args.out_features, args.in_features, stream,
+                                   args.groups);
+    const auto launch = [&](auto bn_tag) {
+      return launch_tc<false, decltype(bn_tag)::value>(args.input, args.weight, ep, args.rows, args.out_features,
+                                                       args.in_features, stream, args.groups);
+    };
+    if (args.gate_mode != 0 || args.out_features >= 256) return launch(std::integral_constant<int, 256>{});
+    if (args.out_features >= 128) return launch(std::integral_constant<int, 128>{});
+    if (args.out_features >= 64) return launch(std::integral_constant<int, 64>{});
+    return launch(std::integral_constant<int, 32>{});
   }
   const std::size_t pitch = args.in_features * (fp8 ? 1 : 2);
   const bool tma_ok =

@@ -9,6 +9,7 @@
 #include <cuda_fp8.h>
 
 #include "common.cuh"
+#include "gates.cuh"
 #include "ops_internal.hpp"
 
 namespace evob {
@@ -29,6 +30,11 @@ struct GemvParams {
   float alpha;
   int bias_mode, gate_mode;
   int dependent_launch;  // launched with programmatic stream serialisation: see the kernel
+  float gate_limit, softcap;
+  // grouped weights [groups, N, K]: blockIdx.y = output row r, x row r / row_fanout, weight of group row_group[r]
+  const int *row_group;
+  int row_fanout;
+  const float *row_scale;  // grouped weights only
 };
 
 template <bool kFp8>
@@ -105,14 +111,21 @@ gemv_kernel(const GemvParams p) {
     for (int r = 0; r < kRows; ++r) acc[c][r] = 0.0F;
   const int chunks = p.K / kPerChunk;
   const std::size_t row_bytes = static_cast<std::size_t>(p.K) * (kFp8 ? 1 : 2);
-  const unsigned char *const wb = static_cast<const unsigned char *>(p.w);
-  const unsigned char *const xb = static_cast<const unsigned char *>(p.x);
+  const unsigned char *wb = static_cast<const unsigned char *>(p.w);
+  const unsigned char *xb = static_cast<const unsigned char *>(p.x);
   // Programmatic dependent launch (one-row steps inside the captured decode graph): this grid may be
   // started while the kernel that produces x is still running.  The weights do not depend on that
   // kernel, so the CTA first asks L2 for its weight rows, lets the grid after it start as well, and only
   // then waits for the producer to finish and its writes to be visible.  Without such a launch the two
   // instructions do nothing.
-  if (p.dependent_launch != 0) {
+  const bool grouped = p.row_group != nullptr;
+  if (grouped) {
+    // which weights these are is a result of the kernel in front
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    wb += static_cast<std::size_t>(p.row_group[blockIdx.y]) * p.N * row_bytes;
+    xb += static_cast<std::size_t>(blockIdx.y / p.row_fanout) * row_bytes;
+  } else if (p.dependent_launch != 0) {
     for (int chunk = threadIdx.x * 8; chunk < chunks; chunk += kThreads * 8) {  // one request per 128-byte line
 #pragma unroll
       for (int c = 0; c < kColumns; ++c)
@@ -158,6 +171,8 @@ gemv_kernel(const GemvParams p) {
   const int r = item / per_cta, local = item % per_cta;
   const int column = column0 + local;
   if (r >= p.rows || column >= out_columns) return;
+  const std::size_t out_index = grouped ? blockIdx.y : r;
+  const float alpha = grouped && p.row_scale != nullptr ? p.alpha * p.row_scale[out_index] : p.alpha;
   const auto total = [&](const int c) {
     float sum = 0.0F;
 #pragma unroll
@@ -165,19 +180,27 @@ gemv_kernel(const GemvParams p) {
     return sum;
   };
   if (p.out_f32 != nullptr) {
-    float *const slot = p.out_f32 + static_cast<std::size_t>(r) * out_columns + column;
-    float value = total(local) * p.alpha;
+    float *const slot = p.out_f32 + out_index * out_columns + column;
+    float value = total(local) * alpha;
     if (p.bias_f32 != nullptr) value += p.bias_f32[column];
-    *slot = p.accumulate_f32 != 0 ? *slot + value : value;
+    *slot = soft_cap(p.accumulate_f32 != 0 ? *slot + value : value, p.softcap);
     return;
   }
-  bf16 *const out_row = p.out + static_cast<std::size_t>(r) * out_columns;
-  if (gated) {
+  bf16 *const out_row = p.out + out_index * out_columns;
+  if (p.gate_mode >= kGateRelu) {
+    float value = total(2 * local) * alpha, up = total(2 * local + 1) * alpha;
+    if (p.bias_f32 != nullptr) {
+      const int row = (column / 128) * 256 + column % 128;
+      value += p.bias_f32[row];
+      up += p.bias_f32[row + 128];
+    }
+    out_row[column] = f2bf(gated_value(p.gate_mode, p.gate_limit, value, up));
+  } else if (gated) {
     const float first = total(2 * local) * p.alpha, second = rbf(total(2 * local + 1) * p.alpha);
     const float activated = p.gate_mode == 2 ? bf2f(gelu_round_small(first)) : rbf(first);
     out_row[column] = f2bf(activated * second);
   } else {
-    float value = total(local) * p.alpha;
+    float value = total(local) * alpha;
     if (p.bias_mode == 1) value += bf2f(p.bias[column]);
     value = rbf(value);
     if (p.bias_mode == 2) value = rbf(value + bf2f(p.bias[column]));
@@ -198,18 +221,21 @@ int launch_gemv(const GemvParams &p, cudaStream_t stream) {
   const int out_columns = p.gate_mode != 0 ? p.N / 2 : p.N;
   const int per_cta = p.gate_mode != 0 ? kColumnsPerCta / 2 : kColumnsPerCta;
   const unsigned int grid = static_cast<unsigned int>((out_columns + per_cta - 1) / per_cta);
-  if (p.rows == 1 && p.dependent_launch != 0) {
+  if (p.row_group != nullptr || (p.rows == 1 && p.dependent_launch != 0)) {
+    const unsigned int rows = p.row_group != nullptr ? static_cast<unsigned int>(p.rows) : 1U;
+    GemvParams q = p;
+    q.rows = 1;
     cudaLaunchAttribute attribute{};
     attribute.id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attribute.val.programmaticStreamSerializationAllowed = 1;
     cudaLaunchConfig_t config{};
-    config.gridDim = dim3(grid);
+    config.gridDim = dim3(grid, rows);
     config.blockDim = dim3(kThreads);
     config.dynamicSmemBytes = 0;
     config.stream = stream;
     config.attrs = &attribute;
-    config.numAttrs = 1;
-    if (cudaLaunchKernelEx(&config, gemv_kernel<kFp8, 1, kColumnsPerCta>, p) != cudaSuccess)
+    config.numAttrs = p.dependent_launch != 0 ? 1 : 0;
+    if (cudaLaunchKernelEx(&config, gemv_kernel<kFp8, 1, kColumnsPerCta>, q) != cudaSuccess)
       return fail(kCuda, "cannot launch the small-batch projection kernel");
   } else if (p.rows == 1)
     gemv_kernel<kFp8, 1, kColumnsPerCta><<<grid, kThreads, 0, stream>>>(p);
@@ -227,7 +253,7 @@ int launch_gemv(const GemvParams &p, cudaStream_t stream) {
 bool small_batch_linear_applicable(const LinearArgs &a) {
   const bool fp8 = a.operand_type == OperandType::kE4m3;
   const std::size_t per_chunk = fp8 ? 16 : 8;
-  return a.rows >= 1 && a.rows <= static_cast<std::size_t>(kMaxRows) && !a.force_simt &&
+  return a.rows >= 1 && a.rows <= (a.row_group != nullptr ? std::size_t{65535} : static_cast<std::size_t>(kMaxRows)) && !a.force_simt &&
          a.in_features % per_chunk == 0 && a.in_features >= per_chunk &&
          (reinterpret_cast<std::uintptr_t>(a.input) & 15U) == 0 &&
          (reinterpret_cast<std::uintptr_t>(a.weight) & 15U) == 0 &&
@@ -251,7 +277,12 @@ int small_batch_linear(const LinearArgs &a, cudaStream_t stream) {
   p.alpha = a.alpha;
   p.bias_mode = a.bias_mode;
   p.gate_mode = a.gate_mode;
-  p.dependent_launch = a.dependent_launch && a.rows == 1 ? 1 : 0;
+  p.dependent_launch = a.dependent_launch && (a.rows == 1 || a.row_group != nullptr) ? 1 : 0;
+  p.gate_limit = a.gate_limit;
+  p.softcap = a.softcap;
+  p.row_group = a.row_group;
+  p.row_fanout = static_cast<int>(a.row_fanout);
+  p.row_scale = a.row_scale;
   return a.operand_type == OperandType::kE4m3 ? launch_gemv<true>(p, stream)
                                               : launch_gemv<false>(p, stream);
 }

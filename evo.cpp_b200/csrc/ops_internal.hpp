@@ -63,6 +63,8 @@ int e4m3_emulated_gemm(const void *input_codes, const void *weight_codes,
 
 // ---- gemm_tcgen05.cu
 enum class OperandType { kBf16, kE4m3 };
+// LinearArgs::gate_mode
+constexpr int kGateProduct = 1, kGateGelu = 2, kGateRelu = 3, kGateClamped = 4;
 struct LinearArgs {
   const void *input = nullptr;   // [rows, in_features] BF16 or E4M3 codes
   const void *weight = nullptr;  // [out_features, in_features], same type
@@ -83,7 +85,11 @@ struct LinearArgs {
   // reads besides `weight` is still being written by work further back than the previous kernel.
   bool dependent_launch = false;
   int bias_mode = 0;   // 0 none, 1 fused F32 add, 2 separate BF16-rounded add
-  int gate_mode = 0;   // 0 none, 1 a*b, 2 gelu(a)*b over 128-column halves
+  // over 128-column halves (row-interleaved weights): 0 none, 1 a*b, 2 gelu(a)*b, 3 max(a, 0)*b, 4 clamped SwiGLU
+  // with gate_limit (gates.cuh).  3 and 4 work on the F32 accumulators (plus bias_f32 in the weight's row order)
+  // and round once.
+  int gate_mode = 0;
+  float gate_limit = 0.0F;
   bool force_simt = false;
   // F32-result mode (BF16 operands, tensor-core path only): the F32 accumulator
   // times alpha, plus bias_f32, is stored (or added) to output_f32 [rows,
@@ -101,8 +107,20 @@ struct LinearArgs {
   float *output_f32 = nullptr;
   const float *bias_f32 = nullptr;
   bool accumulate_f32 = false;
+  float softcap = 0.0F;  // F32 results: softcap tanh(value / softcap) last (0: none)
   std::size_t weight_wrap_features = 0;
+  // Grouped weights [groups, out_features, in_features] (BF16).  Tile form: rows come in whole tiles of tile_rows
+  // (128 or 256), tile t belongs to group tile_group[t], *tile_count tiles are in use (both on the device; `rows`
+  // is the capacity, unused tiles are not touched).  Row form (a few rows): output row r is input row
+  // r / row_fanout times the weight of group row_group[r].
+  std::size_t groups = 0;
+  const int *tile_group = nullptr, *tile_count = nullptr;
+  std::size_t tile_rows = 128;
+  const int *row_group = nullptr;
+  std::size_t row_fanout = 1;
 };
+// Whether linear() takes the tile form of grouped weights at these sizes.
+bool grouped_linear_applicable(const LinearArgs &args);
 int linear(const LinearArgs &args, cudaStream_t stream);
 // gemv.cu: weight-streaming kernel that linear() uses for 1..8 rows.
 bool small_batch_linear_applicable(const LinearArgs &args);

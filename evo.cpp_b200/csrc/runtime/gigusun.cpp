@@ -12,8 +12,7 @@
 #include <cmath>
 
 #include "../decoder_ops.hpp"
-#include "json.hpp"
-#include "weights.hpp"
+#include "decoder_config.hpp"
 
 namespace evob {
 namespace {
@@ -23,27 +22,6 @@ namespace {
     const int status__ = (expr);    \
     if (status__ != kOk) return status__; \
   } while (0)
-
-int size_member(const Json &object, const char *key, const std::string &where, const std::size_t minimum,
-                std::size_t *out) {
-  const Json *value = object.get(key);
-  if (value == nullptr || value->kind != Json::kNumber || !(value->number >= static_cast<double>(minimum)) ||
-      value->number > 2147483647.0 || value->number != std::floor(value->number))
-    return fail(kModelFormat, "config.json: " + where + "." + key + " must be an integer of at least " +
-                                  std::to_string(minimum));
-  *out = static_cast<std::size_t>(value->number);
-  return kOk;
-}
-
-int real_member(const Json &object, const char *key, const std::string &where, const bool positive, float *out) {
-  const Json *value = object.get(key);
-  if (value == nullptr || value->kind != Json::kNumber || !std::isfinite(value->number) ||
-      (positive && !(value->number > 0.0)))
-    return fail(kModelFormat, "config.json: " + where + "." + key + " must be a " +
-                                  (positive ? "positive " : "") + "number");
-  *out = static_cast<float>(value->number);
-  return kOk;
-}
 
 int read_block(const ModelFile &file, const Json &entry, const std::size_t index, DecoderBlock *block) {
   const std::string where = "layers[" + std::to_string(index) + "]";
@@ -90,6 +68,7 @@ int read_block(const ModelFile &file, const Json &entry, const std::size_t index
     const Json *kind = mlp->get("kind");
     if (mlp->kind != Json::kObject || kind == nullptr || kind->kind != Json::kString || kind->text != "dense")
       return fail(kUnsupported, "config.json: " + where + ".mlp is not a dense feed-forward");
+    b.feed_forward = FeedForward::kPolyNorm;
     EVOB_TRY(size_member(*mlp, "ff", where + ".mlp", 1, &b.inner_width));
   }
   *block = b;
@@ -101,13 +80,13 @@ std::vector<float> one_plus(std::vector<float> values) {
   return values;
 }
 
-}  // namespace
-
 int read_gigusun_config(const ModelFile &file, ModelConfig *config) {
   const Json *const root = file.configuration();
   if (root == nullptr) return fail(kModelFormat, "the model directory has no config.json");
   ModelConfig c;
   c.graph = BlockGraph::kDecoder;
+  c.design = &kGigusunDesign;
+  c.learned_positions = true;
   c.architecture = "Gigusun";
   c.artifact_profile = "decoder-config-v1";
   EVOB_TRY(size_member(*root, "vocab", "model", 1, &c.vocab));
@@ -285,5 +264,10 @@ int upload_gigusun_block(const ModelFile &file, const ModelConfig &c, const std:
   }
   return kOk;
 }
+
+}  // namespace
+
+const DecoderDesign kGigusunDesign = {"Gigusun",          read_gigusun_config,  gigusun_model_tensors, gigusun_block_tensors,
+                                      upload_gigusun_model, upload_gigusun_block};
 
 }  // namespace evob

@@ -456,7 +456,8 @@ const char *profile_category_name(const int category) {
   static const char *const names[kProfileCategories] = {
       "rms_norm", "gemm_bf16_tcgen05", "gemm_e4m3_tcgen05", "gemm_e4m3_emulated", "hcs_fused_fir",
       "hcm_fused_fir", "hcl_modal_scan", "attention", "state_step", "elementwise", "row_quantize",
-      "gemm_e4m3_ffn_tcgen05", "gated_linear_attention", "gated_delta_rule", "poly_norm"};
+      "gemm_e4m3_ffn_tcgen05", "gated_linear_attention", "gated_delta_rule", "poly_norm",
+      "gemm_grouped", "routing"};
   return category >= 0 && category < kProfileCategories ? names[category] : "";
 }
 

@@ -18,13 +18,17 @@
 
 namespace evob {
 
-// The last three are mixers of decoder blocks (BlockGraph::kDecoder).
-enum class MixerType { kHcs, kHcm, kHcl, kAttention, kWindowAttention, kGatedLinear, kGatedDelta };
+// The last four are mixers of decoder blocks (BlockGraph::kDecoder).
+enum class MixerType { kHcs, kHcm, kHcl, kAttention, kWindowAttention, kGatedLinear, kGatedDelta, kLatentAttention };
 
 // Which block graph a model runs through: StripedHyena2 (BF16 residual, RoPE / Hyena mixers, gated MLP,
 // tied head) or the decoder graph (F32 residual, a mixer and an optional feed-forward per block, each
-// with its own sizes, learned positions, own head).
+// with its own sizes, own head).
 enum class BlockGraph { kStripedHyena2, kDecoder };
+
+// Feed-forwards of decoder blocks: W_down poly(W_up h); W_down (relu(W_gate h + b) * (W_up h + b)) + b; a mixture
+// of experts with clamped gates.
+enum class FeedForward { kNone, kPolyNorm, kReluGated, kExperts };
 
 // Operator classes reported by the optional per-operator timing.
 enum ProfileCategory : int {
@@ -43,6 +47,8 @@ enum ProfileCategory : int {
   kCatGatedLinear,     // gated linear attention: preparation, recurrence, output norm and gate
   kCatGatedDelta,      // gated delta rule: the same, with the short convolutions
   kCatPolyNorm,        // normalised polynomial activation of a decoder's feed-forward
+  kCatGemmGrouped,     // projections of a mixture of experts
+  kCatRouting,         // router choice and regrouping of rows by expert
   kProfileCategories
 };
 const char *profile_category_name(int category);
@@ -97,9 +103,24 @@ struct DecoderBlock {
   std::size_t conv_taps = 0;             // kGatedDelta
   std::size_t decay_rank = 0;            // kGatedLinear: width of the bottleneck in front of the decays
   float tau = 1.0F;                      // kGatedLinear
-  std::size_t inner_width = 0;           // feed-forward, 0: none
+  // kLatentAttention: widths of the query latent and of the cached key/value latent; a learned score per head in
+  // the softmax's denominator
+  std::size_t query_rank = 0, latent_rank = 0;
+  bool sink = false;
+  FeedForward feed_forward = FeedForward::kNone;
+  std::size_t inner_width = 0;           // of the feed-forward, or of one expert
+  std::size_t experts = 0, top = 0;      // kExperts
+  float gate_limit = 0.0F;
+  // gated feed-forwards keep their inner columns in whole blocks of 128 (zero weights behind the last)
+  std::size_t inner_columns() const {
+    return feed_forward == FeedForward::kPolyNorm ? inner_width : (inner_width + 127) / 128 * 128;
+  }
+  // weight rows of the router: zeros up to a whole tile of the projection kernels
+  std::size_t router_rows() const { return (experts + 63) / 64 * 64; }
 
-  // Columns of the fused input projection [queries | keys | values | output gate | beta or decay
+  // Latent attention: the fused input projection is [query latent | key/value latent].
+  std::size_t latent_column() const { return padded(query_rank); }
+  // Columns of the other mixers' fused input projection [queries | keys | values | output gate | beta or decay
   // bottleneck | decay]; every segment starts at a multiple of eight columns (zero weight rows between).
   std::size_t query_width() const { return mixer == MixerType::kGatedDelta ? kv_heads * dim : heads * dim; }
   std::size_t key_width() const { return kv_heads * dim; }
@@ -117,10 +138,13 @@ struct DecoderBlock {
   }
   std::size_t decay_column() const { return beta_column() + padded(beta_width()); }
   std::size_t projection_width() const {
+    if (mixer == MixerType::kLatentAttention) return latent_column() + padded(latent_rank);
     return decay_column() + (mixer == MixerType::kGatedDelta ? padded(heads) : 0);
   }
   std::size_t output_width() const { return heads * value_dim; }
 };
+
+struct DecoderDesign;  // decoder_config.hpp
 
 struct ModelConfig {
   std::string architecture, model_id, model_name, artifact_profile;
@@ -133,6 +157,13 @@ struct ModelConfig {
   std::vector<MixerType> mixers;  // one per block
   BlockGraph graph = BlockGraph::kStripedHyena2;
   std::vector<DecoderBlock> blocks;  // decoder graphs: one per block
+  const DecoderDesign *design = nullptr;  // decoder graphs
+  // decoder graphs: RMS norms in front of the sublayers, or (output_norms) sublayers that read the stream itself
+  // and layer norms on what they add to it; the final norm is of the same kind
+  bool output_norms = false;
+  bool learned_positions = false;
+  // logits = softcap tanh(scale head(x) / softcap), softcap 0: none
+  float logit_scale = 1.0F, logit_softcap = 0.0F;
   bool decoder() const { return graph == BlockGraph::kDecoder; }
   // bytes of one residual element
   std::size_t hidden_bytes() const { return decoder() ? sizeof(float) : 2; }
@@ -141,8 +172,6 @@ struct ModelConfig {
 
 // Picks the design by the architecture that the file names (config.json, else the typed metadata).
 int read_model_config(const ModelFile &file, bool allow_test_fixture, ModelConfig *config);
-// gigusun.cpp: the reader of a Gigusun config.json (sizes of the decay bottlenecks come from the tensors).
-int read_gigusun_config(const ModelFile &file, ModelConfig *config);
 // Every tensor the configuration calls for is there with its type and shape, and nothing else is
 // (host only; load_weights makes the same checks while it gathers the views).
 int check_tensor_set(const ModelFile &file, const ModelConfig &config);
@@ -161,9 +190,15 @@ struct LayerWeights {
   const void *l1 = nullptr, *l2 = nullptr, *l3 = nullptr;
   const void *l12 = nullptr;  // row-interleaved [2I, D] for the fused gate GEMM
   std::size_t payload_bytes = 0;
-  // ---- decoder blocks.  pre_norm / post_norm hold the whole gain (one plus the stored weight),
-  // projection the fused input projection (DecoderBlock), l1 / l3 the feed-forward's up and down weights.
-  const float *query_norm = nullptr, *key_norm = nullptr;  // [dim]
+  // ---- decoder blocks.  pre_norm / post_norm hold the whole gain of the norms in front of (output_norms: behind)
+  // the mixer and the feed-forward, projection the fused input projection (DecoderBlock), l1 / l3 the
+  // feed-forward's up and down weights, l12 the row-interleaved gate and up weights (of all experts: [experts,
+  // 2 inner_columns, width], then l3 is [experts, width, inner_columns]).
+  const float *query_norm = nullptr, *key_norm = nullptr;  // [dim]; latent attention: [query_rank], [latent_rank]
+  const void *query_up = nullptr, *key_up = nullptr, *value_up = nullptr;  // latent attention: [heads * dim, rank]
+  const float *sink_logit = nullptr;                       // [heads]
+  const void *router = nullptr;                            // [router_rows, width]
+  const float *l12_bias = nullptr, *l3_bias = nullptr;     // [2 inner_columns] in l12's row order, [width]
   const float *distance_bias = nullptr;                    // [heads, max_seqlen]
   const float *conv = nullptr;                             // [gate_column, conv_taps], by projection column
   const float *decay_rate = nullptr, *decay_shift = nullptr;  // delta: -exp(A_log), dt_bias [heads]
@@ -311,8 +346,13 @@ class Context {
   int run_decoder_stage(Stage &stage, std::size_t rows, Mode mode, std::size_t position, long capture_layer,
                         std::vector<float> *captured, const DumpPlan *dumps);
   int decoder_head(Stage &stage, std::size_t rows);
-  int decoder_linear(Stage &stage, const void *input, const void *weight, std::size_t rows, std::size_t in_features,
-                     std::size_t out_features, void *output, float *output_f32, bool accumulate);
+  int decoder_linear(Stage &stage, const struct DecoderProduct &product);
+  int latent_mixer(Stage &stage, std::size_t local_layer, std::size_t rows, std::size_t position, const int *dynamic);
+  // Feed-forwards with gates; what they leave for the norm behind them is described by *norm.
+  int gated_feed_forward(Stage &stage, std::size_t local_layer, std::size_t rows, const void *input,
+                         struct LayerNormArgs *norm);
+  int expert_feed_forward(Stage &stage, std::size_t local_layer, std::size_t rows, const void *input,
+                          struct LayerNormArgs *norm);
   // Taps of block `layer` of `stage` (dumps.cu-style helpers in model.cu).
   int dump_mixer_taps(Stage &stage, std::size_t local_layer, std::size_t rows, Mode mode,
                       const DumpPlan &dumps);

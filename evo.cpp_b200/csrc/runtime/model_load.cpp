@@ -14,6 +14,7 @@
 
 #include "../common.cuh"
 #include "../ops_internal.hpp"
+#include "decoder_config.hpp"
 #include "json.hpp"
 #include "model.hpp"
 
@@ -48,15 +49,9 @@ namespace {
 
 int read_striped_hyena_config(const ModelFile &file, bool allow_test_fixture, ModelConfig *config);
 
-// Designs that a config.json describes, by the architecture it names.  (StripedHyena2 artifacts carry
-// typed metadata inside the Safetensors file instead.)
-struct ConfiguredDesign {
-  const char *architecture;
-  int (*read)(const ModelFile &file, ModelConfig *config);
-};
-const ConfiguredDesign kConfiguredDesigns[] = {
-    {"Gigusun", read_gigusun_config},
-};
+// Designs that a config.json describes.  (StripedHyena2 artifacts carry typed metadata inside the Safetensors
+// file instead.)
+const DecoderDesign *const kConfiguredDesigns[] = {&kGigusunDesign, &kKikepelDesign};
 
 }  // namespace
 
@@ -65,8 +60,8 @@ int read_model_config(const ModelFile &file, const bool allow_test_fixture, Mode
   if (const Json *root = file.configuration()) {
     const Json *architecture = root->get("architecture");
     if (architecture != nullptr && architecture->kind == Json::kString) {
-      for (const ConfiguredDesign &design : kConfiguredDesigns)
-        if (architecture->text == design.architecture) return design.read(file, config);
+      for (const DecoderDesign *design : kConfiguredDesigns)
+        if (architecture->text == design->architecture) return design->read(file, config);
       if (file.metadata("evo2.profile") == nullptr)
         return fail(kUnsupported, "config.json names an unknown architecture: " + architecture->text);
     }

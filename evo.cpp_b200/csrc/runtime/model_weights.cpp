@@ -14,6 +14,7 @@
 
 #include "../common.cuh"
 #include "../ops_internal.hpp"
+#include "decoder_config.hpp"
 #include "model.hpp"
 #include "weights.hpp"
 
@@ -21,7 +22,7 @@ namespace evob {
 namespace {
 
 std::vector<ExpectedTensor> expected_block_tensors(const ModelConfig &c, const std::size_t layer) {
-  if (c.decoder()) return gigusun_block_tensors(c, layer);
+  if (c.decoder()) return c.design->block_tensors(c, layer);
   const std::string p = "blocks." + std::to_string(layer) + ".";
   const std::size_t D = c.width, I = c.inner_width;
   std::vector<ExpectedTensor> list;
@@ -67,14 +68,14 @@ bool gate_fusable(const ModelConfig &c) {
 
 // Tensors outside the blocks.
 std::vector<ExpectedTensor> expected_model_tensors(const ModelConfig &c) {
-  if (c.decoder()) return gigusun_model_tensors(c);
+  if (c.decoder()) return c.design->model_tensors(c);
   return {{"embedding_layer.weight", TensorType::kBF16, {c.vocab, c.width}},
           {"unembed.weight", TensorType::kBF16, {c.vocab, c.width}},
           {"norm.scale", TensorType::kF32, {c.width}}};
 }
 
 int upload_model_tensors(const ModelFile &file, const ModelConfig &c, WeightUploader *up, StageWeights *stage) {
-  if (c.decoder()) return upload_gigusun_model(file, c, up, stage);
+  if (c.decoder()) return c.design->upload_model(file, c, up, stage);
   const void *p = nullptr;
   int status = up->tensor(*file.find("embedding_layer.weight"), &stage->embedding);
   if (status == kOk) status = up->tensor(*file.find("norm.scale"), &p);
@@ -85,7 +86,7 @@ int upload_model_tensors(const ModelFile &file, const ModelConfig &c, WeightUplo
 
 int upload_layer(const ModelFile &file, const ModelConfig &c, const std::size_t layer,
                  WeightUploader *up, LayerWeights *w, std::vector<unsigned char> *host_scratch) {
-  if (c.decoder()) return upload_gigusun_block(file, c, layer, up, w);
+  if (c.decoder()) return c.design->upload_block(file, c, layer, up, w);
   const std::vector<ExpectedTensor> expected = expected_block_tensors(c, layer);
   std::vector<const TensorView *> t(expected.size());
   for (std::size_t i = 0; i < expected.size(); ++i) {

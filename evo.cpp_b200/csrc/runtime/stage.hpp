@@ -52,7 +52,8 @@ struct LayerState {
   float *short_cache = nullptr;  // [3D, short_taps-1]
   float *inner_cache = nullptr;  // [D, taps-1]
   float *modal_state = nullptr;  // [D, S]
-  // [context, D] BF16; decoders: [context, kv_heads, dim] and [context, kv_heads, value_dim], type of the activations
+  // [context, D] BF16; decoders: [context, kv_heads, dim] and [context, kv_heads, value_dim], type of the activations;
+  // latent attention: [context, latent_rank], keys and values in one
   void *key_cache = nullptr, *value_cache = nullptr;
   // decoders: the last conv_taps - 1 projection rows, oldest first, and the matrix state of a recurrent mixer
   void *conv_history = nullptr;       // [conv_taps - 1, channels], type of the activations
@@ -93,6 +94,20 @@ struct Context::Stage {
   void *mlp_first = nullptr, *mlp_second = nullptr;
   void *short_filtered = nullptr, *x2 = nullptr, *x1 = nullptr, *value = nullptr, *pregate = nullptr;
   float *modal_scratch = nullptr;
+  // decoders with norms on the sublayers' outputs: what a sublayer adds, F32 [T, width]
+  void *sublayer = nullptr;
+  // latent attention: normed query latents [T, query_rank]; of up to kLatentRows rows the queries against latents and
+  // the mixed latents [rows, heads, latent_rank]; expanded keys and values of the tokens that a pass sees
+  void *query_latent = nullptr, *absorbed = nullptr, *latent_mix = nullptr;
+  void *expanded_keys = nullptr, *expanded_values = nullptr;
+  // gated feed-forwards whose gate is not applied by the projection: F32 [rows, 2 inner_columns]
+  void *gate_products = nullptr;
+  // mixtures of experts: rows in the experts' tiles and their results, the router's scores, per (row, place) the
+  // expert, its score, the place among the expert's rows and the row's slot; the table of tiles
+  void *grouped_rows = nullptr, *expert_out = nullptr;
+  float *router_logits = nullptr, *pair_score = nullptr, *slot_score = nullptr;
+  int *pair_expert = nullptr, *pair_rank = nullptr, *pair_slot = nullptr;
+  int *expert_counts = nullptr, *tile_group = nullptr, *tile_count = nullptr;
   void *recurrent_workspace = nullptr;  // decoders: recurrent_workspace_bytes of the largest recurrent block
   void *split_workspace = nullptr;  // F32 partial sums of split-K projections (<= 128 rows)
   // fast-q8-kv: BF16 images [context, D] of the keys and values one attention block at a time

@@ -65,6 +65,20 @@ struct WeightUploader {
       return fail(kCuda, "weight upload failed");
     return kOk;
   }
+  // `rows` rows of row_bytes, source_pitch apart, to rows `pitch` apart.
+  int copy_rows(void *dst, const std::size_t pitch, const void *src, const std::size_t source_pitch,
+                const std::size_t row_bytes, const std::size_t rows) {
+    if (dry_run || rows == 0 || row_bytes == 0) return kOk;
+    if (cudaMemcpy2DAsync(dst, pitch, src, source_pitch, row_bytes, rows, cudaMemcpyHostToDevice, stream) != cudaSuccess)
+      return fail(kCuda, "weight upload failed");
+    return kOk;
+  }
+  // A piece of the slab filled with zeros.
+  int zeros(const std::size_t bytes, unsigned char **out) {
+    *out = static_cast<unsigned char *>(place(bytes));
+    if (!dry_run && cudaMemsetAsync(*out, 0, bytes, stream) != cudaSuccess) return fail(kCuda, "weight upload failed");
+    return kOk;
+  }
   int tensor(const TensorView &t, const void **out) {
     void *dst = place(t.bytes);
     *out = dst;
@@ -79,12 +93,5 @@ struct WeightUploader {
     return copy(dst, staged.back().data(), bytes);
   }
 };
-
-// gigusun.cpp
-std::vector<ExpectedTensor> gigusun_model_tensors(const ModelConfig &config);
-std::vector<ExpectedTensor> gigusun_block_tensors(const ModelConfig &config, std::size_t layer);
-int upload_gigusun_model(const ModelFile &file, const ModelConfig &config, WeightUploader *up, StageWeights *stage);
-int upload_gigusun_block(const ModelFile &file, const ModelConfig &config, std::size_t layer, WeightUploader *up,
-                         LayerWeights *weights);
 
 }  // namespace evob

@@ -73,7 +73,7 @@ EVO_API size_t evo_b200_context_activation_capacity(const evo_context *context);
  * with the configuration, an unsupported projection dtype and tensors outside the profile's exact set
  * are rejected here, before any device work).  mixer_types (optional) receives one code per block -
  * 0 HCS, 1 HCM, 2 HCL, 3 attention; decoder blocks 4 window attention, 5 gated linear attention,
- * 6 gated delta rule - up to mixer_capacity.  Models described by a config.json (a directory path) report
+ * 6 gated delta rule, 7 latent attention - up to mixer_capacity.  Models described by a config.json (a directory path) report
  * the largest head count, state size and inner width of their blocks.  The three names are NUL-terminated and cut
  * at 63 bytes. */
 typedef struct evo_b200_model_config {

@@ -230,7 +230,12 @@ def test_attention_refusals(pkg, ops):
     with pytest.raises(pkg.OpsError) as error:
         window_case(pkg, ops, rows=40, position=0, heads=2, kv_heads=1, dim=40, vdim=64, window=8, keep_first=0, kernel=TENSOR)
     assert error.value.code == 5
-    for bad in (dict(heads=3, kv_heads=2), dict(dim=300), dict(softcap=-1.0)):
+    for size in ("dim", "vdim"):                                     # wide heads run in the row kernel only
+        with pytest.raises(pkg.OpsError) as error:
+            window_case(pkg, ops, **(dict(rows=2, position=0, heads=2, kv_heads=1, dim=16, vdim=16, window=8, keep_first=0,
+                                          kernel=TILE) | {size: 300}))
+        assert error.value.code == 5
+    for bad in (dict(heads=3, kv_heads=2), dict(dim=1032), dict(softcap=-1.0)):
         case = dict(rows=2, position=0, heads=2, kv_heads=1, dim=16, vdim=16, window=8, keep_first=0, kernel=0) | bad
         with pytest.raises(pkg.OpsError) as error:
             window_case(pkg, ops, **case)
