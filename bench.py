@@ -874,9 +874,10 @@ def main() -> None:
                         help="do not also time the opt-in b200-fp8 profile")
     parser.add_argument("--decode-tokens", type=int, default=64,
                         help="cached-decode steps timed after a 1,024-token prompt (0 disables)")
-    parser.add_argument("--design", default=None, choices=["gigusun"],
-                        help="instead of the headline workload: a decoder of this design beside a StripedHyena2 stack "
-                             "of equal width, block count and weights (prefill, decode, operator classes)")
+    parser.add_argument("--design", default=None, choices=["gigusun", "kikepel"],
+                        help="instead of the headline workload: a decoder of this design beside the closest other model "
+                             "(gigusun: a StripedHyena2 stack, kikepel: a Gigusun stack of window attention) of equal "
+                             "width, block count and weights (prefill, decode, operator classes)")
     parser.add_argument("--design-widths", default="2048,4096", help="model widths of --design")
     args = parser.parse_args()
     select_model(args.model)
@@ -890,7 +891,7 @@ def main() -> None:
         package = load_package()
         bench = importlib.import_module("evo_cpp_b200.decoder_bench")
         print(json.dumps(bench.run(package, ClockSampler, args.steps, max(args.warmup, 3), [1024, 8192],
-                                   [int(w) for w in args.design_widths.split(",")], args.decode_tokens)))
+                                   [int(w) for w in args.design_widths.split(",")], args.decode_tokens, args.design)))
     elif args.impl == "reference":
         run_reference(args, rank, world)
     elif world > 1 and args.multi_gpu == "pipeline":

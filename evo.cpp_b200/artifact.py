@@ -351,17 +351,74 @@ def gigusun_values(name: str, shape: tuple[int, ...], rng: np.random.Generator) 
     return rng.normal(0.0, 1.0 / math.sqrt(shape[-1]), shape)
 
 
-def gigusun_weights(config: dict, seed: int, decay_rank: int = 16) -> dict[str, np.ndarray]:
+# ---- Kikepel decoders
+def kikepel_config(layers: list[dict], *, vocab: int, width: int, logit_scale: float = 1.0, logit_softcap: float = 30.0,
+                   eps: float = 1e-6) -> dict:
+    return {"architecture": "Kikepel", "vocab": vocab, "width": width, "logit_scale": logit_scale,
+            "logit_softcap": logit_softcap, "norm": {"eps": eps}, "layers": layers}
+
+
+def kikepel_manifest(config: dict) -> list[tuple[str, tuple[int, ...]]]:
+    """(tensor name, shape) of a configuration, in file order."""
+    D = config["width"]
+    rows = [("embed", (config["vocab"], D))]
+    for i, layer in enumerate(config["layers"]):
+        m, p, f, mlp = layer["mixer"], f"l{i}.mix.", f"l{i}.mlp.", layer["mlp"]
+        H, q, c = m["heads"], m["q_rank"], m["kv_rank"]
+        rows += [(f"l{i}.norm1", (D,)), (p + "dq", (q, D)), (p + "dq.norm", (q,)), (p + "uq", (H * m["dim"], q)),
+                 (p + "dkv", (c, D)), (p + "dkv.norm", (c,)), (p + "uk", (H * m["dim"], c)), (p + "uv", (H * m["vdim"], c)),
+                 (p + "o", (D, H * m["vdim"]))]
+        if layer["type"] == "latent_attention":
+            rows.append((p + "sink", (H,)))
+        if mlp is None:
+            continue
+        rows.append((f"l{i}.norm2", (D,)))
+        if mlp["kind"] == "dense":
+            ff = mlp["ff"]
+            rows += [(f + "gate", (ff, D)), (f + "gate.b", (ff,)), (f + "up", (ff, D)), (f + "up.b", (ff,)),
+                     (f + "down", (D, ff)), (f + "down.b", (D,))]
+            continue
+        ff = mlp["expert"]["ff"]
+        rows.append((f + "router", (mlp["router"]["experts"], D)))
+        for e in range(mlp["router"]["experts"]):
+            rows += [(f"{f}e{e}.gate", (ff, D)), (f"{f}e{e}.up", (ff, D)), (f"{f}e{e}.down", (D, ff))]
+    return rows + [("final.norm", (D,)), ("head", (config["vocab"], D))]
+
+
+def kikepel_values(name: str, shape: tuple[int, ...], rng: np.random.Generator) -> np.ndarray:
+    """Random F32 values of one tensor on a scale that keeps every mechanism alive."""
+    if "norm" in name.rsplit(".", 1)[-1]:
+        return rng.uniform(0.6, 1.5, shape)
+    if name.endswith(".sink"):
+        return rng.uniform(-1.0, 3.0, shape)
+    if name.endswith(".b"):
+        return rng.normal(0.0, 0.5, shape)
+    if name == "embed":
+        return rng.normal(0.0, 1.0, shape)
+    return rng.normal(0.0, 1.0 / math.sqrt(shape[-1]), shape)
+
+
+# ---- either design: a directory with config.json and model.safetensors
+def decoder_manifest(config: dict, decay_rank: int = 16) -> list[tuple[str, tuple[int, ...]]]:
+    return kikepel_manifest(config) if config["architecture"] == "Kikepel" else gigusun_manifest(config, decay_rank)
+
+
+def decoder_values(config: dict):
+    """values(name, shape, rng) of the design."""
+    return kikepel_values if config["architecture"] == "Kikepel" else gigusun_values
+
+
+def decoder_weights(config: dict, seed: int, decay_rank: int = 16) -> dict[str, np.ndarray]:
     """{name: F32 values that BF16 holds exactly}."""
     rng = np.random.default_rng(seed)
-    weights = {}
-    for name, shape in gigusun_manifest(config, decay_rank):
-        bits = np.frombuffer(_bf16_bytes(gigusun_values(name, shape, rng)), np.uint16).astype(np.uint32) << 16
+    weights, values = {}, decoder_values(config)
+    for name, shape in decoder_manifest(config, decay_rank):
+        bits = np.frombuffer(_bf16_bytes(values(name, shape, rng)), np.uint16).astype(np.uint32) << 16
         weights[name] = bits.view(np.float32).reshape(shape)
     return weights
 
 
-def write_gigusun(directory: Path, config: dict, weights: dict[str, np.ndarray]) -> Path:
+def write_decoder(directory: Path, config: dict, weights: dict[str, np.ndarray]) -> Path:
     """Writes config.json and model.safetensors; returns the directory (what a loader is pointed at)."""
     directory = Path(directory)
     directory.mkdir(parents=True, exist_ok=True)
@@ -371,8 +428,8 @@ def write_gigusun(directory: Path, config: dict, weights: dict[str, np.ndarray])
     return directory
 
 
-def write_gigusun_random(directory: Path, config: dict, seed: int, device: str, decay_rank: int = 16) -> Path:
-    """As write_gigusun with seeded weights; the large matrices are drawn by torch on `device`."""
+def write_decoder_random(directory: Path, config: dict, seed: int, device: str, decay_rank: int = 16) -> Path:
+    """As write_decoder with seeded weights; the large matrices are drawn by torch on `device`."""
     import torch
 
     directory = Path(directory)
@@ -381,15 +438,16 @@ def write_gigusun_random(directory: Path, config: dict, seed: int, device: str, 
     rng = np.random.default_rng(seed)
     generator = torch.Generator(device=device)
     generator.manual_seed(seed)
+    values = decoder_values(config)
 
     def tensors():
-        for name, shape in gigusun_manifest(config, decay_rank):
+        for name, shape in decoder_manifest(config, decay_rank):
             if len(shape) == 2 and math.prod(shape) >= 1 << 16:
                 std = 1.0 if name == "embed" else 0.5 if name == "pos" else 1.0 / math.sqrt(shape[-1])
                 drawn = (torch.randn(math.prod(shape), generator=generator, device=device) * std).bfloat16()
                 payload = drawn.view(torch.int16).cpu().numpy().tobytes()
             else:
-                payload = _bf16_bytes(gigusun_values(name, shape, rng))
+                payload = _bf16_bytes(values(name, shape, rng))
             yield name, "BF16", list(shape), payload
 
     write_model(directory / "model.safetensors", {}, tensors(), max_shard_bytes=1 << 40)

@@ -175,6 +175,12 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
         __syncwarp();
         const int at = n0 + c * 32 + (lane % 8) * 4;
         if (c + 1 < chunks) fetch_old(c + 1);
+        if (ep.softcap > 0.0F) {  // (capped results carry no bias)
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            sums[i] = make_float4(fast_soft_cap(sums[i].x, ep.softcap), fast_soft_cap(sums[i].y, ep.softcap),
+                                  fast_soft_cap(sums[i].z, ep.softcap), fast_soft_cap(sums[i].w, ep.softcap));
+        }
         if (at < n_limit) {
           float4 shift = make_float4(0.0F, 0.0F, 0.0F, 0.0F);
           if (ep.bias_f32 != nullptr)
@@ -182,13 +188,9 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const int r = m0 + quarter * 32 + 4 * i + lane / 8;
-            if (r >= M) continue;
-            float4 result =
-                make_float4(sums[i].x + shift.x, sums[i].y + shift.y, sums[i].z + shift.z, sums[i].w + shift.w);
-            if (ep.softcap > 0.0F)
-              result = make_float4(soft_cap(result.x, ep.softcap), soft_cap(result.y, ep.softcap),
-                                   soft_cap(result.z, ep.softcap), soft_cap(result.w, ep.softcap));
-            *reinterpret_cast<float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at) = result;
+            if (r < M)
+              *reinterpret_cast<float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at) =
+                  make_float4(sums[i].x + shift.x, sums[i].y + shift.y, sums[i].z + shift.z, sums[i].w + shift.w);
           }
         }
         continue;
@@ -201,7 +203,7 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
             float value = __uint_as_float(v[j]) * scale;
             if (ep.bias_f32 != nullptr) value += ep.bias_f32[col + j];
             if (ep.accumulate_f32 != 0) value += out_row[col + j];
-            out_row[col + j] = soft_cap(value, ep.softcap);
+            out_row[col + j] = fast_soft_cap(value, ep.softcap);
           }
         }
       }
@@ -210,18 +212,27 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
     if (row < M && col < n_limit) {
       bf16 *const out_row = ep.out + static_cast<std::size_t>(row) * ep.ld_out;
       float r[32];
+      // (the weight rows of output column j of this chunk: n0 + c * 32 + j, and 128 further on)
+      if (ep.gate_mode == kGateRelu) {
+        const float *const bias = ep.bias_f32 != nullptr ? ep.bias_f32 + n0 + c * 32 : nullptr;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          float value = __uint_as_float(v[j]) * scale, up = __uint_as_float(w[j]) * scale;
+          if (bias != nullptr) {
+            value += __ldg(bias + j);
+            up += __ldg(bias + BN / 2 + j);
+          }
+          r[j] = relu_gate(value, up);
+        }
+      } else if (ep.gate_mode == kGateClamped) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+          r[j] = clamped_gate<true>(ep.gate_limit, __uint_as_float(v[j]) * scale, __uint_as_float(w[j]) * scale);
+      } else
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
         float value = __uint_as_float(v[j]) * scale;
-        if (ep.gate_mode >= kGateRelu) {
-          // (the weight rows of this output column: n0 + c * 32 + j, and 128 further on)
-          float up = __uint_as_float(w[j]) * scale;
-          if (ep.bias_f32 != nullptr) {
-            value += __ldg(ep.bias_f32 + n0 + c * 32 + j);
-            up += __ldg(ep.bias_f32 + n0 + BN / 2 + c * 32 + j);
-          }
-          r[j] = gated_value(ep.gate_mode, ep.gate_limit, value, up);
-        } else if (gated) {
+        if (gated) {
           const float first =
               ep.gate_mode == 2 ? bf2f(gelu_round(value)) : rbf(value);
           const float second = rbf(__uint_as_float(w[j]) * scale);
@@ -1232,6 +1243,8 @@ int linear(const LinearArgs &args, cudaStream_t stream) {
   if (args.rows == 0) return kOk;
   if (args.gate_mode >= kGateRelu && (fp8 || args.output_f32 != nullptr))
     return fail(kInvalidArgument, "the F32 gates take BF16 operands and give BF16 results");
+  if (args.softcap > 0.0F && (args.output_f32 == nullptr || args.bias_f32 != nullptr))
+    return fail(kInvalidArgument, "a soft cap goes with F32 results without a bias");
   if (args.output_f32 != nullptr &&
       (fp8 || args.gate_mode != 0 || args.bias_mode != 0 || args.residual != nullptr))
     return fail(kInvalidArgument, "the F32-result mode takes BF16 operands and no BF16 epilogue");

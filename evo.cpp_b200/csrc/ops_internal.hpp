@@ -107,7 +107,7 @@ struct LinearArgs {
   float *output_f32 = nullptr;
   const float *bias_f32 = nullptr;
   bool accumulate_f32 = false;
-  float softcap = 0.0F;  // F32 results: softcap tanh(value / softcap) last (0: none)
+  float softcap = 0.0F;  // F32 results without a bias: softcap tanh(value / softcap) last (0: none)
   std::size_t weight_wrap_features = 0;
   // Grouped weights [groups, out_features, in_features] (BF16).  Tile form: rows come in whole tiles of tile_rows
   // (128 or 256), tile t belongs to group tile_group[t], *tile_count tiles are in use (both on the device; `rows`

@@ -1,7 +1,9 @@
-"""Throughput of a Gigusun decoder beside a StripedHyena2 stack of equal size (bench.py --design gigusun).
+"""Throughput of a decoder design beside the framework's closest other model at equal size (bench.py --design).
 
-Both models have the same width, number of blocks and weight count (the decoder's two feed-forward matrices
-are half again as wide as the three of the gated MLP), random weights and random tokens.  For every width:
+gigusun: beside a StripedHyena2 stack of the same width, number of blocks and weight count (the decoder's two
+feed-forward matrices are half again as wide as the three of the gated MLP).  kikepel: beside a Gigusun stack of
+window attention blocks of the same width, heads, head size, window and number of blocks, whose feed-forward has
+as many weights as a token meets in Kikepel's.  Random weights and random tokens.  For every width:
 prefill at several lengths (token ids on the device, CUDA events on the context's stream), cached decode
 (one public decode call per token, greedy, logits to the host), and the time of every operator class with its
 algorithmic work against the measured peaks.  Weights and activations exceed the 126 MB L2 in every step.
@@ -44,6 +46,94 @@ def decoder_config(art, width: int, max_positions: int) -> dict:
                               max_positions=max_positions)
 
 
+LATENT_BLOCKS = 6
+LATENT_EXPERTS = {2048: 32, 4096: 16}
+LATENT_TOP = 4
+
+
+def latent_config(art, width: int) -> dict:
+    """Kikepel: one dense block, then mixtures of experts; sinks in every other block."""
+    s = shapes(width)
+    H, experts = s["heads"], LATENT_EXPERTS[width]
+    layers = []
+    for i in range(LATENT_BLOCKS):
+        mlp = {"kind": "dense", "ff": s["inner"]} if i == 0 else {
+            "kind": "moe", "expert": {"ff": s["inner"] // LATENT_TOP, "limit": 7.0}, "router": {"experts": experts, "top": LATENT_TOP}}
+        layers.append({"type": ("latent_attention", "latent_attention_2")[i % 2], "mlp": mlp,
+                       "mixer": {"heads": H, "dim": 128, "vdim": 128, "q_rank": width * 3 // 8, "kv_rank": 512,
+                                 "scale": 128 ** -0.5, "mask": {"size": WINDOW}}})
+    return art.kikepel_config(layers, vocab=VOCAB, width=width)
+
+
+def window_stack_config(art, width: int, max_positions: int) -> dict:
+    """Gigusun's attention block alone, with a key/value head per query head."""
+    s = shapes(width)
+    H = s["heads"]
+    block = {"type": "attention", "mlp": {"kind": "dense", "ff": s["ff"]},
+             "mixer": {"heads": H, "kv_heads": H, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+                       "mask": {"size": WINDOW, "keep_first": 0}}}
+    return art.gigusun_config([block] * LATENT_BLOCKS, vocab=VOCAB, width=width, max_positions=max_positions)
+
+
+def seen_keys(tokens: int, context: int, size: int, keep: int = 0) -> int:
+    first = context - tokens
+    return sum(min(first + i + 1, size) + min(keep, max(0, first + i + 1 - size)) for i in range(tokens))
+
+
+def latent_work(config: dict, tokens: int, context: int) -> dict:
+    """class_work of a Kikepel configuration (prompts: keys and values are expanded from the latents)."""
+    D, T = config["width"], tokens
+    gemm, grouped, routing, attention = [0.0, 0.0], [0.0, 0.0], [0.0, 0.0], [0.0, 0.0]
+    norm_bytes = 6.0 * T * D
+
+    def product(total, rows, k, n, out_bytes):
+        total[0] += 2.0 * rows * k * n
+        total[1] += 2.0 * k * n + 2.0 * rows * k + rows * n * out_bytes
+
+    product(gemm, T, D, config["vocab"], 4.0)
+    for layer in config["layers"]:
+        m, mlp = layer["mixer"], layer["mlp"]
+        H, dim, vdim, q, c = m["heads"], m["dim"], m["vdim"], m["q_rank"], m["kv_rank"]
+        span = min(context, T + m["mask"]["size"] - 1)
+        product(gemm, T, D, q + c, 2.0)
+        product(gemm, T, q, H * dim, 2.0)
+        product(gemm, span, c, H * dim, 2.0)
+        product(gemm, span, c, H * vdim, 2.0)
+        product(gemm, T, H * vdim, D, 4.0)
+        norm_bytes += 4.0 * T * (q + c) + T * D * (4.0 + 8.0 + 2.0)
+        attention[0] += 2.0 * H * (dim + vdim) * seen_keys(T, context, m["mask"]["size"])
+        attention[1] += 2.0 * H * (T * (dim + vdim) + span * (dim + vdim))
+        if mlp is None:
+            continue
+        if mlp["kind"] == "dense":
+            product(gemm, T, D, 2 * mlp["ff"], 1.0)
+            product(gemm, T, mlp["ff"], D, 4.0)
+            norm_bytes += T * D * (4.0 + 8.0 + 2.0)
+            continue
+        E, top, ff = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+        pairs = T * top
+        grouped[0] += 6.0 * pairs * D * ff
+        grouped[1] += 6.0 * min(E, pairs) * D * ff + 2.0 * pairs * (2 * D + 2 * ff)
+        product(routing, T, D, E, 4.0)
+        routing[1] += 2.0 * T * D + 2.0 * pairs * D
+        norm_bytes += T * D * (2.0 * top + 8.0 + 2.0)
+    return {"gemm_bf16_tcgen05": (gemm[0], 0.0, gemm[1]), "gemm_grouped": (grouped[0], 0.0, grouped[1]),
+            "attention": (attention[0], 0.0, attention[1]), "rms_norm": (0.0, 0.0, norm_bytes),
+            "routing": (routing[0], 0.0, routing[1])}
+
+
+def token_weight_bytes(config: dict, art) -> float:
+    """Bytes of the weights that one token meets (its experts' only; one embedding row)."""
+    total = 0.0
+    for name, shape in art.decoder_manifest(config):
+        share = 1.0
+        if ".mlp.e" in name:
+            router = config["layers"][int(name[1:name.index(".")])]["mlp"]["router"]
+            share = router["top"] / router["experts"]
+        total += 2.0 * share * (shape[-1] if name in ("embed", "pos") else float(np.prod(shape)))
+    return total
+
+
 def class_work(config: dict, tokens: int, context: int) -> dict:
     """{operator class: (FLOPs on the tensor cores, F32 multiply-adds of the recurrences, HBM bytes)} of one pass
     over `tokens` rows whose last sees `context` keys."""
@@ -60,9 +150,7 @@ def class_work(config: dict, tokens: int, context: int) -> dict:
         if layer["type"] == "attention":
             columns = (H + G) * dim + G * vdim + H
             size, keep = m["mask"]["size"], m["mask"]["keep_first"]
-            first = context - T
-            seen = sum(min(first + i + 1, size) + min(keep, max(0, first + i + 1 - size)) for i in range(T))
-            attention_flops += 2.0 * H * (dim + vdim) * seen
+            attention_flops += 2.0 * H * (dim + vdim) * seen_keys(T, context, size, keep)
             keys = min(context, size + keep + T)
             attention_bytes += 2.0 * (T * H * (2 * dim + vdim) + 2 * G * (dim + vdim) * (T + keys))
         elif layer["type"] == "gla":
@@ -148,7 +236,7 @@ def timed_decode(context, prompt: list[int], steps: int) -> float:
 
 
 def measure(model, flags: int, lengths: list[int], decode_steps: int, steps: int, warmup: int, work, peaks: dict,
-            torch) -> dict:
+            torch, weight_bytes: float | None = None) -> dict:
     context = model.context(max(lengths) + 64, flags)
     vocab = model.vocab
     result = {"prefill": {}, "operators": {}}
@@ -166,16 +254,44 @@ def measure(model, flags: int, lengths: list[int], decode_steps: int, steps: int
     prompt = [int(t) for t in rng.integers(0, vocab, 1024)]
     if decode_steps:
         seconds = timed_decode(context, prompt, decode_steps)
+        read = weight_bytes if weight_bytes is not None else sum(s.weight_bytes for s in context.stages())
         result["decode_after_1024_tokens"] = {"ms_per_token": round(seconds * 1e3, 4),
-                                              "tokens_per_second": round(1.0 / seconds, 1),
-                                              "weight_bytes": sum(s.weight_bytes for s in context.stages()),
-                                              "of_weight_stream": round(sum(s.weight_bytes for s in context.stages()) /
-                                                                        (peaks["hbm_gbs"] * 1e9) / seconds, 3)}
+                                              "tokens_per_second": round(1.0 / seconds, 1), "weight_bytes": read,
+                                              "of_weight_stream": round(read / (peaks["hbm_gbs"] * 1e9) / seconds, 3)}
     context.close()
     return result
 
 
-def run(package, clock_sampler, steps: int, warmup: int, lengths: list[int], widths: list[int], decode_steps: int) -> dict:
+def decoder_arm(library, art, base: Path, config: dict, work, arguments: tuple, peaks: dict, torch) -> dict:
+    lengths, decode_steps, steps, warmup = arguments
+    directory = art.write_decoder_random(base / config["architecture"], config, 5, "cuda")
+    model = library.load(directory)
+    result = measure(model, 0, lengths, decode_steps, steps, warmup, lambda t: work(config, t, t), peaks, torch,
+                     token_weight_bytes(config, art))
+    model.close()
+    shutil.rmtree(directory)
+    gc.collect()
+    return result
+
+
+def hyena_arm(library, art, rt, base: Path, width: int, arguments: tuple, peaks: dict, torch) -> dict:
+    lengths, decode_steps, steps, warmup = arguments
+    s = shapes(width)
+    spec = art.fixture_spec(width=width, layers=BLOCKS, heads=s["heads"], inner=s["inner"], hcs_groups=width // 16,
+                            hcm_groups=width // 16, vocab=VOCAB)
+    path = base / f"hyena-{width}"
+    art.write_synthetic(path / "model.safetensors", spec, 6, device="cuda", max_shard_bytes=1 << 40)
+    model = library.load(path / "model.safetensors", flags=rt.MODEL_FLAG_ALLOW_SYNTHETIC)
+    result = measure(model, rt.CONTEXT_FLAG_TENSORCORE_FP8 | rt.CONTEXT_FLAG_FULL_ARENA, lengths, decode_steps, steps, warmup,
+                     lambda t: reference_work(width, BLOCKS, t), peaks, torch)
+    model.close()
+    shutil.rmtree(path)
+    gc.collect()
+    return result
+
+
+def run(package, clock_sampler, steps: int, warmup: int, lengths: list[int], widths: list[int], decode_steps: int,
+        design: str = "gigusun") -> dict:
     import torch
 
     art, rt = (importlib.import_module(f"{package.__name__}.{name}") for name in ("artifact", "runtime"))
@@ -186,32 +302,27 @@ def run(package, clock_sampler, steps: int, warmup: int, lengths: list[int], wid
         peaks.update({k: v for k, v in json.loads(peaks_file.read_text()).items() if k in peaks})
     properties = torch.cuda.get_device_properties(0)
     peaks["fma_per_second"] = 128.0 * properties.multi_processor_count * 1.9e9
-    line = {"design": "Gigusun", "dtype": "bf16", "data": "synthetic", "blocks": BLOCKS, "steps": steps, "warmup": warmup,
-            "window": WINDOW, "keep_first": KEEP, "peaks": peaks, "sizes": {}}
+    line = {"design": design.capitalize(), "dtype": "bf16", "data": "synthetic",
+            "blocks": LATENT_BLOCKS if design == "kikepel" else BLOCKS, "steps": steps, "warmup": warmup,
+            "window": WINDOW, "keep_first": 0 if design == "kikepel" else KEEP, "peaks": peaks, "sizes": {}}
     base = Path(tempfile.mkdtemp(prefix="decoder_bench_"))
+    arguments = (lengths, decode_steps, steps, warmup)
     try:
         with clock_sampler(0) as clocks:
             for width in widths:
-                s = shapes(width)
                 longest = max(lengths)
-                config = decoder_config(art, width, longest + 64)
-                directory = art.write_gigusun_random(base / f"decoder-{width}", config, 5, "cuda")
-                model = library.load(directory)
-                decoder = measure(model, 0, lengths, decode_steps, steps, warmup,
-                                  lambda t: class_work(config, t, t), peaks, torch)
-                model.close()
-                shutil.rmtree(directory)
-                spec = art.fixture_spec(width=width, layers=BLOCKS, heads=s["heads"], inner=s["inner"],
-                                        hcs_groups=width // 16, hcm_groups=width // 16, vocab=VOCAB)
-                path = base / f"hyena-{width}"
-                art.write_synthetic(path / "model.safetensors", spec, 6, device="cuda", max_shard_bytes=1 << 40)
-                model = library.load(path / "model.safetensors", flags=rt.MODEL_FLAG_ALLOW_SYNTHETIC)
-                hyena = measure(model, rt.CONTEXT_FLAG_TENSORCORE_FP8 | rt.CONTEXT_FLAG_FULL_ARENA, lengths, decode_steps,
-                                steps, warmup, lambda t: reference_work(width, BLOCKS, t), peaks, torch)
-                model.close()
-                shutil.rmtree(path)
-                gc.collect()
-                line["sizes"][str(width)] = {"shape": s, "gigusun": decoder, "striped_hyena2": hyena}
+                result = {"shape": shapes(width)}
+                if design == "kikepel":
+                    result["shape"].update(experts=LATENT_EXPERTS[width], top=LATENT_TOP)
+                    result["kikepel"] = decoder_arm(library, art, base, latent_config(art, width), latent_work, arguments,
+                                                    peaks, torch)
+                    result["gigusun_attention"] = decoder_arm(library, art, base, window_stack_config(art, width, longest + 64),
+                                                              class_work, arguments, peaks, torch)
+                else:
+                    result["gigusun"] = decoder_arm(library, art, base, decoder_config(art, width, longest + 64), class_work,
+                                                    arguments, peaks, torch)
+                    result["striped_hyena2"] = hyena_arm(library, art, rt, base, width, arguments, peaks, torch)
+                line["sizes"][str(width)] = result
         line["clocks"] = clocks.summary()
     finally:
         shutil.rmtree(base, ignore_errors=True)

@@ -32,11 +32,11 @@ def make_model(pkg, directory, layers, seed=1, *, vocab=300, width=56, max_posit
     change the F32 weights in place (values are rounded to BF16 again before they are written)."""
     art = artifacts(pkg)
     config = art.gigusun_config(layers, vocab=vocab, width=width, max_positions=max_positions, eps=eps)
-    weights = art.gigusun_weights(config, seed, decay_rank)
+    weights = art.decoder_weights(config, seed, decay_rank)
     if edit is not None:
         edit(weights)
         for name, values in weights.items():
             bits = np.frombuffer(art._bf16_bytes(values), np.uint16).astype(np.uint32) << 16
             weights[name] = bits.view(np.float32).reshape(values.shape)
-    art.write_gigusun(directory, config, weights)
+    art.write_decoder(directory, config, weights)
     return directory, config, {name: values.astype(np.float64) for name, values in weights.items()}

@@ -66,7 +66,7 @@ def test_missing_tensors_are_refused_and_foreign_headers_are_read(pkg, rt, evo, 
     directory, config, weights = make_model(pkg, tmp_path / "m", [gla()])
     art = artifacts(pkg)
     kept = {k: v.astype(np.float32) for k, v in weights.items() if k != "l0.mix.a2.b"}
-    art.write_gigusun(tmp_path / "missing", config, kept)
+    art.write_decoder(tmp_path / "missing", config, kept)
     with pytest.raises(rt.EvoError) as error:
         evo.read_model_config(tmp_path / "missing")
     assert error.value.code == 4 and "a2.b" in str(error.value)
