@@ -76,6 +76,15 @@ OPS_SIGNATURES.update({
     "evo_b200_head_norm_append": [_P, _P],
     "evo_b200_window_attention": [_P, _P],
     "evo_b200_recurrent_mixer": [_P, _P],
+    "evo_b200_embed_rows": [_P, _P, _Z, _Z, _Z, _P, _P, _I, _P],
+    "evo_b200_layer_norm": [_P, _P],
+    "evo_b200_projection": [_P, _P],
+    "evo_b200_gated_activation": [_P, _I, _F, _Z, _Z, _P, _I, _P, _Z, _P],
+    "evo_b200_route_rows": [_P, _P],
+    "evo_b200_group_rows": [_P, _P],
+    "evo_b200_latent_norm_append": [_P, _P],
+    "evo_b200_absorb_queries": [_P, _P, _Z, _Z, _Z, _Z, _P, _I, _P],
+    "evo_b200_expand_values": [_P, _P, _Z, _Z, _Z, _Z, _P, _I, _P],
 })
 
 
@@ -98,7 +107,33 @@ class HeadNorm(_Arguments):
 class WindowAttention(_Arguments):
     _fields_ = _fields("z struct_size|p query key_cache value_cache gate|z gate_stride|p distance_bias|z bias_stride|"
                        "p output|z rows position capacity heads kv_heads dim value_dim window keep_first|"
-                       "f scale softcap|i sink float32 kernel")
+                       "f scale softcap|i sink float32 kernel|p sink_logit")
+
+
+class LayerNorm(_Arguments):
+    _fields_ = _fields("z struct_size|p input slots gain residual output|z parts rows width|f epsilon|"
+                       "i input_float32 output_float32")
+
+
+class Projection(_Arguments):
+    _fields_ = _fields("z struct_size|p input weight bias row_scale output|z rows in_features out_features|"
+                       "f alpha softcap gate_limit|i gate f32_result float32|z groups|p tile_group tile_count row_group|"
+                       "z tile_rows row_fanout|p split_workspace|z split_workspace_bytes")
+
+
+class Route(_Arguments):
+    _fields_ = _fields("z struct_size|p input router logits|z logit_stride rows width experts top|"
+                       "p expert score counts rank|i float32")
+
+
+class GroupRows(_Arguments):
+    _fields_ = _fields("z struct_size|p input expert rank counts score grouped slot_score slot tile_group tile_count|"
+                       "z rows width experts top tile_rows|i float32")
+
+
+class LatentNorm(_Arguments):
+    _fields_ = _fields("z struct_size|p projection query_gain latent_gain query_latent cache|z stride latent_column rows "
+                       "position capacity query_rank latent_rank|f epsilon|i float32")
 
 
 class Recurrent(_Arguments):
@@ -109,7 +144,7 @@ class Recurrent(_Arguments):
 
 
 # entry points that do not return a status
-OPS_OTHER = ("evo_b200_last_error", "evo_b200_recurrent_workspace_bytes", "evo_b200_hcl_scratch_floats", "evo_b200_linear_executor_free",
+OPS_OTHER = ("evo_b200_last_error", "evo_b200_recurrent_workspace_bytes", "evo_b200_grouped_tiles", "evo_b200_hcl_scratch_floats", "evo_b200_linear_executor_free",
              "evo_b200_linear_executor_name", "evo_b200_linear_executor_cached_bytes",
              "evo_b200_e4m3_encode", "evo_b200_e4m3_decode", "evo_b200_e4m3_scaled_roundtrip")
 
@@ -132,6 +167,8 @@ class Ops:
         self.lib.evo_b200_last_error.restype = ctypes.c_char_p
         self.lib.evo_b200_recurrent_workspace_bytes.restype = _Z
         self.lib.evo_b200_recurrent_workspace_bytes.argtypes = [_I, _Z, _Z, _Z, _Z, _Z, _I]
+        self.lib.evo_b200_grouped_tiles.restype = _Z
+        self.lib.evo_b200_grouped_tiles.argtypes = [_Z, _Z, _Z, _Z]
         self.lib.evo_b200_hcl_scratch_floats.restype = _Z
         self.lib.evo_b200_hcl_scratch_floats.argtypes = [_Z, _Z, _Z]
         self.lib.evo_b200_linear_executor_free.restype = None

@@ -680,6 +680,7 @@ int evo_b200_window_attention(const evo_b200_window_attention_args *args, void *
   a.scale = args->scale;
   a.softcap = args->softcap;
   a.sink = args->sink != 0;
+  a.sink_logit = static_cast<const float *>(args->sink_logit);
   a.type = activation_of(args->float32);
   a.force = args->kernel;
   return window_attention(a, as_stream(stream));
@@ -722,6 +723,142 @@ int evo_b200_recurrent_mixer(const evo_b200_recurrent_args *args, void *stream) 
   a.output = args->output;
   a.type = activation_of(args->float32);
   return recurrent_mixer(a, as_stream(stream));
+}
+int evo_b200_embed_rows(const void *tokens, const void *table, size_t rows, size_t width, size_t vocabulary,
+                        void *stream_rows, void *copy, int float32, void *stream) {
+  return embed_rows(static_cast<const std::uint32_t *>(tokens), table, rows, width, vocabulary,
+                    static_cast<float *>(stream_rows), copy, activation_of(float32), as_stream(stream));
+}
+int evo_b200_layer_norm(const evo_b200_layer_norm_args *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args)) return fail(kInvalidArgument, "layer norm arguments are required");
+  LayerNormArgs a;
+  a.input = args->input;
+  a.input_type = activation_of(args->input_float32);
+  a.slots = static_cast<const int *>(args->slots);
+  a.parts = args->parts;
+  a.gain = static_cast<const float *>(args->gain);
+  a.residual = static_cast<float *>(args->residual);
+  a.output = args->output;
+  a.output_type = activation_of(args->output_float32);
+  a.rows = args->rows;
+  a.width = args->width;
+  a.epsilon = args->epsilon;
+  return layer_norm(a, as_stream(stream));
+}
+int evo_b200_projection(const evo_b200_projection_args *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args)) return fail(kInvalidArgument, "projection arguments are required");
+  const auto shared = [&](auto &a) {
+    a.input = args->input;
+    a.weight = args->weight;
+    a.row_scale = static_cast<const float *>(args->row_scale);
+    a.rows = args->rows;
+    a.in_features = args->in_features;
+    a.out_features = args->out_features;
+    a.alpha = args->alpha;
+    a.softcap = args->softcap;
+    a.tile_group = static_cast<const int *>(args->tile_group);
+    a.tile_count = static_cast<const int *>(args->tile_count);
+    a.row_group = static_cast<const int *>(args->row_group);
+    a.tile_rows = args->tile_rows;
+    a.row_fanout = args->row_fanout;
+  };
+  if (args->float32 != 0) {
+    if (args->gate != 0) return fail(kInvalidArgument, "F32 projections apply no gate");
+    LinearF32Args a;
+    shared(a);
+    a.input_type = activation_of(args->float32 == 1);
+    a.bias = static_cast<const float *>(args->bias);
+    a.output = static_cast<float *>(args->output);
+    return linear_f32(a, as_stream(stream));
+  }
+  LinearArgs a;
+  shared(a);
+  a.bias_f32 = static_cast<const float *>(args->bias);
+  a.groups = args->groups;
+  a.gate_mode = args->gate;
+  a.gate_limit = args->gate_limit;
+  a.split_workspace = args->split_workspace;
+  a.split_workspace_bytes = args->split_workspace_bytes;
+  if (args->f32_result != 0) a.output_f32 = static_cast<float *>(args->output);
+  else a.output = args->output;
+  return linear(a, as_stream(stream));
+}
+int evo_b200_gated_activation(const void *input, int gate, float limit, size_t rows, size_t inner, void *output,
+                              int float32, const void *tile_count, size_t tile_rows, void *stream) {
+  return gated_activation(static_cast<const float *>(input), gate, limit, rows, inner, output, activation_of(float32),
+                          static_cast<const int *>(tile_count), tile_rows, as_stream(stream));
+}
+int evo_b200_route_rows(const evo_b200_route_args *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args)) return fail(kInvalidArgument, "router arguments are required");
+  RouteArgs a;
+  a.input = args->input;
+  a.type = activation_of(args->float32);
+  a.router = args->router;
+  a.logits = static_cast<const float *>(args->logits);
+  a.logit_stride = args->logit_stride;
+  a.rows = args->rows;
+  a.width = args->width;
+  a.experts = args->experts;
+  a.top = args->top;
+  a.expert = static_cast<int *>(args->expert);
+  a.score = static_cast<float *>(args->score);
+  a.counts = static_cast<int *>(args->counts);
+  a.rank = static_cast<int *>(args->rank);
+  return route_rows(a, as_stream(stream));
+}
+int evo_b200_group_rows(const evo_b200_group_rows_args *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args))
+    return fail(kInvalidArgument, "row grouping arguments are required");
+  GroupRowsArgs a;
+  a.input = args->input;
+  a.type = activation_of(args->float32);
+  a.rows = args->rows;
+  a.width = args->width;
+  a.experts = args->experts;
+  a.top = args->top;
+  a.tile_rows = args->tile_rows;
+  a.expert = static_cast<const int *>(args->expert);
+  a.rank = static_cast<const int *>(args->rank);
+  a.counts = static_cast<const int *>(args->counts);
+  a.score = static_cast<const float *>(args->score);
+  a.grouped = args->grouped;
+  a.slot_score = static_cast<float *>(args->slot_score);
+  a.slot = static_cast<int *>(args->slot);
+  a.tile_group = static_cast<int *>(args->tile_group);
+  a.tile_count = static_cast<int *>(args->tile_count);
+  return group_rows(a, as_stream(stream));
+}
+size_t evo_b200_grouped_tiles(size_t rows, size_t top, size_t experts, size_t tile_rows) {
+  return tile_rows == 0 ? 0 : grouped_tiles(rows, top, experts, tile_rows);
+}
+int evo_b200_latent_norm_append(const evo_b200_latent_norm_args *args, void *stream) {
+  if (args == nullptr || args->struct_size < sizeof(*args))
+    return fail(kInvalidArgument, "latent norm arguments are required");
+  LatentNormArgs a;
+  a.projection = args->projection;
+  a.stride = args->stride;
+  a.latent_column = args->latent_column;
+  a.query_gain = static_cast<const float *>(args->query_gain);
+  a.latent_gain = static_cast<const float *>(args->latent_gain);
+  a.query_latent = args->query_latent;
+  a.cache = args->cache;
+  a.rows = args->rows;
+  a.position = args->position;
+  a.capacity = args->capacity;
+  a.query_rank = args->query_rank;
+  a.latent_rank = args->latent_rank;
+  a.epsilon = args->epsilon;
+  a.type = activation_of(args->float32);
+  return latent_norm_append(a, as_stream(stream));
+}
+int evo_b200_absorb_queries(const void *query, const void *key_up, size_t rows, size_t heads, size_t dim,
+                            size_t latent_rank, void *absorbed, int float32, void *stream) {
+  return absorb_queries(query, key_up, rows, heads, dim, latent_rank, absorbed, activation_of(float32), as_stream(stream));
+}
+int evo_b200_expand_values(const void *mixed, const void *value_up, size_t rows, size_t heads, size_t value_dim,
+                           size_t latent_rank, void *output, int float32, void *stream) {
+  return expand_values(mixed, value_up, rows, heads, value_dim, latent_rank, output, activation_of(float32),
+                       as_stream(stream));
 }
 
 }  // extern "C"

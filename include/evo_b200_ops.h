@@ -407,9 +407,11 @@ typedef struct evo_b200_head_norm {
 EVO_B200_API int evo_b200_head_norm_append(const evo_b200_head_norm *args, void *stream);
 /* Softmax attention with grouped key/value heads [capacity, kv_heads, dim]: the query at position i sees key
  * j <= i if i - j < window (0: no limit) or j < keep_first; score = softcap tanh(q.k scale / softcap)
- * (softcap 0: q.k scale) - distance_bias[head, i - j] (optional); sink != 0 adds exp(0) to the denominator;
+ * (softcap 0: q.k scale) - distance_bias[head, i - j] (optional); sink != 0 adds exp(sink_logit[head]) to the
+ * denominator (exp(0) without sink_logit, F32 on the device);
  * output [rows, heads, value_dim] times sigmoid(gate[r * gate_stride + head]) (optional).  kernel: 0 chosen by
- * size, 1 row kernel, 2 tile kernel, 3 tcgen05 kernel (EVO_STATUS_UNSUPPORTED where it does not apply). */
+ * size, 1 row kernel, 2 tile kernel, 3 tcgen05 kernel (EVO_STATUS_UNSUPPORTED where it does not apply).  Head sizes
+ * up to 256; up to 1024 in the row kernel. */
 typedef struct evo_b200_window_attention_args {
   size_t struct_size;
   const void *query, *key_cache, *value_cache, *gate;
@@ -420,6 +422,7 @@ typedef struct evo_b200_window_attention_args {
   size_t rows, position, capacity, heads, kv_heads, dim, value_dim, window, keep_first;
   float scale, softcap;
   int32_t sink, float32, kernel;
+  const void *sink_logit;
 } evo_b200_window_attention_args;
 EVO_B200_API int evo_b200_window_attention(const evo_b200_window_attention_args *args, void *stream);
 /* Gated linear attention (delta == 0) or the gated delta rule with its short convolutions, with the output
@@ -447,6 +450,87 @@ typedef struct evo_b200_recurrent_args {
 EVO_B200_API size_t evo_b200_recurrent_workspace_bytes(int delta, size_t rows, size_t heads, size_t kv_heads,
                                                        size_t dim, size_t value_dim, int float32);
 EVO_B200_API int evo_b200_recurrent_mixer(const evo_b200_recurrent_args *args, void *stream);
+/* stream_rows[r] = table[token[r]] widened to F32, and the same row in the activation type in copy (optional). */
+EVO_B200_API int evo_b200_embed_rows(const void *tokens, const void *table, size_t rows, size_t width,
+                                     size_t vocabulary, void *stream_rows, void *copy, int float32, void *stream);
+/* y = the sum of the `parts` input rows slots[r * parts + k] (r * parts + k without slots);
+ * n = (y - mean) / sqrt(variance + epsilon) * gain.  With a residual (F32): residual[r] += n and the new row in
+ * output (optional); without: n in output. */
+typedef struct evo_b200_layer_norm_args {
+  size_t struct_size;
+  const void *input, *slots, *gain;
+  void *residual, *output;
+  size_t parts, rows, width;
+  float epsilon;
+  int32_t input_float32, output_float32;
+} evo_b200_layer_norm_args;
+EVO_B200_API int evo_b200_layer_norm(const evo_b200_layer_norm_args *args, void *stream);
+/* Projections with gates and groups.  output (or, with f32_result, an F32 output) = alpha row_scale[r] x W^T + bias,
+ * soft cap softcap tanh(. / softcap) last.  gate 3: max(a, 0) b, 4: g sigmoid(1.702 g) (u + 1) with g = min(a, limit),
+ * u = clamp(b, +-limit), over weight rows in alternating blocks of 128 gate and 128 up rows; output [rows,
+ * out_features / 2].  bias F32 in the weight's row order.  Grouped weights [groups, out, in]: row_group [rows] with
+ * row_fanout output rows per input row, or tiles of tile_rows (128, 256) rows with tile_group and tile_count (all
+ * int32 on the device).  float32: F32 operands and results in F32 multiply-adds (gate: 0 only); 2: BF16 operands in
+ * the same kernels. */
+typedef struct evo_b200_projection_args {
+  size_t struct_size;
+  const void *input, *weight, *bias, *row_scale;
+  void *output;
+  size_t rows, in_features, out_features;
+  float alpha, softcap, gate_limit;
+  int32_t gate, f32_result, float32;
+  size_t groups;
+  const void *tile_group, *tile_count, *row_group;
+  size_t tile_rows, row_fanout;
+  void *split_workspace;
+  size_t split_workspace_bytes;
+} evo_b200_projection_args;
+EVO_B200_API int evo_b200_projection(const evo_b200_projection_args *args, void *stream);
+/* The gates 3 and 4 on F32 products [rows, 2 * inner] in blocks of 128 columns; output [rows, inner]; with tile_count
+ * only the rows of its tiles. */
+EVO_B200_API int evo_b200_gated_activation(const void *input, int gate, float limit, size_t rows, size_t inner,
+                                           void *output, int float32, const void *tile_count, size_t tile_rows,
+                                           void *stream);
+/* Mixture of experts: the `top` largest of sigmoid(x . router[e]) per row, best first (expert, score [rows * top]),
+ * from logits [rows, logit_stride] or from the products the kernel makes itself; counts [experts] and rank
+ * [rows * top] (optional) number the rows of every expert. */
+typedef struct evo_b200_route_args {
+  size_t struct_size;
+  const void *input, *router, *logits;
+  size_t logit_stride, rows, width, experts, top;
+  void *expert, *score, *counts, *rank;
+  int32_t float32;
+} evo_b200_route_args;
+EVO_B200_API int evo_b200_route_rows(const evo_b200_route_args *args, void *stream);
+/* Copies of the rows grouped by expert, every expert in whole tiles of tile_rows: grouped[slot[pair]] =
+ * input[pair / top], slot_score[slot[pair]] = score[pair]; tile_group[t] and *tile_count describe the tiles (at most
+ * evo_b200_grouped_tiles of them, which also bounds grouped and slot_score). */
+typedef struct evo_b200_group_rows_args {
+  size_t struct_size;
+  const void *input, *expert, *rank, *counts, *score;
+  void *grouped, *slot_score, *slot, *tile_group, *tile_count;
+  size_t rows, width, experts, top, tile_rows;
+  int32_t float32;
+} evo_b200_group_rows_args;
+EVO_B200_API int evo_b200_group_rows(const evo_b200_group_rows_args *args, void *stream);
+EVO_B200_API size_t evo_b200_grouped_tiles(size_t rows, size_t top, size_t experts, size_t tile_rows);
+/* RMS norms of the query latent (column 0, to query_latent [rows, query_rank]) and the key/value latent (column
+ * latent_column, to row position + r of cache [capacity, latent_rank]) of projection rows. */
+typedef struct evo_b200_latent_norm_args {
+  size_t struct_size;
+  const void *projection, *query_gain, *latent_gain;
+  void *query_latent, *cache;
+  size_t stride, latent_column, rows, position, capacity, query_rank, latent_rank;
+  float epsilon;
+  int32_t float32;
+} evo_b200_latent_norm_args;
+EVO_B200_API int evo_b200_latent_norm_append(const evo_b200_latent_norm_args *args, void *stream);
+/* Up to eight rows: absorbed[r, h] = sum_d query[r, h, d] key_up[h * dim + d, :], and output[r, h, d] =
+ * value_up[h * value_dim + d, :] . mixed[r, h, :]. */
+EVO_B200_API int evo_b200_absorb_queries(const void *query, const void *key_up, size_t rows, size_t heads, size_t dim,
+                                         size_t latent_rank, void *absorbed, int float32, void *stream);
+EVO_B200_API int evo_b200_expand_values(const void *mixed, const void *value_up, size_t rows, size_t heads,
+                                        size_t value_dim, size_t latent_rank, void *output, int float32, void *stream);
 
 #ifdef __cplusplus
 }
