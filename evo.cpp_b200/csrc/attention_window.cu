@@ -481,6 +481,7 @@ int window_attention(const WindowAttentionArgs &a, cudaStream_t stream) {
     if (window_attention_tcgen05_applicable(a)) return window_attention_tcgen05(a, stream);
     if (a.force == 3) return fail(kUnsupported, "the tensor-core attention kernel does not take these sizes");
   }
+  if (a.force == 4 || (a.force == 0 && a.rows <= kLatentRows && latent_decode_applicable(a))) return latent_decode(a, stream);
   const bool wide = a.dim > kDecoderMaxHeadDim || a.value_dim > kDecoderMaxHeadDim;
   if (a.force == 1 || (a.force == 0 && (a.rows <= 8 || wide))) {
     if (a.rows > 65535) return fail(kInvalidArgument, "too many rows for the row kernel");

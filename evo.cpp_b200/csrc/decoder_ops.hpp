@@ -178,12 +178,17 @@ struct WindowAttentionArgs {
   const float *sink_logit = nullptr;  // [heads]
   Activation type = Activation::kBf16;
   const int *dynamic_position = nullptr;
-  int force = 0;  // tests: 1 the row kernel, 2 the tile kernel, 3 the tcgen05 kernel (refused where it does not apply)
+  // tests: 1 the row kernel, 2 the tile kernel, 3 the tcgen05 kernel, 4 the latent kernel (refused where it does not apply)
+  int force = 0;
 };
 int window_attention(const WindowAttentionArgs &args, cudaStream_t stream);
 // attention_tcgen05_k64.cu: the same contract on the tensor cores (BF16, head sizes up to 128 in steps of 8).
 bool window_attention_tcgen05_applicable(const WindowAttentionArgs &args);
 int window_attention_tcgen05(const WindowAttentionArgs &args, cudaStream_t stream);
+// latent_attention.cu: the same contract for a few BF16 queries of all heads to one shared head whose keys are its
+// values (latents of up to 512 columns in steps of 64), plain softmax in a window, with or without sinks.
+bool latent_decode_applicable(const WindowAttentionArgs &args);
+int latent_decode(const WindowAttentionArgs &args, cudaStream_t stream);
 
 // ---- recurrent_mixers.cu
 // Both recurrences keep one F32 state [heads, dim, value_dim] per sequence.  `fresh` starts from zero

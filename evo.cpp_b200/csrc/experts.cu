@@ -76,7 +76,7 @@ route_logits_kernel(const float *__restrict__ logits, const std::size_t stride, 
 }
 
 // A cluster per row: every CTA makes its share of the products, rank 0 chooses.
-template <typename T, bool kVector>
+template <typename T, bool kVector, int kPerLane>
 __global__ void __launch_bounds__(32 * kRouteWarps)
 route_rows_kernel(const T *__restrict__ input, const bf16 *__restrict__ router, const int width, const Choice c) {
   // a grouped projection launched with programmatic stream serialisation may start under this kernel
@@ -108,10 +108,10 @@ route_rows_kernel(const T *__restrict__ input, const bf16 *__restrict__ router, 
   }
   cluster.sync();
   if (split != 0 || warp != 0) return;
-  float logit[kMaxPerLane];
+  float logit[kPerLane];
 #pragma unroll
-  for (int i = 0; i < kMaxPerLane; ++i) logit[i] = lane + 32 * i < c.experts ? logits[lane + 32 * i] : -INFINITY;
-  choose<kMaxPerLane>(logit, c, row, lane);
+  for (int i = 0; i < kPerLane; ++i) logit[i] = lane + 32 * i < c.experts ? logits[lane + 32 * i] : -INFINITY;
+  choose<kPerLane>(logit, c, row, lane);
 }
 
 constexpr int kGroupThreads = 256;
@@ -179,7 +179,10 @@ int launch_route_rows(const RouteArgs &a, const Choice &c, cudaStream_t stream) 
   config.stream = stream;
   config.attrs = &attribute;
   config.numAttrs = 1;
-  if (cudaLaunchKernelEx(&config, vector ? route_rows_kernel<T, true> : route_rows_kernel<T, false>,
+  const auto kernel = a.experts <= 64 ? (vector ? route_rows_kernel<T, true, 2> : route_rows_kernel<T, false, 2>)
+                                      : (vector ? route_rows_kernel<T, true, kMaxPerLane>
+                                                : route_rows_kernel<T, false, kMaxPerLane>);
+  if (cudaLaunchKernelEx(&config, kernel,
                          static_cast<const T *>(a.input), static_cast<const bf16 *>(a.router), static_cast<int>(a.width),
                          c) != cudaSuccess)
     return fail(kCuda, std::string("cannot launch the router kernel: ") + cudaGetErrorString(cudaGetLastError()));

@@ -410,7 +410,8 @@ EVO_B200_API int evo_b200_head_norm_append(const evo_b200_head_norm *args, void 
  * (softcap 0: q.k scale) - distance_bias[head, i - j] (optional); sink != 0 adds exp(sink_logit[head]) to the
  * denominator (exp(0) without sink_logit, F32 on the device);
  * output [rows, heads, value_dim] times sigmoid(gate[r * gate_stride + head]) (optional).  kernel: 0 chosen by
- * size, 1 row kernel, 2 tile kernel, 3 tcgen05 kernel (EVO_STATUS_UNSUPPORTED where it does not apply).  Head sizes
+ * size, 1 row kernel, 2 tile kernel, 3 tcgen05 kernel, 4 latent kernel (EVO_STATUS_UNSUPPORTED where it does not
+ * apply).  Head sizes
  * up to 256; up to 1024 in the row kernel. */
 typedef struct evo_b200_window_attention_args {
   size_t struct_size;

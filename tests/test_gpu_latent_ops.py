@@ -377,6 +377,18 @@ def test_grouped_refusals(pkg, ops):
 
 
 # ---------------------------------------------------------------- attention
+def last_rows(q, k, v, *, scale, window, sink):
+    """oracle.attention of the last len(q) rows alone."""
+    position = len(k) - len(q)
+    out = np.zeros((*q.shape[:2], v.shape[2]))
+    for r in range(len(q)):
+        seen = oracle.visible_keys(position + r, window)
+        for h in range(q.shape[1]):
+            g = h // (q.shape[1] // k.shape[1])
+            out[r, h] = oracle.softmax((k[seen, g] @ q[r, h]) * scale, None if sink is None else float(sink[h])) @ v[seen, g]
+    return out
+
+
 def attention_case(pkg, ops, *, rows, position, heads, kv_heads, dim, vdim, window, kernel, float32=0, sinks=True, seed=0,
                    edit=None, sink_range=(-2.0, 4.0)):
     """Plain softmax in a window with learned sinks; returns (output, expected [rows, heads, vdim])."""
@@ -393,11 +405,7 @@ def attention_case(pkg, ops, *, rows, position, heads, kv_heads, dim, vdim, wind
         query=dq.data_ptr(), key_cache=dk.data_ptr(), value_cache=dv.data_ptr(), output=out.data_ptr(), rows=rows, position=position,
         capacity=capacity, heads=heads, kv_heads=kv_heads, dim=dim, value_dim=vdim, window=window, scale=dim ** -0.5,
         sink=int(sinks), sink_logit=ds.data_ptr(), float32=float32, kernel=kernel))
-    group = heads // kv_heads
-    expected = oracle.attention(np.concatenate([np.zeros((position, heads, dim)), q]), np.repeat(k[:total], group, axis=1),
-                                np.repeat(v[:total], group, axis=1), scale=dim ** -0.5, size=window,
-                                sink=sink if sinks else None)[position:]
-    return out, expected
+    return out, last_rows(q, k[:total], v[:total], scale=dim ** -0.5, window=window, sink=sink if sinks else None)
 
 
 ROW, TILE, TENSOR = 1, 2, 3
@@ -457,6 +465,56 @@ def test_one_key_stands_out(pkg, ops, kernel, dim, key_at):
     assert visible[60] == (key_at in ("oldest in the window", "own"))
 
 
+LATENT = 4
+
+
+def latent_case(pkg, ops, *, rows, position, heads, rank, window, sinks=True, seed=0, edit=None, kernel=LATENT):
+    """Queries against latents that are keys and values; returns (output, expected [rows, heads, rank])."""
+    rng = np.random.default_rng(seed)
+    total, capacity = position + rows, position + rows + 70
+    q, c = rng.normal(0, 1, (rows, heads, rank)), rng.normal(0, 1, (capacity, rank))
+    if edit is not None:
+        edit(q, c)
+    c[total:] = np.nan                                              # what lies behind the last token is never read
+    (dq, q), (dc, c) = activation(q, 0), activation(c, 0)
+    sink = rng.uniform(-2.0, 4.0, heads).astype(np.float32)
+    ds, out = cuda(sink), empty((rows, heads, rank), 0)
+    call(ops, "window_attention", pkg.WindowAttention(
+        query=dq.data_ptr(), key_cache=dc.data_ptr(), value_cache=dc.data_ptr(), output=out.data_ptr(), rows=rows, position=position,
+        capacity=capacity, heads=heads, kv_heads=1, dim=rank, value_dim=rank, window=window, scale=rank ** -0.5, sink=int(sinks),
+        sink_logit=ds.data_ptr(), kernel=kernel))
+    shared = c[:total, None]
+    return out, last_rows(q, shared, shared, scale=rank ** -0.5, window=window, sink=sink if sinks else None)
+
+
+@pytest.mark.parametrize("kernel", [LATENT, 0])
+@pytest.mark.parametrize("sinks", [True, False])
+@pytest.mark.parametrize("rank", [64, 128, 192, 256, 320, 384, 448, 512])
+def test_latent_kernel(pkg, ops, rank, sinks, kernel):
+    for rows, position, heads, window in ((1, 0, 1, 9), (1, 6, 16, 100), (2, 500, 17, 500), (8, 700, 5, 127), (1, 1300, 33, 1024),
+                                          (3, 65, 12, 64)):
+        out, expected = latent_case(pkg, ops, rows=rows, position=position, heads=heads, rank=rank, window=window, sinks=sinks,
+                                    seed=rank + rows, kernel=kernel)
+        assert_near(out, expected, 0, factor=2.0)
+
+
+@pytest.mark.parametrize("target", [0, 1, 62, 63, 64, 65, 127, 300, 511, 512])
+def test_one_latent_stands_out(pkg, ops, target):
+    """One token far above the rest, at the borders of tiles and of the shares of a cluster, just inside and just
+    outside the window."""
+    position, window = 600, 537                                      # sees 64 .. 600; the row before it 63 .. 599
+
+    def plant(q, c):
+        q *= 0.02
+        q[..., 0], c[:, 0] = 4.0, 0.0
+        c[target, 0], c[target, 1:] = 40.0, 9.0
+
+    out, expected = latent_case(pkg, ops, rows=2, position=position - 1, heads=3, rank=128, window=window, edit=plant, sinks=False)
+    assert_near(out, expected, 0, factor=2.0)
+    mean = out.float().cpu().numpy()[..., 1:].mean(axis=(1, 2))
+    assert list(mean > 6.0) == [target >= 63, target >= 64]
+
+
 @TYPES
 @pytest.mark.parametrize("rows, heads, dim, vdim, rank", [(1, 3, 24, 40, 72), (2, 5, 128, 128, 512), (4, 1, 1, 3, 1), (7, 4, 33, 7, 51),
                                                          (8, 2, 200, 96, 1000)])
@@ -487,6 +545,9 @@ def test_absorbed_heads_equal_expanded_heads(pkg, ops, float32, rows, heads, dim
 
 def test_latent_refusals(pkg, ops):
     x = empty((64, 64), 0)
+    with pytest.raises(pkg.OpsError) as error:
+        latent_case(pkg, ops, rows=1, position=3, heads=2, rank=72, window=5)
+    assert error.value.code == 5
     for rows, rank in ((9, 8), (1, 1025)):
         with pytest.raises(pkg.OpsError) as error:
             ops.call("absorb_queries", x.data_ptr(), x.data_ptr(), rows, 1, 8, rank, x.data_ptr(), 0, stream())
