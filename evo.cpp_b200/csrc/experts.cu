@@ -81,14 +81,13 @@ __global__ void __launch_bounds__(32 * kRouteWarps)
 route_rows_kernel(const T *__restrict__ input, const bf16 *__restrict__ router, const int width, const Choice c) {
   // a grouped projection launched with programmatic stream serialisation may start under this kernel
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  __shared__ float logits[kDecoderMaxExperts];  // rank 0's are complete
+  __shared__ float logits[kDecoderMaxExperts / kRouterSplits + kRouteWarps];  // of this CTA's experts
   cg::cluster_group cluster = cg::this_cluster();
   const int split = static_cast<int>(cluster.block_rank()), warp = threadIdx.x / 32, lane = threadIdx.x % 32;
   const std::size_t row = blockIdx.y;
   const T *const x = input + row * width;
-  float *const target = cluster.map_shared_rank(logits, 0);
-  cluster.sync();  // rank 0 runs before anything is written to it
-  for (int e = split * kRouteWarps + warp; e < c.experts; e += kRouterSplits * kRouteWarps) {
+  // expert e is the CTA's number e / kRouterSplits
+  for (int e = split + kRouterSplits * warp; e < c.experts; e += kRouterSplits * kRouteWarps) {
     const bf16 *const w = router + static_cast<std::size_t>(e) * width;
     float sum = 0.0F;
     if constexpr (kVector) {
@@ -104,13 +103,19 @@ route_rows_kernel(const T *__restrict__ input, const bf16 *__restrict__ router, 
       for (int k = lane; k < width; k += 32) sum = fmaf(to_float(x[k]), bf2f(w[k]), sum);
     }
     sum = warp_sum(sum);
-    if (lane == 0) target[e] = sum;
+    if (lane == 0) logits[e / kRouterSplits] = sum;
   }
   cluster.sync();
-  if (split != 0 || warp != 0) return;
   float logit[kPerLane];
+  if (split == 0 && warp == 0) {
 #pragma unroll
-  for (int i = 0; i < kPerLane; ++i) logit[i] = lane + 32 * i < c.experts ? logits[lane + 32 * i] : -INFINITY;
+    for (int i = 0; i < kPerLane; ++i) {
+      const int e = lane + 32 * i;
+      logit[i] = e < c.experts ? cluster.map_shared_rank(logits, e % kRouterSplits)[e / kRouterSplits] : -INFINITY;
+    }
+  }
+  cluster.sync();  // remote shared memory stays alive until rank 0 has read it
+  if (split != 0 || warp != 0) return;
   choose<kPerLane>(logit, c, row, lane);
 }
 

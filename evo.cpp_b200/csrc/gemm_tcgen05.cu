@@ -133,6 +133,8 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
   const int chunks = gated ? BN / 64 : BN / 32;
   float *const f32_base =
       ep.out_f32 != nullptr ? ep.out_f32 + static_cast<std::size_t>(split) * ep.partial_stride : nullptr;
+  const bool plain = ep.gate_mode == 0 && ep.bias_mode == 0 && ep.residual == nullptr && ep.out_f32 == nullptr &&
+                     (ep.ld_out % 8) == 0 && (reinterpret_cast<std::uintptr_t>(ep.out) & 15U) == 0;
   const bool f32_vectors = ep.out_f32 != nullptr && (ep.ld_out % 4) == 0 && (ep.partial_stride % 4) == 0 && (N % 4) == 0 &&
                            (reinterpret_cast<std::uintptr_t>(ep.out_f32) & 15U) == 0;
   float4 old[8];
@@ -141,12 +143,13 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const int r = m0 + quarter * 32 + 4 * i + lane / 8;
-      old[i] = ep.accumulate_f32 != 0 && r < M && at < N
+      old[i] = r < M && at < N
                    ? *reinterpret_cast<const float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at)
                    : make_float4(0.0F, 0.0F, 0.0F, 0.0F);
     }
   };
-  if (f32_vectors) fetch_old(0);
+  const bool accumulating = f32_vectors && ep.accumulate_f32 != 0;
+  if (accumulating) fetch_old(0);
   for (int c = 0; c < chunks; ++c) {
     std::uint32_t v[32];
     std::uint32_t w[32];
@@ -167,14 +170,16 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
         __syncwarp();
         float4 sums[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const float4 value =
-              *reinterpret_cast<const float4 *>(staging + (4 * i + lane / 8) * kStagingStride + (lane % 8) * 4);
-          sums[i] = make_float4(value.x + old[i].x, value.y + old[i].y, value.z + old[i].z, value.w + old[i].w);
+        for (int i = 0; i < 8; ++i)
+          sums[i] = *reinterpret_cast<const float4 *>(staging + (4 * i + lane / 8) * kStagingStride + (lane % 8) * 4);
+        if (ep.accumulate_f32 != 0) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            sums[i] = make_float4(sums[i].x + old[i].x, sums[i].y + old[i].y, sums[i].z + old[i].z, sums[i].w + old[i].w);
         }
         __syncwarp();
         const int at = n0 + c * 32 + (lane % 8) * 4;
-        if (c + 1 < chunks) fetch_old(c + 1);
+        if (accumulating && c + 1 < chunks) fetch_old(c + 1);
         if (ep.softcap > 0.0F) {  // (capped results carry no bias)
 #pragma unroll
           for (int i = 0; i < 8; ++i)
@@ -182,15 +187,16 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
                                   fast_soft_cap(sums[i].z, ep.softcap), fast_soft_cap(sums[i].w, ep.softcap));
         }
         if (at < n_limit) {
-          float4 shift = make_float4(0.0F, 0.0F, 0.0F, 0.0F);
-          if (ep.bias_f32 != nullptr)
-            shift = make_float4(ep.bias_f32[at], ep.bias_f32[at + 1], ep.bias_f32[at + 2], ep.bias_f32[at + 3]);
+          if (ep.bias_f32 != nullptr) {
+            const float4 shift = make_float4(ep.bias_f32[at], ep.bias_f32[at + 1], ep.bias_f32[at + 2], ep.bias_f32[at + 3]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              sums[i] = make_float4(sums[i].x + shift.x, sums[i].y + shift.y, sums[i].z + shift.z, sums[i].w + shift.w);
+          }
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const int r = m0 + quarter * 32 + 4 * i + lane / 8;
-            if (r < M)
-              *reinterpret_cast<float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at) =
-                  make_float4(sums[i].x + shift.x, sums[i].y + shift.y, sums[i].z + shift.z, sums[i].w + shift.w);
+            if (r < M) *reinterpret_cast<float4 *>(f32_base + static_cast<std::size_t>(r) * ep.ld_out + at) = sums[i];
           }
         }
         continue;
@@ -205,6 +211,21 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
             if (ep.accumulate_f32 != 0) value += out_row[col + j];
             out_row[col + j] = fast_soft_cap(value, ep.softcap);
           }
+        }
+      }
+      continue;
+    }
+    if (plain && col + 32 <= n_limit) {
+      // the accumulators alone, whole 16-byte words: the same values as below
+      if (row < M) {
+        uint4 *const out_words = reinterpret_cast<uint4 *>(ep.out + static_cast<std::size_t>(row) * ep.ld_out + col);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          std::uint32_t words[4];
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            words[i] = pack_bf16x2(__uint_as_float(v[8 * q + 2 * i]) * scale, __uint_as_float(v[8 * q + 2 * i + 1]) * scale);
+          out_words[q] = make_uint4(words[0], words[1], words[2], words[3]);
         }
       }
       continue;
@@ -228,21 +249,20 @@ __device__ __forceinline__ void epilogue_tile(const EpilogueParams &ep, const in
 #pragma unroll
         for (int j = 0; j < 32; ++j)
           r[j] = clamped_gate<true>(ep.gate_limit, __uint_as_float(v[j]) * scale, __uint_as_float(w[j]) * scale);
-      } else
+      } else if (ep.gate_mode == kGateGelu) {
 #pragma unroll
-      for (int j = 0; j < 32; ++j) {
-        float value = __uint_as_float(v[j]) * scale;
-        if (gated) {
-          const float first =
-              ep.gate_mode == 2 ? bf2f(gelu_round(value)) : rbf(value);
-          const float second = rbf(__uint_as_float(w[j]) * scale);
-          r[j] = rbf(first * second);
-        } else {
-          if (ep.bias_mode == 1 && col + j < n_limit)
-            value += bf2f(ep.bias[col + j]);
+        for (int j = 0; j < 32; ++j)
+          r[j] = rbf(bf2f(gelu_round(__uint_as_float(v[j]) * scale)) * rbf(__uint_as_float(w[j]) * scale));
+      } else if (gated) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) r[j] = rbf(rbf(__uint_as_float(v[j]) * scale) * rbf(__uint_as_float(w[j]) * scale));
+      } else {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          float value = __uint_as_float(v[j]) * scale;
+          if (ep.bias_mode == 1 && col + j < n_limit) value += bf2f(ep.bias[col + j]);
           value = rbf(value);
-          if (ep.bias_mode == 2 && col + j < n_limit)
-            value = rbf(value + bf2f(ep.bias[col + j]));
+          if (ep.bias_mode == 2 && col + j < n_limit) value = rbf(value + bf2f(ep.bias[col + j]));
           r[j] = value;
         }
       }

@@ -302,7 +302,7 @@ latent_decode_kernel(const LatentDecodeParams p) {
     __syncthreads();
     const bf16 *const tile = tiles + (t & 1) * kTokens * kStride;
     // scores of tokens 8 warp .. 8 warp + 7
-    float s[4] = {0.0F, 0.0F, 0.0F, 0.0F};
+    float s[4] = {0.0F, 0.0F, 0.0F, 0.0F}, s_odd[4] = {0.0F, 0.0F, 0.0F, 0.0F};  // two chains of MMAs
     const std::uint32_t key_address = shared_address(tile + (8 * warp + lane % 8) * kStride + (lane / 8) * 8);
 #pragma unroll
     for (int k = 0; k < kRank / 32; ++k) {  // 32 columns: two MMAs
@@ -311,10 +311,11 @@ latent_decode_kernel(const LatentDecodeParams p) {
       load_matrices(query_address + k * 64U, a0);
       load_matrices(query_address + k * 64U + 32U, a1);
       mma_bf16(s, a0, b[0], b[1]);
-      mma_bf16(s, a1, b[2], b[3]);
+      mma_bf16(s_odd, a1, b[2], b[3]);
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
+      s[i] += s_odd[i];
       const int token = 8 * warp + 2 * (lane % 4) + i % 2, head = lane / 4 + 8 * (i / 2);
       scores[head * kScoreStride + token] = begin + t * kTokens + token < end ? s[i] * p.scale : -INFINITY;
     }
@@ -376,26 +377,36 @@ latent_decode_kernel(const LatentDecodeParams p) {
     *reinterpret_cast<float2 *>(partial + (lane / 4 + 8) * kRank + column) = make_float2(out[n][2], out[n][3]);
   }
   cluster.sync();
-  // this CTA's share of the columns: kRank / kSplits
-  constexpr int kShare = kRank / kSplits;
+  // this CTA's share of the columns, four at a time
+  constexpr int kShare = kRank / kSplits / 4;
   for (int i = threadIdx.x; i < kHeadGroup * kShare; i += kThreads) {
-    const int head = i / kShare, column = split * kShare + i % kShare;
+    const int head = i / kShare, column = 4 * (split * kShare + i % kShare);
     if (head0 + head >= p.heads) continue;
-    float peak = p.sink_logit != nullptr ? p.sink_logit[head0 + head] : -INFINITY;
-    float maxima[kSplits];
+    const float sink = p.sink_logit != nullptr ? p.sink_logit[head0 + head] : -INFINITY;
+    float maxima[kSplits], sums[kSplits];
+    float4 parts[kSplits];
 #pragma unroll
     for (int other = 0; other < kSplits; ++other) {
       maxima[other] = cluster.map_shared_rank(head_max, other)[head];
-      peak = fmaxf(peak, maxima[other]);
+      sums[other] = cluster.map_shared_rank(head_sum, other)[head];
+      parts[other] = *reinterpret_cast<const float4 *>(cluster.map_shared_rank(partial, other) + head * kRank + column);
     }
-    float total = p.sink_logit != nullptr ? expf(p.sink_logit[head0 + head] - peak) : 0.0F, sum = 0.0F;
+    float peak = sink;
+#pragma unroll
+    for (int other = 0; other < kSplits; ++other) peak = fmaxf(peak, maxima[other]);
+    float total = expf(sink - peak);  // 0 without a sink
+    float4 mixed = make_float4(0.0F, 0.0F, 0.0F, 0.0F);
 #pragma unroll
     for (int other = 0; other < kSplits; ++other) {
       const float factor = expf(maxima[other] - peak);  // 0 for a CTA without tokens
-      total = fmaf(cluster.map_shared_rank(head_sum, other)[head], factor, total);
-      sum = fmaf(cluster.map_shared_rank(partial, other)[head * kRank + column], factor, sum);
+      total = fmaf(sums[other], factor, total);
+      mixed.x = fmaf(parts[other].x, factor, mixed.x);
+      mixed.y = fmaf(parts[other].y, factor, mixed.y);
+      mixed.z = fmaf(parts[other].z, factor, mixed.z);
+      mixed.w = fmaf(parts[other].w, factor, mixed.w);
     }
-    p.output[(static_cast<std::size_t>(row) * p.heads + head0 + head) * kRank + column] = f2bf(sum / total);
+    const float y[4] = {mixed.x / total, mixed.y / total, mixed.z / total, mixed.w / total};
+    store_quad(p.output + (static_cast<std::size_t>(row) * p.heads + head0 + head) * kRank + column, y);
   }
   cluster.sync();  // remote shared memory stays alive until every CTA has read it
 }
@@ -511,7 +522,7 @@ bool latent_decode_applicable(const WindowAttentionArgs &a) {
   return a.type == Activation::kBf16 && a.kv_heads == 1 && a.key_cache == a.value_cache && a.dim == a.value_dim &&
          a.dim % 64 == 0 && a.dim <= static_cast<std::size_t>(kWidestTile) && a.keep_first == 0 && a.softcap == 0.0F &&
          a.distance_bias == nullptr && a.gate == nullptr && (!a.sink || a.sink_logit != nullptr) && a.rows > 0 &&
-         a.rows <= 65535 && a.heads <= 65535 && aligned16(a.query) && aligned16(a.key_cache) &&
+         a.rows <= 65535 && a.heads <= 65535 && aligned16(a.query) && aligned16(a.key_cache) && aligned16(a.output) &&
          a.position + a.rows < 0x7fff0000U;
 }
 
