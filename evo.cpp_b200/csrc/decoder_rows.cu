@@ -220,8 +220,9 @@ struct LayerNormParams {
   float epsilon;
 };
 
-// Mean and variance from the row itself (two sweeps over registers), one read and one write of the residual.
-template <typename In, typename Out, bool kVector>
+// Mean and variance from the row itself (two sweeps over registers), one read and one write of the residual.  A
+// thread keeps kKeep groups of eight elements between the sweeps.
+template <typename In, typename Out, bool kVector, int kKeep>
 __global__ void __launch_bounds__(kThreads)
 layer_norm_kernel(const In *__restrict__ input, Out *__restrict__ output, const LayerNormParams p) {
   // a one-row projection launched with programmatic stream serialisation may start under this kernel
@@ -243,10 +244,10 @@ layer_norm_kernel(const In *__restrict__ input, Out *__restrict__ output, const 
     }
   };
   const auto live = [&](const int group, const int i) { return kVector || 8 * group + i < p.width; };
-  float cached[kCached][8], old[kCached][8];
+  float cached[kKeep][8], old[kKeep][8];
   float sum = 0.0F;
 #pragma unroll
-  for (int c = 0; c < kCached; ++c) {
+  for (int c = 0; c < kKeep; ++c) {
     const int group = threadIdx.x + c * kThreads;
     if (group < groups) {
       load(group, cached[c]);
@@ -255,7 +256,7 @@ layer_norm_kernel(const In *__restrict__ input, Out *__restrict__ output, const 
       for (int i = 0; i < 8; ++i) sum += cached[c][i];
     }
   }
-  for (int group = threadIdx.x + kCached * kThreads; group < groups; group += kThreads) {
+  for (int group = threadIdx.x + kKeep * kThreads; group < groups; group += kThreads) {
     float v[8];
     load(group, v);
 #pragma unroll
@@ -271,11 +272,11 @@ layer_norm_kernel(const In *__restrict__ input, Out *__restrict__ output, const 
     }
   };
 #pragma unroll
-  for (int c = 0; c < kCached; ++c) {
+  for (int c = 0; c < kKeep; ++c) {
     const int group = threadIdx.x + c * kThreads;
     if (group < groups) deviate(group, cached[c]);
   }
-  for (int group = threadIdx.x + kCached * kThreads; group < groups; group += kThreads) {
+  for (int group = threadIdx.x + kKeep * kThreads; group < groups; group += kThreads) {
     float v[8];
     load(group, v);
     deviate(group, v);
@@ -294,11 +295,11 @@ layer_norm_kernel(const In *__restrict__ input, Out *__restrict__ output, const 
     if (output != nullptr) store_group<Out, kVector>(output + row * p.width, group, p.width, y);
   };
 #pragma unroll
-  for (int c = 0; c < kCached; ++c) {
+  for (int c = 0; c < kKeep; ++c) {
     const int group = threadIdx.x + c * kThreads;
     if (group < groups) emit(group, cached[c], old[c]);
   }
-  for (int group = threadIdx.x + kCached * kThreads; group < groups; group += kThreads) {
+  for (int group = threadIdx.x + kKeep * kThreads; group < groups; group += kThreads) {
     float v[8], before[8] = {};
     load(group, v);
     if (p.residual != nullptr) load_group<float, kVector>(p.residual + row * p.width, group, p.width, before);
@@ -534,7 +535,10 @@ int layer_norm(const LayerNormArgs &a, cudaStream_t stream) {
   const auto launch = [&](auto in_tag, auto out_tag) {
     using In = decltype(in_tag);
     using Out = decltype(out_tag);
-    const auto kernel = vector ? layer_norm_kernel<In, Out, true> : layer_norm_kernel<In, Out, false>;
+    const auto kernel = !vector                      ? layer_norm_kernel<In, Out, false, kCached>
+                        : a.width <= 8 * kThreads  ? layer_norm_kernel<In, Out, true, 1>
+                        : a.width <= 16 * kThreads ? layer_norm_kernel<In, Out, true, 2>
+                                                   : layer_norm_kernel<In, Out, true, kCached>;
     kernel<<<static_cast<unsigned int>(a.rows), kThreads, 0, stream>>>(static_cast<const In *>(a.input),
                                                                        static_cast<Out *>(a.output), p);
   };

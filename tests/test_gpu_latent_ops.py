@@ -58,7 +58,7 @@ def assert_near(actual, expected, float32, factor=1.0):
 # ---------------------------------------------------------------- norms and embedding
 @TYPES
 @pytest.mark.parametrize("input32", [0, 1])
-@pytest.mark.parametrize("width", [1, 8, 77, 1536, 8200, 16392])
+@pytest.mark.parametrize("width", [1, 8, 77, 1536, 2056, 4104, 8200, 16392])
 def test_layer_norm(pkg, ops, float32, input32, width):
     rng = np.random.default_rng(width)
     rows, parts, eps = 5, 3, 1e-3
